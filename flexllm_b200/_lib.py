@@ -5,6 +5,7 @@ import os
 _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.environ.get("FLEXLLM_B200_LIB") or os.path.join(_HERE, "libflexllm_b200.so")   # the override is a development aid
 
+F32, BF16 = 0, 1
 OK, EINVAL, ECUDA, ETIMEDOUT, ENOTSUP, ENOMEM, ETOOBIG, EDEVDATA, EIO = 0, -1, -2, -3, -4, -5, -6, -7, -8
 
 # name -> argument types, in the order of include/flexllm_b200.h (return type is int unless noted)
@@ -47,6 +48,7 @@ SIGNATURES = {
     "flexllm_mha_i8xi8_prefill": [_P] * 9 + [_I, _I, _I, _I, _P, _P, _P, _SZ, _P],
     "flexllm_mha_i8xi8_prefill_online": [_P] * 8 + [_I, _I, _I, _I, _P, _P, _SZ, _P],
     "flexllm_kv_cache_create": [_P, _I, _I, _I, _I],
+    "flexllm_kv_cache_create_float": [_P, _I, _I, _P, _I, _I],
     "flexllm_kv_cache_destroy": [_P],
     "flexllm_kv_cache_reset": [_P, _P],
     "flexllm_kv_cache_pools": [_P, _I, _P, _P, _P, _P],
@@ -73,6 +75,15 @@ SIGNATURES = {
     "flexllm_model_prefill": [_P, _P, _I, _I, _P, _P],
     "flexllm_model_prefill_embeds": [_P, _P, _I, _I, _I, _P, _P],
     "flexllm_model_embed_tokens": [_P, _P, _I, _P, _P],
+    "flexllm_model_extend": [_P, _P, _I, _I, _P, _I, _P, _P, _P],
+    "flexllm_model_extend_host": [_P, _P, _I, _I, _P, _I, _P, _P, _P],
+    "flexllm_model_reset": [_P, _P],
+    "flexllm_model_create_decoder": [_P, _P],
+    "flexllm_model_load_tensor": [_P, C.c_char_p, _I, _I, _P, _P, _P],
+    "flexllm_model_load_safetensors": [_P, C.c_char_p, _P],
+    "flexllm_model_set_trace": [_P, _P, _SZ],
+    "flexllm_linear_float": [_I, _P, _L, _P, _L, _P, _I, _I, _I, _I, _P, _L, _I, _P],
+    "flexllm_sandwich_norm": [_I, _P, _L, _I, _I, _F, _P, _L, _P, _P, _P, _P, _L, _P],
     "flexllm_hmt_create": [_P, _P, _P, _I, _P, _P, _P],
     "flexllm_hmt_destroy": [_P],
     "flexllm_hmt_prefill": [_P, _P, _I, _P, _P, _P],
@@ -80,6 +91,7 @@ SIGNATURES = {
     "flexllm_model_decode": [_P, _I, _I, _P],
     "flexllm_model_generate_host": [_P, _P, _I, _I, _I, _P, _I, _P],
     "flexllm_model_set_sampling": [_P, _I, _I, _P],
+    "flexllm_model_set_sampling_host": [_P, _I, _I, _P, _I, _I],
     "flexllm_model_buffer": [_P, _I, _P],
     "flexllm_model_limits": [_P, _P, _P, _P],
     "flexllm_debug_hook": [_I, C.c_longlong],
@@ -90,6 +102,16 @@ SIGNATURES = {
 class ModelConfig(C.Structure):
     _fields_ = [("layers", _I), ("hidden", _I), ("heads_q", _I), ("heads_kv", _I), ("ffn", _I), ("vocab", _I),
                 ("eps", _F), ("fht_scale", _F), ("max_batch", _I), ("max_prefill", _I), ("max_ctx", _I)]
+
+
+class DecoderLayer(C.Structure):
+    _fields_ = [("heads", _I), ("kv_heads", _I), ("dim", _I), ("vdim", _I), ("window", _I), ("bias_max", _I), ("scale", _F), ("softcap", _F),
+                ("ff", _I)]
+
+
+class DecoderConfig(C.Structure):
+    _fields_ = [("layers", _I), ("width", _I), ("vocab", _I), ("eps", _F), ("embed_scale", _F), ("loop_start", _I), ("loop_stop", _I),
+                ("loop_times", _I), ("max_batch", _I), ("max_prefill", _I), ("max_ctx", _I), ("dtype", _I), ("layer", C.POINTER(DecoderLayer))]
 
 
 class CkptLayerBuffers(C.Structure):

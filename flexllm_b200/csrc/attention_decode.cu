@@ -343,7 +343,7 @@ extern "C" int flexllm_kv_cache_create(flexllm_kv_cache** out, int layers, int n
     if (page != PAGE) return FLEXLLM_ENOTSUP;
     flexllm_kv_cache* c = new (std::nothrow) flexllm_kv_cache();
     if (!c) return FLEXLLM_ENOMEM;
-    c->layers = layers; c->n_pages = n_pages; c->hkv = hkv; c->page = page;
+    c->layers = layers; c->n_pages = n_pages; c->hkv = hkv; c->page = page; c->elem_bytes = 1; c->k_bytes = c->v_bytes = 0;
     c->page_bytes = (size_t)n_pages * hkv * PAGE * 64;
     c->scale_bytes = (size_t)n_pages * hkv * PAGE * sizeof(float);
     c->k = c->v = nullptr; c->ks = c->vs = nullptr;
@@ -351,6 +351,36 @@ extern "C" int flexllm_kv_cache_create(flexllm_kv_cache** out, int layers, int n
     if (e == cudaSuccess) e = cudaMalloc(&c->v, c->page_bytes * layers);
     if (e == cudaSuccess) e = cudaMalloc(&c->ks, c->scale_bytes * layers);
     if (e == cudaSuccess) e = cudaMalloc(&c->vs, c->scale_bytes * layers);
+    if (e != cudaSuccess) {
+        flexllm_kv_cache_destroy(c);
+        g_last_cuda_error = (int)e;
+        return e == cudaErrorMemoryAllocation ? FLEXLLM_ENOMEM : FLEXLLM_ECUDA;
+    }
+    *out = c;
+    return flexllm_kv_cache_reset(c, nullptr);
+}
+
+// Floating-point flavour: one pool pair per layer, each with its own shape (256-byte aligned inside two allocations).
+extern "C" int flexllm_kv_cache_create_float(flexllm_kv_cache** out, int layers, int n_pages, const flexllm_kv_shape* shapes, int page,
+                                             int elem_bytes) {
+    FLEXLLM_REQUIRE(out && layers > 0 && n_pages > 0 && shapes && (elem_bytes == 2 || elem_bytes == 4));
+    if (page != PAGE) return FLEXLLM_ENOTSUP;
+    for (int l = 0; l < layers; l++) FLEXLLM_REQUIRE(shapes[l].hkv > 0 && shapes[l].kdim > 0 && shapes[l].vdim > 0);
+    flexllm_kv_cache* c = new (std::nothrow) flexllm_kv_cache();
+    if (!c) return FLEXLLM_ENOMEM;
+    c->layers = layers; c->n_pages = n_pages; c->hkv = 0; c->page = page; c->elem_bytes = elem_bytes;
+    c->page_bytes = c->scale_bytes = 0;
+    c->k = c->v = nullptr; c->ks = c->vs = nullptr;
+    c->shape.assign(shapes, shapes + layers);
+    size_t nk = 0, nv = 0;
+    for (int l = 0; l < layers; l++) {
+        c->k_off.push_back(nk); c->v_off.push_back(nv);
+        nk += align_up((size_t)n_pages * shapes[l].hkv * PAGE * shapes[l].kdim * elem_bytes, 256);
+        nv += align_up((size_t)n_pages * shapes[l].hkv * PAGE * shapes[l].vdim * elem_bytes, 256);
+    }
+    c->k_bytes = nk; c->v_bytes = nv;
+    cudaError_t e = cudaMalloc(&c->k, nk);
+    if (e == cudaSuccess) e = cudaMalloc(&c->v, nv);
     if (e != cudaSuccess) {
         flexllm_kv_cache_destroy(c);
         g_last_cuda_error = (int)e;
@@ -370,6 +400,11 @@ extern "C" int flexllm_kv_cache_destroy(flexllm_kv_cache* c) {
 extern "C" int flexllm_kv_cache_reset(flexllm_kv_cache* c, void* stream) {
     FLEXLLM_REQUIRE(c);
     cudaStream_t st = (cudaStream_t)stream;
+    if (c->elem_bytes != 1) {
+        FLEXLLM_CHECK_CUDA(cudaMemsetAsync(c->k, 0, c->k_bytes, st));
+        FLEXLLM_CHECK_CUDA(cudaMemsetAsync(c->v, 0, c->v_bytes, st));
+        return FLEXLLM_OK;
+    }
     FLEXLLM_CHECK_CUDA(cudaMemsetAsync(c->k, 0, c->page_bytes * c->layers, st));
     FLEXLLM_CHECK_CUDA(cudaMemsetAsync(c->v, 0, c->page_bytes * c->layers, st));
     FLEXLLM_CHECK_CUDA(cudaMemsetAsync(c->ks, 0, c->scale_bytes * c->layers, st));
@@ -379,6 +414,13 @@ extern "C" int flexllm_kv_cache_reset(flexllm_kv_cache* c, void* stream) {
 
 extern "C" int flexllm_kv_cache_pools(flexllm_kv_cache* c, int layer, int8_t** k, float** ks, int8_t** v, float** vs) {
     FLEXLLM_REQUIRE(c && layer >= 0 && layer < c->layers);
+    if (c->elem_bytes != 1) {
+        if (k) *k = c->k + c->k_off[layer];
+        if (ks) *ks = nullptr;
+        if (v) *v = c->v + c->v_off[layer];
+        if (vs) *vs = nullptr;
+        return FLEXLLM_OK;
+    }
     KvLayer l = kv_layer(c, layer);
     if (k) *k = l.k;
     if (ks) *ks = l.ks;
@@ -414,7 +456,7 @@ int mha_decode_run(flexllm_kv_cache* c, int layer, const int8_t* q, const float*
 // Modules/MHA.h:484-513, :773-801): store the new token's K and V heads at position ctx[b], nothing else.
 extern "C" int flexllm_kv_append(flexllm_kv_cache* c, int layer, const int8_t* k, const float* ks, const int8_t* v, const float* vs,
                                  const int32_t* page_table, int max_pages, const int32_t* ctx, int max_ctx, int B, void* stream) {
-    FLEXLLM_REQUIRE(c && layer >= 0 && layer < c->layers && B >= 0 && max_ctx >= 0 && max_pages > 0);
+    FLEXLLM_REQUIRE(c && c->elem_bytes == 1 && layer >= 0 && layer < c->layers && B >= 0 && max_ctx >= 0 && max_pages > 0);
     if (B == 0) return FLEXLLM_OK;
     FLEXLLM_REQUIRE(k && ks && v && vs && page_table && ctx);
     FLEXLLM_REQUIRE((long)max_pages * PAGE > max_ctx);
@@ -430,7 +472,7 @@ extern "C" int flexllm_mha_i8xi8_decode(flexllm_kv_cache* c, int layer, const in
                                         const int32_t* page_table, int max_pages, const int32_t* ctx, int max_ctx,
                                         int B, int HQ, float* out, int32_t* oacc, void* workspace,
                                         size_t workspace_bytes, void* stream) {
-    FLEXLLM_REQUIRE(c && layer >= 0 && layer < c->layers && B >= 0 && HQ > 0 && max_ctx >= 0 && max_pages > 0);
+    FLEXLLM_REQUIRE(c && c->elem_bytes == 1 && layer >= 0 && layer < c->layers && B >= 0 && HQ > 0 && max_ctx >= 0 && max_pages > 0);
     if (B == 0) return FLEXLLM_OK;
     FLEXLLM_REQUIRE(q && qs && k && ks && v && vs && cos_t && sin_t && a_s && page_table && ctx && out && workspace);
     FLEXLLM_REQUIRE(HQ % c->hkv == 0);

@@ -2,14 +2,8 @@
 // paged KV-cache view and the fused per-(sequence, KV head) attention step.
 #pragma once
 #include "common.cuh"
+#include "kv_cache.h"
 #include "tc_common.cuh"
-
-// Paged int8 KV cache, all layers (layout at the top of attention_decode.cu).
-struct flexllm_kv_cache {
-    int layers, n_pages, hkv, page;
-    int8_t* k; float* ks; int8_t* v; float* vs;   // [layers][...]
-    size_t page_bytes, scale_bytes;               // per layer
-};
 
 namespace flexllm {
 

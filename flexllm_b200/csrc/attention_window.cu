@@ -1,0 +1,693 @@
+// Sliding-window grouped-query attention over the paged cache, floating point (bf16, or fp32 in the 32-bit mode):
+//   q, k = rms norm over the whole projection, before the split into heads
+//   s    = softcap * tanh(scale * (q . k) / softcap) + bias[head][i - j]          0 <= i - j < window
+//   p    = exp(s) / (sink + sum exp(s)),   out = (sum p v) * logistic(gate)
+// Softcap, sink and gate are optional; the distance bias and the window are one table per layer (-inf outside the
+// window), so that a masked key costs nothing extra. Scores, weights and sums are fp32.
+//
+// Cache pages hold 64 tokens, K [page][G][64][dkp] and V transposed [page][G][dv][64] (as the int8 cache does).
+//   one token per sequence : attn_row_kernel<FUSED>: norms, append and attention in one launch, keys split over CTAs
+//   prompts, bf16          : attn_prepare_kernel, then attn_window_prefill_kernel on tcgen05
+//   prompts, otherwise     : attn_prepare_kernel, then attn_row_kernel row by row
+// The sink is a score of 0, so max(0, largest score) is a valid softmax shift; without a sink the running maximum is.
+#include <math.h>
+
+#include <atomic>
+
+#include "float_common.cuh"
+#include "tc_common.cuh"
+
+namespace flexllm {
+
+using namespace tc;
+
+namespace {
+
+constexpr int PG = 64;                     // tokens per page
+constexpr int TILE_PAGES = 4;              // pages per key tile of the row kernel
+constexpr int TILE_KEYS = TILE_PAGES * PG;
+
+// Start position of sequence b; a value that would leave the page-table row is clamped and reported.
+__device__ __forceinline__ int start_pos(const AttnCall& c, int b, int* error_flag) {
+    int pos = c.ctx[b];
+    if (pos < 0 || pos + c.Sc - 1 > c.max_pos) {
+        if (error_flag) atomicOr(error_flag, 2);
+        pos = pos < 0 ? 0 : c.max_pos - (c.Sc - 1);
+    }
+    return pos;
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Norm of q and k over their whole projections, q to the scratch, k rows and v columns to the pages.
+// CTAs 0 .. B*Sc-1: one row each. The rest: one (page, V head, sequence) each, transposing through shared memory.
+template <class T>
+__global__ void __launch_bounds__(256) attn_prepare_kernel(const AttnCall c, int v_pages, int* error_flag) {
+    __shared__ float red[16];
+    __shared__ T tile[PG][PG + 2];
+    pdl_sync();
+    const AttnShape& s = c.s;
+    const int rows = c.B * c.Sc, tid = threadIdx.x;
+    if ((int)blockIdx.x < rows) {
+        const int m = blockIdx.x, b = m / c.Sc;
+        const int pos = start_pos(c, b, error_flag) + m % c.Sc;
+        const T* src = (const T*)c.proj + (long)m * s.ld;
+        const int nq = s.H * s.dk, nk = s.G * s.dk;
+        float sq = 0.0f, sk = 0.0f;
+        for (int i = tid; i < nq; i += 256) { const float v = to_f(src[s.q_off + i]); sq = __fmaf_rn(v, v, sq); }
+        for (int i = tid; i < nk; i += 256) { const float v = to_f(src[s.k_off + i]); sk = __fmaf_rn(v, v, sk); }
+        const float2 ss = block_sum2<256>(sq, sk, red);
+        const float rq = 1.0f / sqrtf(ss.x / (float)nq + c.eps), rk = 1.0f / sqrtf(ss.y / (float)nk + c.eps);
+        T* q = (T*)c.q + (long)m * s.H * s.dkp;
+        for (int i = tid; i < s.H * s.dkp; i += 256) {
+            const int h = i / s.dkp, e = i - h * s.dkp, j = h * s.dk + e;
+            q[i] = from_f<T>(e < s.dk ? (to_f(src[s.q_off + j]) * rq) * c.q_gain[j] : 0.0f);
+        }
+        const long page = c.page_table[(long)b * c.max_pages + pos / PG];
+        T* kp = (T*)c.k_pool + (page * s.G * PG + (pos & (PG - 1))) * s.dkp;
+        for (int i = tid; i < s.G * s.dkp; i += 256) {
+            const int g = i / s.dkp, e = i - g * s.dkp, j = g * s.dk + e;
+            kp[(long)g * PG * s.dkp + e] = from_f<T>(e < s.dk ? (to_f(src[s.k_off + j]) * rk) * c.k_gain[j] : 0.0f);
+        }
+        return;
+    }
+    int id = blockIdx.x - rows;
+    const int pi = id % v_pages; id /= v_pages;
+    const int g = id % s.G, b = id / s.G;
+    const int p0 = start_pos(c, b, error_flag);
+    const int page_i = p0 / PG + pi;
+    const int lo = max(p0, page_i * PG), hi = min(p0 + c.Sc, (page_i + 1) * PG);     // positions [lo, hi)
+    if (lo >= hi) return;
+    const long page = c.page_table[(long)b * c.max_pages + page_i];
+    T* vp = (T*)c.v_pool + (page * s.G + g) * (long)s.dv * PG;
+    const T* src = (const T*)c.proj + ((long)b * c.Sc + (lo - p0)) * s.ld + s.v_off + g * s.dv;
+    const int n = hi - lo, slot0 = lo & (PG - 1);
+    for (int d0 = 0; d0 < s.dv; d0 += PG) {
+        const int nd = min(PG, s.dv - d0);
+        for (int i = tid; i < n * PG; i += 256) {
+            const int t = i >> 6, d = i & (PG - 1);
+            if (d < nd) tile[t][d] = src[(long)t * s.ld + d0 + d];
+        }
+        __syncthreads();
+        for (int i = tid; i < nd * PG; i += 256) {
+            const int d = i >> 6, t = i & (PG - 1);
+            if (t < n) vp[(long)(d0 + d) * PG + slot0 + t] = tile[t][d];
+        }
+        __syncthreads();
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// One query row (position) x one key/value head per CTA, its keys split over gridDim.x CTAs.
+// RC: query heads handled at a time; L lanes share a key (8 elements each, WIDE: several times 8).
+struct RowSmem { long q, sc, o, m, l, al, total; };
+__host__ __device__ inline RowSmem row_smem(int R, int dkp, int dv) {
+    RowSmem r;
+    r.q = 0;                                    // [R][dkp]
+    r.sc = r.q + (long)R * dkp;                 // [R][TILE_KEYS]
+    r.o = r.sc + (long)R * TILE_KEYS;           // [R][dv]
+    r.m = r.o + (((long)R * dv + 3) & ~3L);
+    r.l = r.m + R; r.al = r.l + R;
+    r.total = r.al + R;
+    return r;
+}
+
+template <class T, int RC, bool FUSED, bool WIDE>
+__global__ void __launch_bounds__(256) attn_row_kernel(const AttnCall c, int L, int* error_flag) {
+    constexpr bool FAST = sizeof(T) == 2;
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float red[16];
+    __shared__ int last_sm;
+    const AttnShape& s = c.s;
+    const int R = s.H / s.G;
+    const RowSmem o = row_smem(R, s.dkp, s.dv);
+    float *q_sm = sm + o.q, *s_sm = sm + o.sc, *o_sm = sm + o.o, *m_sm = sm + o.m, *l_sm = sm + o.l, *al_sm = sm + o.al;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+    const int split = blockIdx.x, n_split = gridDim.x, g = blockIdx.y, row = blockIdx.z;
+    pdl_sync();
+    const int b = row / c.Sc;
+    const int pos = start_pos(c, b, error_flag) + row % c.Sc;
+    const int32_t* pt = c.page_table + (long)b * c.max_pages;
+    const T* prow = (const T*)c.proj + (long)row * s.ld;
+    const long kh = (long)PG * s.dkp, vh = (long)PG * s.dv;          // one head of a page
+    if (FUSED) {
+        const int nq = s.H * s.dk, nk = s.G * s.dk;
+        float sq = 0.0f, sk = 0.0f;
+        for (int i = tid; i < nq; i += 256) { const float v = to_f(prow[s.q_off + i]); sq = __fmaf_rn(v, v, sq); }
+        for (int i = tid; i < nk; i += 256) { const float v = to_f(prow[s.k_off + i]); sk = __fmaf_rn(v, v, sk); }
+        const float2 ss = block_sum2<256>(sq, sk, red);
+        const float rq = 1.0f / sqrtf(ss.x / (float)nq + c.eps), rk = 1.0f / sqrtf(ss.y / (float)nk + c.eps);
+        for (int i = tid; i < R * s.dkp; i += 256) {
+            const int r = i / s.dkp, e = i - r * s.dkp, j = (g * R + r) * s.dk + e;
+            q_sm[i] = e < s.dk ? (to_f(prow[s.q_off + j]) * rq) * c.q_gain[j] : 0.0f;
+        }
+        if (split == n_split - 1) {               // the split that holds the newest key appends it
+            const long page = pt[pos / PG];
+            const int slot = pos & (PG - 1);
+            T* kp = (T*)c.k_pool + (page * s.G + g) * kh + (long)slot * s.dkp;
+            for (int e = tid; e < s.dkp; e += 256) {
+                const int j = g * s.dk + e;
+                kp[e] = from_f<T>(e < s.dk ? (to_f(prow[s.k_off + j]) * rk) * c.k_gain[j] : 0.0f);
+            }
+            T* vp = (T*)c.v_pool + (page * s.G + g) * vh + slot;
+            for (int d = tid; d < s.dv; d += 256) vp[(long)d * PG] = prow[s.v_off + g * s.dv + d];
+        }
+    } else {
+        const T* q = (const T*)c.q + ((long)row * s.H + (long)g * R) * s.dkp;
+        for (int i = tid; i < R * s.dkp; i += 256) q_sm[i] = to_f(q[i]);
+    }
+    for (int i = tid; i < R * s.dv; i += 256) o_sm[i] = 0.0f;
+    for (int i = tid; i < R; i += 256) { m_sm[i] = s.sink ? 0.0f : -INFINITY; l_sm[i] = 0.0f; }
+    __syncthreads();
+
+    const int lo = max(0, pos - s.window + 1);
+    const int p_lo = lo / PG, n_pg = pos / PG - p_lo + 1;
+    const int n_tiles = (n_pg + TILE_PAGES - 1) / TILE_PAGES;
+    const int t_beg = (int)((long)split * n_tiles / n_split), t_end = (int)((long)(split + 1) * n_tiles / n_split);
+    const float* bias_g = c.bias + (long)g * (2 * kBiasPad + s.window) * R;
+    const float inv_cap = s.softcap > 0.0f ? s.scale / s.softcap : 0.0f;
+    const int kpw = 32 / L, sub = lane / L, ln = lane % L;            // keys per warp step, this lane's key and part
+    for (int t = t_beg; t < t_end; t++) {
+        const int pg0 = p_lo + t * TILE_PAGES, npg = min(TILE_PAGES, n_pg - t * TILE_PAGES);
+        // ---- scores of the tile's keys
+        for (int r0 = 0; r0 < R; r0 += RC) {
+            float qr[RC][8];
+            if (!WIDE)
+#pragma unroll
+                for (int r = 0; r < RC; r++)
+#pragma unroll
+                    for (int e = 0; e < 8; e++) qr[r][e] = (r0 + r < R && ln * 8 < s.dkp) ? q_sm[(r0 + r) * s.dkp + ln * 8 + e] : 0.0f;
+#pragma unroll 2
+            for (int k = warp * kpw + sub; k < npg * PG; k += 8 * kpw) {
+                const T* kp = (const T*)c.k_pool + ((long)pt[pg0 + (k >> 6)] * s.G + g) * kh + (long)(k & (PG - 1)) * s.dkp;
+                float acc[RC];
+#pragma unroll
+                for (int r = 0; r < RC; r++) acc[r] = 0.0f;
+                if (WIDE) {
+                    for (int e0 = ln * 8; e0 < s.dkp; e0 += L * 8) {
+                        float kf[8];
+                        load8(kp + e0, kf);
+#pragma unroll
+                        for (int r = 0; r < RC; r++)
+                            if (r0 + r < R)
+#pragma unroll
+                                for (int e = 0; e < 8; e++) acc[r] = __fmaf_rn(q_sm[(r0 + r) * s.dkp + e0 + e], kf[e], acc[r]);
+                    }
+                } else if (ln * 8 < s.dkp) {
+                    float kf[8];
+                    load8(kp + ln * 8, kf);
+#pragma unroll
+                    for (int r = 0; r < RC; r++)
+#pragma unroll
+                        for (int e = 0; e < 8; e++) acc[r] = __fmaf_rn(qr[r][e], kf[e], acc[r]);
+                }
+                // the loop bound is the same for all lanes of a warp step: npg * 64 is a multiple of 8 * kpw
+                for (int off = L >> 1; off > 0; off >>= 1)
+#pragma unroll
+                    for (int r = 0; r < RC; r++) acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], off);
+                const int d = pos - (pg0 * PG + k);
+#pragma unroll
+                for (int r = 0; r < RC; r++)
+                    if (r0 + r < R && ln == (r & (L - 1))) {
+                        float v = -INFINITY;
+                        if (d >= 0 && d < s.window) {
+                            if (s.softcap > 0.0f) {
+                                const float z = acc[r] * inv_cap;
+                                v = s.softcap * (FAST ? 1.0f - 2.0f * rcp_fast(1.0f + ex2_fast(z * (2.0f * kLog2e))) : tanhf(z));
+                            } else {
+                                v = acc[r] * s.scale;
+                            }
+                            v += bias_g[(long)(d + kBiasPad) * R + r0 + r];
+                        }
+                        s_sm[(r0 + r) * TILE_KEYS + k] = v;
+                    }
+            }
+        }
+        __syncthreads();
+        // ---- running maximum, weights, sums: one warp per head
+        for (int r = warp; r < R; r += 8) {
+            float* sr = s_sm + r * TILE_KEYS;
+            float mx = -INFINITY;
+            for (int k = lane; k < npg * PG; k += 32) mx = fmaxf(mx, sr[k]);
+            mx = warp_max(mx);
+            const float m_old = m_sm[r], m_new = fmaxf(m_old, mx);
+            const float ref = m_new == -INFINITY ? 0.0f : m_new;
+            float sum = 0.0f;
+            for (int k = lane; k < npg * PG; k += 32) {
+                const float p = FAST ? ex2_fast((sr[k] - ref) * kLog2e) : expf(sr[k] - ref);
+                sr[k] = p;
+                sum += p;
+            }
+            sum = warp_sum(sum);
+            __syncwarp();
+            if (lane == 0) {
+                const float al = m_old == -INFINITY ? 0.0f : expf(m_old - ref);
+                al_sm[r] = al; m_sm[r] = m_new; l_sm[r] = __fmaf_rn(l_sm[r], al, sum);
+            }
+        }
+        __syncthreads();
+        // ---- values: 8 lanes share one row (dimension) of a V^T page, 8 tokens each
+        const int dl = lane >> 3, tv = lane & 7;
+        for (int r0 = 0; r0 < R; r0 += RC) {
+            for (int db = warp * 4; db < s.dv; db += 32) {
+                const int d = db + dl;
+                float acc[RC];
+#pragma unroll
+                for (int r = 0; r < RC; r++) acc[r] = 0.0f;
+                if (d < s.dv) {
+#pragma unroll 4
+                    for (int p = 0; p < npg; p++) {
+                        float vf[8];
+                        load8((const T*)c.v_pool + ((long)pt[pg0 + p] * s.G + g) * vh + (long)d * PG + tv * 8, vf);
+#pragma unroll
+                        for (int r = 0; r < RC; r++) {
+                            if (r0 + r >= R) continue;
+                            const float* pr = s_sm + (r0 + r) * TILE_KEYS + p * PG + tv * 8;
+                            const float4 x = load4(pr), y = load4(pr + 4);
+                            float t8 = acc[r];
+                            t8 = __fmaf_rn(x.x, vf[0], t8); t8 = __fmaf_rn(x.y, vf[1], t8); t8 = __fmaf_rn(x.z, vf[2], t8); t8 = __fmaf_rn(x.w, vf[3], t8);
+                            t8 = __fmaf_rn(y.x, vf[4], t8); t8 = __fmaf_rn(y.y, vf[5], t8); t8 = __fmaf_rn(y.z, vf[6], t8); t8 = __fmaf_rn(y.w, vf[7], t8);
+                            acc[r] = t8;
+                        }
+                    }
+                }
+#pragma unroll
+                for (int off = 4; off > 0; off >>= 1)
+#pragma unroll
+                    for (int r = 0; r < RC; r++) acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], off);
+                if (tv == 0 && d < s.dv)
+#pragma unroll
+                    for (int r = 0; r < RC; r++)
+                        if (r0 + r < R) { float* op = o_sm + (r0 + r) * s.dv + d; *op = __fmaf_rn(*op, al_sm[r0 + r], acc[r]); }
+            }
+        }
+        __syncthreads();
+    }
+
+    if (n_split > 1) {
+        // partial (maximum, sum, values) per head; the last CTA of this (row, head) combines them in split order
+        const long stride = (long)R * (s.dv + 2);
+        float* part = c.ws + ((long)row * s.G + g) * n_split * stride;
+        float* mine = part + split * stride;
+        for (int i = tid; i < R; i += 256) { mine[i] = m_sm[i]; mine[R + i] = l_sm[i]; }
+        for (int i = tid; i < R * s.dv; i += 256) mine[2 * R + i] = o_sm[i];
+        __threadfence();
+        __syncthreads();
+        int* cnt = c.counters + (long)row * s.G + g;
+        if (tid == 0) last_sm = atomicAdd(cnt, 1) == n_split - 1;
+        __syncthreads();
+        if (!last_sm) return;
+        __threadfence();
+        for (int r = tid; r < R; r += 256) {
+            float m = s.sink ? 0.0f : -INFINITY;
+            for (int k = 0; k < n_split; k++) m = fmaxf(m, __ldcg(part + k * stride + r));
+            float l = 0.0f;
+            for (int k = 0; k < n_split; k++) {
+                const float mk = __ldcg(part + k * stride + r);
+                const float w = mk == -INFINITY ? 0.0f : expf(mk - m);
+                l = __fmaf_rn(__ldcg(part + k * stride + R + r), w, l);
+            }
+            m_sm[r] = m; l_sm[r] = l;
+        }
+        __syncthreads();
+        for (int i = tid; i < R * s.dv; i += 256) {
+            const int r = i / s.dv;
+            float v = 0.0f;
+            for (int k = 0; k < n_split; k++) {
+                const float mk = __ldcg(part + k * stride + r);
+                const float w = mk == -INFINITY ? 0.0f : expf(mk - m_sm[r]);
+                v = __fmaf_rn(__ldcg(part + k * stride + 2 * R + i), w, v);
+            }
+            o_sm[i] = v;
+        }
+        if (tid == 0) *cnt = 0;
+        __syncthreads();
+    }
+    T* out = (T*)c.out + (long)row * c.ldo + (long)g * R * s.dv;
+    for (int i = tid; i < R * s.dv; i += 256) {
+        const int r = i / s.dv;
+        const float den = l_sm[r] + (s.sink ? expf(-m_sm[r]) : 0.0f);
+        float v = o_sm[i] / den;
+        if (s.g_off >= 0) v *= sigmoid_f<FAST>(to_f(prow[s.g_off + (long)g * R * s.dv + i]));
+        out[i] = from_f<T>(v);
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------------
+// Prompt attention on the tensor cores. A CTA takes TQ = 128 / R consecutive positions x the R query heads of one key/value
+// head (row = position * R + head: the heads of a group share the K and V tiles, and a small window wastes few keys), and
+// walks the key pages its window reaches. The scores are bounded by softcap + max|bias|, so the softmax shift is a constant
+// (`shift2`) and the values accumulate in TMEM over all pages without rescaling.
+//   warps 0..3  softmax: one row per thread        warp 4  TMA: Q, then K and V pages        warp 5  MMA issue, TMEM
+struct PrefillArgs {
+    AttnCall c;
+    int R, TQ, n_qt;                  // heads per group, positions per CTA, CTAs per (sequence, group)
+    int kc, vrows;                    // 128-byte blocks of a Q/K row; rows of a V^T tile (dv rounded up to 16)
+    float a2, b2, shift2;             // tanh argument factor and -2 softcap in log2 units; softmax shift
+    int tmem_cols, o_col, p_bufs;
+    int* error_flag;
+};
+constexpr int PF_S_COLS = 64;
+
+struct PrefillSmem { uint32_t k, v, p, bias, bars, total; };
+__host__ __device__ inline PrefillSmem prefill_smem(int kc, int vrows, int R, int TQ, int p_bufs) {
+    PrefillSmem o;
+    o.k = (uint32_t)kc * 16384u;                                   // Q first
+    o.v = o.k + 2u * (uint32_t)kc * 8192u;
+    o.p = o.v + 2u * (((uint32_t)vrows * 128u + 1023u) & ~1023u);
+    o.bias = o.p + (uint32_t)p_bufs * 16384u;
+    const uint32_t bias_floats = (uint32_t)((TQ + 63) * R + 128);
+    o.bars = o.bias + 2u * ((bias_floats * 4u + 15u) & ~15u);
+    o.total = o.bars + 256u + 1024u;
+    return o;
+}
+
+__global__ void __launch_bounds__(192, 2) attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmapQ,
+                                                                  const __grid_constant__ CUtensorMap tmapK,
+                                                                  const __grid_constant__ CUtensorMap tmapV,
+                                                                  const __grid_constant__ PrefillArgs a) {
+    extern __shared__ uint8_t smem_raw[];
+    const uint32_t raw = smem_u32(smem_raw);
+    const uint32_t base = (raw + 1023u) & ~1023u;
+    uint8_t* base_ptr = smem_raw + (base - raw);
+    const AttnShape& s = a.c.s;
+    const int R = a.R, TQ = a.TQ;
+    const PrefillSmem o = prefill_smem(a.kc, a.vrows, R, TQ, a.p_bufs);
+    const uint32_t k_bytes = (uint32_t)a.kc * 8192u, v_bytes = (uint32_t)a.vrows * 128u, v_stride = (v_bytes + 1023u) & ~1023u;
+    uint64_t* bars = reinterpret_cast<uint64_t*>(base_ptr + o.bars);
+    const uint32_t bar_q = smem_u32(bars);
+    const uint32_t bar_kf = bar_q + 8, bar_ke = bar_kf + 16, bar_vf = bar_ke + 16, bar_ve = bar_vf + 16;
+    const uint32_t bar_sf = bar_ve + 16, bar_se = bar_sf + 16, bar_pf = bar_se + 16, bar_pe = bar_pf + 16, bar_o = bar_pe + 16;
+    uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 20);
+    volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+
+    if (threadIdx.x == 0) {
+        mbar_init(bar_q, 1); mbar_init(bar_o, 1);
+        for (int i = 0; i < 2; i++) {
+            mbar_init(bar_kf + 8 * i, 1); mbar_init(bar_ke + 8 * i, 1); mbar_init(bar_vf + 8 * i, 1); mbar_init(bar_ve + 8 * i, 1);
+            mbar_init(bar_sf + 8 * i, 1); mbar_init(bar_se + 8 * i, 4); mbar_init(bar_pf + 8 * i, 4); mbar_init(bar_pe + 8 * i, 1);
+        }
+        *abort_flag = 0;
+        fence_barrier_init();
+    }
+    if (warp == 5) { tmem_alloc(smem_u32(tmem_slot), a.tmem_cols); tmem_relinquish(); }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem_base = *tmem_slot;
+    pdl_sync();
+
+    // the longest-running tiles (late positions) first
+    const int qt = a.n_qt - 1 - (int)blockIdx.x, g = blockIdx.y, b = blockIdx.z;
+    const int p0 = start_pos(a.c, b, a.error_flag);
+    const int q0 = p0 + qt * TQ;                                         // first position of the tile
+    const int q1 = min(p0 + a.c.Sc, q0 + TQ) - 1;                        // last one
+    const int pg_lo = max(0, q0 - s.window + 1) / PG, pg_hi = q1 / PG;
+    const int n_kt = pg_hi - pg_lo + 1;
+    const int32_t* pt = a.c.page_table + (long)b * a.c.max_pages + pg_lo;
+
+    if (warp == 4) {
+        if (lane == 0) {
+            tma_prefetch_desc(&tmapQ); tma_prefetch_desc(&tmapK); tma_prefetch_desc(&tmapV);
+            mbar_expect_tx(bar_q, (uint32_t)a.kc * (uint32_t)(TQ * R) * 128u);
+            for (int i = 0; i < a.kc; i++) tma_load_3d(base + i * 16384u, &tmapQ, bar_q, i * 128, g * R, b * a.c.Sc + qt * TQ);
+            bool ok = true;
+            for (int j = 0; ok && j < n_kt; j++) {
+                const int sb = j & 1;
+                const uint32_t ph = (uint32_t)((j >> 1) & 1) ^ 1u;
+                const int page = __ldg(pt + j);
+                if (!mbar_wait(bar_ke + 8 * sb, ph, abort_flag)) break;
+                mbar_expect_tx(bar_kf + 8 * sb, k_bytes);
+                for (int i = 0; i < a.kc; i++)
+                    tma_load_2d(base + o.k + sb * k_bytes + i * 8192u, &tmapK, bar_kf + 8 * sb, i * 128, (page * s.G + g) * PG);
+                if (!mbar_wait(bar_ve + 8 * sb, ph, abort_flag)) { ok = false; break; }
+                mbar_expect_tx(bar_vf + 8 * sb, v_bytes);
+                tma_load_2d(base + o.v + sb * v_stride, &tmapV, bar_vf + 8 * sb, 0, (page * s.G + g) * s.dv);
+            }
+        }
+    } else if (warp == 5) {
+        if (lane == 0) {
+            const uint32_t idesc_qk = umma_idesc_bf16(128, PF_S_COLS), idesc_pv = umma_idesc_bf16(128, a.vrows);
+            const int ksteps = (s.dkp + 15) / 16;
+            bool ok = mbar_wait(bar_q, 0, abort_flag);
+            auto issue_qk = [&](int j) {
+                const int sb = j & 1;
+                const uint32_t ph = (uint32_t)((j >> 1) & 1);
+                if (!mbar_wait(bar_kf + 8 * sb, ph, abort_flag)) return false;
+                if (!mbar_wait(bar_se + 8 * sb, ph ^ 1u, abort_flag)) return false;
+                tc_fence_after();
+                for (int k = 0; k < ksteps; k++) {
+                    const uint32_t blk = k >> 2, off = 2 * (k & 3);
+                    umma_bf16(tmem_base + sb * PF_S_COLS, umma_desc_k_sw128(base + blk * 16384u) + off,
+                              umma_desc_k_sw128(base + o.k + sb * k_bytes + blk * 8192u) + off, idesc_qk, k > 0 ? 1u : 0u);
+                }
+                umma_commit(bar_sf + 8 * sb);
+                umma_commit(bar_ke + 8 * sb);
+                return true;
+            };
+            if (ok) ok = issue_qk(0);
+            for (int j = 0; ok && j < n_kt; j++) {
+                if (j + 1 < n_kt && !issue_qk(j + 1)) { ok = false; break; }
+                const int sb = j & 1, pb = a.p_bufs == 2 ? sb : 0;
+                if (!mbar_wait(bar_vf + 8 * sb, (uint32_t)((j >> 1) & 1), abort_flag)) { ok = false; break; }
+                if (!mbar_wait(bar_pf + 8 * pb, (uint32_t)((a.p_bufs == 2 ? j >> 1 : j) & 1), abort_flag)) { ok = false; break; }
+                tc_fence_after();
+                const uint64_t pd = umma_desc_k_sw128(base + o.p + pb * 16384u), vd = umma_desc_k_sw128(base + o.v + sb * v_stride);
+                for (int k = 0; k < 4; k++)
+                    umma_bf16(tmem_base + a.o_col, pd + 2 * k, vd + 2 * k, idesc_pv, (j > 0 || k > 0) ? 1u : 0u);
+                umma_commit(bar_pe + 8 * pb);
+                umma_commit(bar_ve + 8 * sb);
+            }
+            if (ok) umma_commit(bar_o);
+        }
+    } else {
+        const int rr = warp * 32 + lane;                       // row: position rr / R of the tile, head rr % R of the group
+        const uint32_t lane_addr = (uint32_t)(warp * 32) << 16;
+        const int n_bias = (TQ + 63) * R;
+        float* bias_sm = reinterpret_cast<float*>(base_ptr + o.bias);
+        const int bias_stride = (n_bias + 128 + 3) & ~3;
+        const float* bias_g = a.c.bias + (long)g * (2 * kBiasPad + s.window) * R;
+        auto wait_bar = [&](uint32_t bar, uint32_t parity) {
+            int got = (lane == 0) ? (mbar_wait(bar, parity, abort_flag) ? 1 : 0) : 1;
+            return __shfl_sync(0xffffffffu, got, 0) != 0;
+        };
+        // biases of key tile j, in log2 units with the constants of the score formula folded in; masked keys stay -inf.
+        // Entry (t + 63 - key) * R + r belongs to position t, head r: consecutive rows read consecutive words.
+        const float badd = s.softcap * kLog2e - a.shift2;
+        auto stage_bias = [&](int j) {
+            const int dmin = q0 - (pg_lo + j) * PG - 63;                 // distance of the first entry
+            const float* src = bias_g + (long)(dmin + kBiasPad) * R;
+            float* dst = bias_sm + (j & 1) * bias_stride;
+            for (int i = rr; i < n_bias; i += 128) dst[i] = __fmaf_rn(src[i], kLog2e, badd);
+        };
+        stage_bias(0);
+        float l = 0.0f;
+        bool ok = true;
+        for (int j = 0; j < n_kt; j++) {
+            const int sb = j & 1, pb = a.p_bufs == 2 ? sb : 0;
+            named_sync<1, 128>();                                        // tile j's biases are in place; j - 1's reads are over
+            if (j + 1 < n_kt) stage_bias(j + 1);
+            const float* bs = bias_sm + sb * bias_stride + rr + 63 * R;
+            if (ok && !wait_bar(bar_sf + 8 * sb, (uint32_t)((j >> 1) & 1))) ok = false;
+            if (ok && !wait_bar(bar_pe + 8 * pb, (uint32_t)((a.p_bufs == 2 ? j >> 1 : j) & 1) ^ 1u)) ok = false;
+            if (!ok) continue;                                           // keep meeting the others at the barrier
+            tc_fence_after();
+            uint8_t* prow = base_ptr + o.p + pb * 16384 + rr * 128;
+            const uint32_t tS = tmem_base + sb * PF_S_COLS + lane_addr;
+#pragma unroll
+            for (int cc = 0; cc < 4; cc++) {
+                uint32_t v[16];
+                tmem_ld_32x16(tS + cc * 16, v);
+                tmem_ld_wait();
+                uint32_t pk[8];
+#pragma unroll
+                for (int i = 0; i < 16; i += 2) {
+                    float p[2];
+#pragma unroll
+                    for (int u = 0; u < 2; u++) {
+                        const float bi = bs[-(cc * 16 + i + u) * R];
+                        const float x = __uint_as_float(v[i + u]) * a.a2;
+                        // softcap * tanh(z) = softcap - 2 softcap / (1 + e^(2 z)); all in log2 units
+                        const float s2 = __fmaf_rn(a.b2, rcp_fast(1.0f + ex2_fast(x)), bi);
+                        p[u] = ex2_fast(s2);
+                    }
+                    l += p[0] + p[1];
+                    pk[i >> 1] = bf_pack(p[0], p[1]);
+                }
+                *reinterpret_cast<uint4*>(prow + (((2 * cc) ^ (rr & 7)) << 4)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+                *reinterpret_cast<uint4*>(prow + (((2 * cc + 1) ^ (rr & 7)) << 4)) = make_uint4(pk[4], pk[5], pk[6], pk[7]);
+            }
+            fence_proxy_async_smem();
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) { mbar_arrive(bar_pf + 8 * pb); mbar_arrive(bar_se + 8 * sb); }
+        }
+        if (ok) ok = wait_bar(bar_o, 0);
+        if (ok) {
+            tc_fence_after();
+            const int t = rr / R, r = rr - t * R;
+            const bool row_ok = rr < TQ * R && q0 + t <= q1;
+            const float rl = 1.0f / (l + (s.sink ? ex2_fast(-a.shift2) : 0.0f));
+            const long m = (long)b * a.c.Sc + qt * TQ + t;
+            const long hcol = (long)(g * R + r) * s.dv;
+            bf16* out = (bf16*)a.c.out + m * a.c.ldo + hcol;
+            const bf16* gate = s.g_off >= 0 ? (const bf16*)a.c.proj + m * s.ld + s.g_off + hcol : nullptr;
+            const bool vec = (s.dv & 7) == 0 && (a.c.ldo & 7) == 0;       // proj offsets and rows are multiples of 8
+            for (int d0 = 0; d0 < a.vrows; d0 += 16) {
+                uint32_t v[16];
+                tmem_ld_32x16(tmem_base + a.o_col + d0 + lane_addr, v);
+                tmem_ld_wait();
+                if (!row_ok) continue;
+#pragma unroll
+                for (int h = 0; h < 2; h++) {
+                    const int d = d0 + 8 * h;
+                    if (d >= s.dv) continue;
+                    float f[8], gf[8];
+                    if (vec) {
+                        if (gate) load8(gate + d, gf);
+#pragma unroll
+                        for (int e = 0; e < 8; e++) { f[e] = __uint_as_float(v[8 * h + e]) * rl; if (gate) f[e] *= sigmoid_f<true>(gf[e]); }
+                        *reinterpret_cast<uint4*>(out + d) = make_uint4(bf_pack(f[0], f[1]), bf_pack(f[2], f[3]), bf_pack(f[4], f[5]), bf_pack(f[6], f[7]));
+                    } else {
+#pragma unroll
+                        for (int e = 0; e < 8; e++)
+                            if (d + e < s.dv) {
+                                float x = __uint_as_float(v[8 * h + e]) * rl;
+                                if (gate) x *= sigmoid_f<true>(to_f(gate[d + e]));
+                                out[d + e] = __float2bfloat16_rn(x);
+                            }
+                    }
+                }
+            }
+        }
+    }
+
+    tc_fence_before();
+    __syncthreads();
+    if (*abort_flag) {
+        const unsigned long long t0 = globaltimer_ns();
+        while (globaltimer_ns() - t0 < 200000ull) { __nanosleep(1000); }
+        if (threadIdx.x == 0 && a.error_flag) atomicOr(a.error_flag, 1);
+        __syncthreads();
+    }
+    if (warp == 5) { tc_fence_after(); tmem_dealloc(tmem_base, a.tmem_cols); }
+}
+
+int set_smem(const void* kern, size_t bytes) {
+    return bytes > 48 * 1024 ? cuda_status(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes)) : FLEXLLM_OK;
+}
+
+template <class T, int RC, bool FUSED, bool WIDE> int launch_row(const AttnCall& c, int splits, int L, cudaStream_t st) {
+    const int R = c.s.H / c.s.G;
+    const size_t smem = (size_t)row_smem(R, c.s.dkp, c.s.dv).total * 4;
+    if (smem > 220 * 1024) return FLEXLLM_ENOTSUP;
+    auto kern = attn_row_kernel<T, RC, FUSED, WIDE>;
+    TRY_RC(set_smem((const void*)kern, smem));
+    launch_k(kern, dim3(splits, c.s.G, c.B * c.Sc), dim3(256), smem, st, c, L, device_error_flag());
+    return launch_status();
+}
+
+template <class T, bool FUSED> int run_row(const AttnCall& c, cudaStream_t st) {
+    const AttnShape& s = c.s;
+    const int R = s.H / s.G;
+    const long ctas = (long)c.B * c.Sc * s.G;
+    if (ctas / s.G > 65535) return FLEXLLM_ENOTSUP;
+    const int reach = s.window < c.max_pos + 1 ? s.window : c.max_pos + 1;
+    const int tiles = (reach + 2 * PG - 2) / PG / TILE_PAGES + 1;
+    long splits = 1;
+    if (FUSED && c.ws) {
+        splits = 2L * gemm_sm_count() / ctas;
+        if (splits > tiles) splits = tiles;
+        const long per = ctas * R * (s.dv + 2);
+        if (splits * per > (long)c.ws_floats) splits = (long)c.ws_floats / per;
+        if (splits < 1 || ctas > c.n_counters) splits = 1;
+    }
+    const int vecs = s.dkp / 8;
+    const int L = vecs <= 8 ? 8 : vecs <= 16 ? 16 : 32;
+#define FLEXLLM_ROW(RC_) return vecs > 32 ? launch_row<T, RC_, FUSED, true>(c, (int)splits, L, st) : launch_row<T, RC_, FUSED, false>(c, (int)splits, L, st)
+    if (R == 1) FLEXLLM_ROW(1);
+    if (R == 2) FLEXLLM_ROW(2);
+    FLEXLLM_ROW(4);
+#undef FLEXLLM_ROW
+}
+
+// Whether the tensor-core kernel covers the call (bf16 only).
+bool prefill_covers(const AttnCall& c, PrefillArgs* a) {
+    const AttnShape& s = c.s;
+    a->c = c;
+    a->R = s.H / s.G; a->TQ = a->R <= 16 ? 128 / a->R : 0;
+    if (a->R > 16 || s.dkp > 256 || s.dv > 256) return false;
+    if (s.softcap <= 0.0f) return false;                                  // no bound on the scores: running maximum needed
+    const float bound2 = (s.softcap + c.bias_max_abs) * kLog2e;
+    a->shift2 = bound2 > 100.0f ? bound2 - 100.0f : 0.0f;
+    if (a->shift2 > (s.sink ? 80.0f : 20.0f)) return false;               // sums could vanish below the smallest floats
+    a->kc = (s.dkp + 63) / 64; a->vrows = (s.dv + 15) / 16 * 16;
+    a->n_qt = (c.Sc + a->TQ - 1) / a->TQ;
+    a->a2 = s.scale / s.softcap * 2.0f * kLog2e; a->b2 = -2.0f * s.softcap * kLog2e;
+    a->o_col = 2 * PF_S_COLS;
+    int cols = 32;
+    while (cols < a->o_col + a->vrows) cols *= 2;
+    a->tmem_cols = cols;
+    // two CTAs per SM where one P buffer makes that possible
+    a->p_bufs = prefill_smem(a->kc, a->vrows, a->R, a->TQ, 2).total <= 113 * 1024 ? 2
+              : prefill_smem(a->kc, a->vrows, a->R, a->TQ, 1).total <= 113 * 1024 ? 1 : 2;
+    if (prefill_smem(a->kc, a->vrows, a->R, a->TQ, a->p_bufs).total > 227 * 1024) a->p_bufs = 1;
+    a->error_flag = device_error_flag();
+    return prefill_smem(a->kc, a->vrows, a->R, a->TQ, a->p_bufs).total <= 227 * 1024;
+}
+
+int run_prefill(const PrefillArgs& a, cudaStream_t st) {
+    const AttnCall& c = a.c;
+    const AttnShape& s = c.s;
+    CUtensorMap tq, tk, tv;
+    TRY_RC(make_tmap_rows3_u8(&tq, c.q, (uint64_t)c.B * c.Sc, (uint64_t)s.H, (uint64_t)s.dkp * 2, (uint32_t)a.TQ, (uint32_t)a.R));
+    TRY_RC(cached_tmap_u8(&tk, c.k_pool, (uint64_t)c.n_pages * s.G * PG, (uint64_t)s.dkp * 2, PG, 0));
+    TRY_RC(cached_tmap_u8(&tv, c.v_pool, (uint64_t)c.n_pages * s.G * s.dv, PG * 2, (uint32_t)a.vrows, 0));
+    const size_t smem = prefill_smem(a.kc, a.vrows, a.R, a.TQ, a.p_bufs).total;
+    auto kern = attn_window_prefill_kernel;
+    TRY_RC(set_smem((const void*)kern, smem));
+    launch_k(kern, dim3(a.n_qt, s.G, c.B), dim3(192), smem, st, tq, tk, tv, a);
+    return launch_status();
+}
+
+template <class T> bool run_tensor_prefill(const AttnCall&, cudaStream_t, int*) { return false; }
+template <> bool run_tensor_prefill<bf16>(const AttnCall& c, cudaStream_t st, int* rc) {
+    PrefillArgs a;
+    if (!prefill_covers(c, &a)) return false;
+    *rc = run_prefill(a, st);
+    return true;
+}
+
+int check_call(const AttnCall& c) {
+    const AttnShape& s = c.s;
+    FLEXLLM_REQUIRE(c.proj && c.q_gain && c.k_gain && c.bias && c.k_pool && c.v_pool && c.page_table && c.ctx && c.out);
+    FLEXLLM_REQUIRE(s.H > 0 && s.G > 0 && s.H % s.G == 0 && s.dk > 0 && s.dv > 0 && s.window > 0 && s.dkp % 8 == 0 && s.dkp >= s.dk);
+    FLEXLLM_REQUIRE(s.ld % 8 == 0 && s.q_off % 8 == 0 && s.k_off % 8 == 0 && s.v_off % 8 == 0 && (s.g_off < 0 || s.g_off % 8 == 0));
+    FLEXLLM_REQUIRE(c.B > 0 && c.Sc > 0 && c.max_pos >= c.Sc - 1 && c.max_pos < c.max_pages * PG && c.n_pages > 0);
+    return FLEXLLM_OK;
+}
+
+}  // namespace
+
+size_t attn_window_ws_floats(int max_batch, int G, int R, int dv) {
+    // splits * CTAs never exceeds twice the SM count plus one CTA row
+    const size_t ctas = (size_t)max_batch * G;
+    const size_t n = 2u * 160u > ctas ? 2u * 160u : ctas;
+    return n * (size_t)R * (dv + 2);
+}
+
+template <class T> int attn_window(const AttnCall& c, cudaStream_t st) {
+    TRY_RC(check_call(c));
+    if (c.Sc == 1) return run_row<T, true>(c, st);
+    FLEXLLM_REQUIRE(c.q);
+    const int v_pages = (c.Sc + PG - 2) / PG + 1;
+    launch_k(attn_prepare_kernel<T>, dim3(c.B * c.Sc + c.B * c.s.G * v_pages), dim3(256), 0, st, c, v_pages, device_error_flag());
+    TRY_RC(launch_status());
+    int rc = FLEXLLM_OK;
+    if (run_tensor_prefill<T>(c, st, &rc)) return rc;
+    return run_row<T, false>(c, st);
+}
+template int attn_window<float>(const AttnCall&, cudaStream_t);
+template int attn_window<bf16>(const AttnCall&, cudaStream_t);
+
+}  // namespace flexllm

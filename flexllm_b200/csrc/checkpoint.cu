@@ -10,6 +10,7 @@
 //                                sum_k w[n][k] * s[n] of the asymmetric dequantiser), RMSNorm_weight[2*layers+1][hidden]
 //                                in w_rmsnorm.h, A_s[layers][heads_q] in A_s.h, PE_sin / PE_cos[pos][32] in
 //                                RoPE_sin_cos.h, w_lm_head_lm_head_s[vocab] / _sum[vocab] in w_lm_head_lm_head.h
+// Models of the decoder family come as one .safetensors file instead (flexllm_model_load_safetensors).
 // The demo re-packs the .bin rows two 4-bit channels per byte into its FPGA lane layout while reading; here rows are
 // kept as int8 [out][in], the layout every linear layer of this library takes.
 #include <cctype>
@@ -19,9 +20,81 @@
 #include <string>
 #include <vector>
 
+#include <fcntl.h>
+#include <sys/mman.h>
+#include <sys/stat.h>
+#include <unistd.h>
+
 #include "common.cuh"
+#include "model.h"
 
 namespace flexllm {
+
+// ---- .safetensors: u64 little-endian header length, a JSON object name -> {dtype, shape, data_offsets}, then the data ----
+struct StTensor { std::string name, dtype; std::vector<int64_t> shape; uint64_t begin = 0, end = 0; };
+
+// Just enough JSON for that header (strings, integers, arrays, one level of nested objects; "__metadata__" is skipped).
+struct StParser {
+    const char *p, *e;
+    bool ok = true;
+    void ws() { while (p < e && isspace((unsigned char)*p)) p++; }
+    bool eat(char c) { ws(); if (p < e && *p == c) { p++; return true; } return false; }
+    std::string str() {
+        std::string s;
+        if (!eat('"')) { ok = false; return s; }
+        while (p < e && *p != '"') {
+            if (*p == '\\' && p + 1 < e) p++;
+            s += *p++;
+        }
+        if (p < e) p++; else ok = false;
+        return s;
+    }
+    int64_t num() {
+        ws();
+        char* q = nullptr;
+        std::string t(p, (size_t)(e - p) < 24 ? (size_t)(e - p) : 24);
+        const long long v = strtoll(t.c_str(), &q, 10);
+        if (q == t.c_str()) ok = false;
+        p += q - t.c_str();
+        return v;
+    }
+    std::vector<int64_t> nums() {
+        std::vector<int64_t> v;
+        if (!eat('[')) { ok = false; return v; }
+        if (eat(']')) return v;
+        do v.push_back(num()); while (ok && eat(','));
+        if (!eat(']')) ok = false;
+        return v;
+    }
+    void skip_object() {
+        if (!eat('{')) { ok = false; return; }
+        if (eat('}')) return;
+        do { str(); if (!eat(':')) ok = false; str(); } while (ok && eat(','));
+        if (!eat('}')) ok = false;
+    }
+    bool parse(std::vector<StTensor>* out) {
+        if (!eat('{')) return false;
+        if (eat('}')) return true;
+        do {
+            StTensor t;
+            t.name = str();
+            if (!eat(':')) return false;
+            if (t.name == "__metadata__") { skip_object(); continue; }
+            if (!eat('{')) return false;
+            do {
+                const std::string k = str();
+                if (!eat(':')) return false;
+                if (k == "dtype") t.dtype = str();
+                else if (k == "shape") t.shape = nums();
+                else if (k == "data_offsets") { const auto o = nums(); if (o.size() != 2 || o[0] < 0 || o[1] < o[0]) return false; t.begin = (uint64_t)o[0]; t.end = (uint64_t)o[1]; }
+                else return false;
+            } while (ok && eat(','));
+            if (!ok || !eat('}')) return false;
+            out->push_back(std::move(t));
+        } while (ok && eat(','));
+        return ok && eat('}');
+    }
+};
 
 static bool slurp(const std::string& path, std::string* out) {
     FILE* f = fopen(path.c_str(), "rb");
@@ -142,4 +215,41 @@ extern "C" int flexllm_ckpt_load_head(const char* dir, int layers, int hidden, i
     if (sin_t) TRY_RC(flexllm_ckpt_read_c_array_f32((d + "RoPE_sin_cos.h").c_str(), "PE_sin", 0, (long)table_len * 32, sin_t));
     if (embed) TRY_RC(flexllm_ckpt_read_bin((d + "model_embed_tokens_fp32.bin").c_str(), 0, (size_t)vocab * hidden * sizeof(float), embed));
     return FLEXLLM_OK;
+}
+
+extern "C" int flexllm_model_load_safetensors(flexllm_model* m, const char* path, void* stream) {
+    FLEXLLM_REQUIRE(m && m->fam && path);
+    const int fd = open(path, O_RDONLY);
+    if (fd < 0) return FLEXLLM_EIO;
+    struct stat sb;
+    void* map = MAP_FAILED;
+    if (fstat(fd, &sb) == 0 && sb.st_size > 8) map = mmap(nullptr, (size_t)sb.st_size, PROT_READ, MAP_PRIVATE, fd, 0);
+    close(fd);
+    if (map == MAP_FAILED) return FLEXLLM_EIO;
+    const uint8_t* base = (const uint8_t*)map;
+    const uint64_t size = (uint64_t)sb.st_size;
+    auto run = [&]() -> int {
+        uint64_t n = 0;
+        for (int i = 7; i >= 0; i--) n = n << 8 | base[i];
+        if (n > size - 8) return FLEXLLM_EIO;
+        StParser ps{(const char*)base + 8, (const char*)base + 8 + n};
+        std::vector<StTensor> ts;
+        if (!ps.parse(&ts)) return FLEXLLM_EIO;
+        const uint8_t* data = base + 8 + n;
+        const uint64_t avail = size - 8 - n;
+        for (const StTensor& t : ts) {
+            if (!m->fam->knows(t.name.c_str())) continue;
+            const int es = t.dtype == "BF16" || t.dtype == "F16" ? 2 : 4;
+            uint64_t count = 1;
+            for (int64_t d : t.shape) { if (d < 0) return FLEXLLM_EIO; count *= (uint64_t)d; }
+            if (t.end > avail || t.end - t.begin != count * es) return FLEXLLM_EIO;
+            if (t.dtype != "BF16") return FLEXLLM_ENOTSUP;
+            TRY_RC(flexllm_model_load_tensor(m, t.name.c_str(), FLEXLLM_BF16, (int)t.shape.size(), t.shape.data(), data + t.begin, stream));
+        }
+        FLEXLLM_CHECK_CUDA(cudaStreamSynchronize((cudaStream_t)stream));      // the mapping goes away
+        return m->fam->check_loaded();
+    };
+    const int rc = run();
+    munmap(map, (size_t)sb.st_size);
+    return rc;
 }

@@ -83,6 +83,22 @@ int make_tmap_3d_u8(CUtensorMap* out, const void* base, uint64_t rows, uint64_t 
     return FLEXLLM_OK;
 }
 
+int make_tmap_rows3_u8(CUtensorMap* out, const void* base, uint64_t outer, uint64_t mid, uint64_t row_bytes, uint32_t box_outer,
+                       uint32_t box_mid) {
+    EncodeTiledFn fn = get_encode_fn();
+    if (!fn) return FLEXLLM_ECUDA;
+    if (!aligned(base, 16) || (row_bytes % 16) != 0 || box_outer == 0 || box_mid == 0 || box_outer > 256 || box_mid > 256) return FLEXLLM_EINVAL;
+    cuuint64_t dims[3] = {row_bytes, mid, outer};
+    cuuint64_t strides[2] = {row_bytes, row_bytes * mid};
+    cuuint32_t box[3] = {128, box_mid, box_outer};
+    cuuint32_t estr[3] = {1, 1, 1};
+    CUresult r = fn(out, CU_TENSOR_MAP_DATA_TYPE_UINT8, 3, const_cast<void*>(base), dims, strides, box, estr,
+                    CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                    CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    if (r != CUDA_SUCCESS) { g_last_cuda_error = (int)r; return FLEXLLM_ECUDA; }
+    return FLEXLLM_OK;
+}
+
 int make_tmap_2d_u8(CUtensorMap* out, const void* base, uint64_t rows, uint64_t row_bytes, uint32_t box_rows) {
     return make_tmap_2d_u8_box(out, base, rows, row_bytes, 128, box_rows, 128);
 }
@@ -490,6 +506,10 @@ static int cached_tmap(CUtensorMap* out, const void* base, uint64_t rows, uint64
     if (cache.size() > 4096) cache.clear();
     cache.emplace(key, *out);
     return FLEXLLM_OK;
+}
+
+int cached_tmap_u8(CUtensorMap* out, const void* base, uint64_t rows, uint64_t row_bytes, uint32_t box_rows, uint32_t kch) {
+    return cached_tmap(out, base, rows, row_bytes, box_rows, kch);
 }
 
 // One error word per device: bit 0 is raised by any kernel of the library whose bounded device-side wait ran

@@ -12,6 +12,9 @@
 // Prefill uses the prefill RMSNorm summation order and the tcgen05 GEMM / attention kernels; decode
 // uses the decode order, the weight-streaming linear layers and the paged attention, and is replayed
 // from a CUDA graph (the token feedback stays on the device, as in the reference's decode graph).
+//
+// The generation loop, token choice, page table and step calls below serve every model family (model.h); the operator
+// graph in this file is the Llama's.
 #include <cstdlib>
 #include <cstring>
 #include <new>
@@ -20,8 +23,7 @@
 #include "attention_decode.cuh"     // layout of the paged KV cache (for the hand-over between partitions)
 #include "common.cuh"
 #include "decode_mega.h"
-
-struct flexllm_tp;
+#include "model.h"
 
 namespace flexllm {
 int gemm_i8_prefill(const int8_t* a, const float* s_tok, const int8_t* w, const float* s_ch, int M, int N, int K,
@@ -100,66 +102,41 @@ __global__ void step_bookkeeping_kernel(const int32_t* __restrict__ next, int B,
 }
 __global__ void set_state_kernel(int32_t* state, int col, int n_cols) { state[0] = col; state[1] = n_cols; }
 
+__global__ void add_ctx_kernel(int32_t* ctx, int B, int v) { if (threadIdx.x < B) ctx[threadIdx.x] += v; }
+// rows[i] of x -> y[i]
+__global__ void gather_rows_kernel(const float* __restrict__ x, const int32_t* __restrict__ rows, int D, float* __restrict__ y) {
+    const float4* src = reinterpret_cast<const float4*>(x + (long)rows[blockIdx.x] * D);
+    float4* dst = reinterpret_cast<float4*>(y + (long)blockIdx.x * D);
+    for (int i = threadIdx.x; i < D / 4; i += blockDim.x) dst[i] = src[i];
+}
+
 __global__ void fill_ctx_kernel(int32_t* ctx, int B, int v) { if (threadIdx.x < B) ctx[threadIdx.x] = v; }
 
 }  // namespace flexllm
 
 using namespace flexllm;
 
-struct LayerW {
-    int8_t *wqkv, *wo, *wgu, *wd;
-    float *sqkv, *so, *sgu, *sd, *g0, *g1, *a_s;
-};
-
-struct flexllm_model {
-    flexllm_model_config cfg;
-    std::vector<LayerW> L;
-    int8_t* lm_w = nullptr; float* lm_s = nullptr; float* g_final = nullptr;
-    float *cos_t = nullptr, *sin_t = nullptr; int table_len = 0;
-    flexllm_kv_cache* cache = nullptr;
-    int max_pages = 0;
-    int32_t *page_table = nullptr, *ctx = nullptr, *next = nullptr, *state = nullptr, *tokens = nullptr, *out_tokens = nullptr;
-    size_t out_capacity = 0;
-    // activations (sized for max_batch * max_prefill rows)
-    float *x = nullptr, *qkv = nullptr, *att = nullptr, *tmp = nullptr, *gu = nullptr, *xs = nullptr, *logits = nullptr, *xlast = nullptr;
-    int8_t *xq = nullptr, *hq = nullptr;
-    void *attn_ws = nullptr, *dec_ws = nullptr;
-    size_t attn_ws_bytes = 0, dec_ws_bytes = 0;
-    // decode state
-    int B = 0, S = 0;
-    int last_chunk = 0;                         // rows per sequence the residual stream x holds after the last prefill
-    int n_new = 0;                              // columns of the token table of the running generation
-    int pos = 0;                                // context length of the batch = position the next decode step writes
-    cudaGraphExec_t graph = nullptr; int graph_B = 0; int graph_kernels = 0;
-    int mega_variant = 0, graph_variant = 0;   // attention variant of the persistent kernel for the current decode call / in the captured step
-    std::vector<void*> owned;
-    // tensor parallelism: g ranks, this one is r; *l = local (per-rank) sizes
-    flexllm_tp* tp = nullptr;
-    int g = 1, r = 0, HQl = 0, HKVl = 0, Fl = 0, Dl = 0, Vl = 0;
-    float *gath = nullptr, *hloc = nullptr;     // all-gather target / local silu(gate)*up slice
-    // token-row partition of the prefill + batch-parallel decode (see flexllm_model_prefill)
-    flexllm_model* dm = nullptr;                // single-GPU model of this rank's sequences: full weights, all KV heads
-    float *amax = nullptr, *xs2 = nullptr;      // per-token largest magnitudes / scales of the row-parallel inputs
-    int8_t* aq = nullptr;                       // quantised attention output, this rank's columns
-    uint8_t *kv_stage = nullptr, *kvs_stage = nullptr;   // KV hand-over: pages / scale rows as received
-    bool rows_mode = false;                     // the last prefill used the token-row partition
-    int32_t* acc32 = nullptr;                   // row-parallel partial sums
-    void *pairs_l = nullptr, *pairs_g = nullptr;
-    // persistent decode-step kernel: -1 not tried yet, 0 not usable for this model, 1 ready
-    flexllm::MegaPlan* mega = nullptr; int mega_state = -1;
-    // token choice: greedy (sample_k == 0) or the reference's top-k sampling with uniform numbers rnd [n_new][B]
-    int sample_lanes = 0, sample_k = 0; const float* sample_rnd = nullptr;
-};
-
-template <class T> static int dmalloc(flexllm_model* m, T** p, size_t n) {
-    void* q = nullptr;
-    cudaError_t e = cudaMalloc(&q, n * sizeof(T) + 256);
-    if (e != cudaSuccess) { g_last_cuda_error = (int)e; return e == cudaErrorMemoryAllocation ? FLEXLLM_ENOMEM : FLEXLLM_ECUDA; }
-    m->owned.push_back(q);
-    *p = (T*)q;
+// What every family's runner holds: page table, context lengths, token tables, row list, logits. Sequence b owns pages
+// [b * seq_pages, (b + 1) * seq_pages) and logical page i lies in the (i % seq_pages)-th of them: with seq_pages == max_pages
+// every position has its own slot; fewer make the pages of a sliding-window model a ring.
+static int runner_alloc(flexllm_model* m, int seq_pages) {
+    const flexllm_model_config& c = m->cfg;
+    TRY(dmalloc(m, &m->page_table, (size_t)c.max_batch * m->max_pages));
+    TRY(dmalloc(m, &m->ctx, 64));
+    TRY(dmalloc(m, &m->next, 64));
+    TRY(dmalloc(m, &m->state, 4));
+    TRY(dmalloc(m, &m->tokens, (size_t)c.max_batch * c.max_ctx));
+    m->out_capacity = (size_t)c.max_batch * (c.max_ctx + 1);
+    TRY(dmalloc(m, &m->out_tokens, m->out_capacity));
+    m->logits_rows = m->fam ? 64 : c.max_batch;
+    TRY(dmalloc(m, &m->rows, 64));
+    TRY(dmalloc(m, &m->logits, (size_t)m->logits_rows * c.vocab));
+    std::vector<int32_t> pt((size_t)c.max_batch * m->max_pages);
+    for (int b = 0; b < c.max_batch; b++)
+        for (int i = 0; i < m->max_pages; i++) pt[(size_t)b * m->max_pages + i] = b * seq_pages + i % seq_pages;
+    FLEXLLM_CHECK_CUDA(cudaMemcpy(m->page_table, pt.data(), pt.size() * 4, cudaMemcpyHostToDevice));
     return FLEXLLM_OK;
 }
-#define TRY(expr) do { int _rc = (expr); if (_rc != FLEXLLM_OK) return _rc; } while (0)
 
 extern "C" int flexllm_model_create(flexllm_model** out, const flexllm_model_config* c) {
     return flexllm_model_create_tp(out, c, nullptr);
@@ -205,20 +182,11 @@ extern "C" int flexllm_model_create_tp(flexllm_model** out, const flexllm_model_
     m->max_pages = (c->max_ctx + 64) / 64;
     const int n_pages = m->max_pages * c->max_batch;
     if ((rc = flexllm_kv_cache_create(&m->cache, NL, n_pages, HKV, 64))) return fail(rc);
-    if ((rc = dmalloc(m, &m->page_table, (size_t)c->max_batch * m->max_pages)) || (rc = dmalloc(m, &m->ctx, 64)) ||
-        (rc = dmalloc(m, &m->next, 64)) || (rc = dmalloc(m, &m->state, 4)) || (rc = dmalloc(m, &m->tokens, (size_t)c->max_batch * c->max_ctx)))
-        return fail(rc);
-    m->out_capacity = (size_t)c->max_batch * (c->max_ctx + 1);
-    if ((rc = dmalloc(m, &m->out_tokens, m->out_capacity))) return fail(rc);
-    {   // identity page table: sequence b owns pages [b*max_pages, (b+1)*max_pages)
-        std::vector<int32_t> pt((size_t)c->max_batch * m->max_pages);
-        for (size_t i = 0; i < pt.size(); i++) pt[i] = (int32_t)i;
-        if (cudaMemcpy(m->page_table, pt.data(), pt.size() * 4, cudaMemcpyHostToDevice) != cudaSuccess) return fail(FLEXLLM_ECUDA);
-    }
+    if ((rc = runner_alloc(m, m->max_pages))) return fail(rc);
     if ((rc = dmalloc(m, &m->x, Mmax * D)) || (rc = dmalloc(m, &m->qkv, Mmax * QKV)) || (rc = dmalloc(m, &m->att, Mmax * D)) ||
         (rc = dmalloc(m, &m->tmp, Mmax * D)) || (rc = dmalloc(m, &m->gu, Mmax * 2 * m->Fl)) || (rc = dmalloc(m, &m->xs, Mmax)) ||
         (rc = dmalloc(m, &m->xq, Mmax * D)) || (rc = dmalloc(m, &m->hq, Mmax * m->Fl)) ||
-        (rc = dmalloc(m, &m->logits, (size_t)c->max_batch * V)) || (rc = dmalloc(m, &m->xlast, (size_t)c->max_batch * D)))
+        (rc = dmalloc(m, &m->xlast, (size_t)c->max_batch * D)))
         return fail(rc);
     if (g > 1) {
         if ((rc = dmalloc(m, &m->gath, Mmax * F)) || (rc = dmalloc(m, &m->hloc, Mmax * m->Fl)) || (rc = dmalloc(m, &m->acc32, Mmax * D)))
@@ -249,6 +217,22 @@ extern "C" int flexllm_model_create_tp(flexllm_model** out, const flexllm_model_
     return FLEXLLM_OK;
 }
 
+// A runner around another family: `seq_pages` pages per sequence of a cache the family has created.
+int flexllm::runner_create(flexllm_model** out, const flexllm_model_config& cfg, ModelFamily* fam, flexllm_kv_cache* cache, int seq_pages,
+                           size_t x_floats) {
+    flexllm_model* m = new (std::nothrow) flexllm_model();
+    if (!m) { delete fam; flexllm_kv_cache_destroy(cache); return FLEXLLM_ENOMEM; }
+    m->cfg = cfg; m->fam = fam; m->cache = cache;
+    m->max_pages = (cfg.max_ctx + 64) / 64;
+    int rc = runner_alloc(m, seq_pages);
+    if (!rc) rc = dmalloc(m, &m->x, x_floats);
+    if (!rc) rc = cuda_status(cudaMemset(m->x, 0, x_floats * 4));
+    if (!rc) rc = flexllm_model_reset(m, nullptr);
+    if (rc) { flexllm_model_destroy(m); return rc; }
+    *out = m;
+    return FLEXLLM_OK;
+}
+
 extern "C" int flexllm_model_destroy(flexllm_model* m) {
     if (!m) return FLEXLLM_OK;
     if (m->graph) cudaGraphExecDestroy(m->graph);
@@ -256,6 +240,8 @@ extern "C" int flexllm_model_destroy(flexllm_model* m) {
     mega_destroy(m->mega);
     if (m->cache) flexllm_kv_cache_destroy(m->cache);
     for (void* p : m->owned) cudaFree(p);
+    if (m->own_rnd) cudaFree(m->own_rnd);
+    delete m->fam;
     delete m;
     return FLEXLLM_OK;
 }
@@ -272,7 +258,7 @@ static int copy_cols(void* dst, const void* src, size_t rows, size_t src_row_byt
 // Takes the FULL layer weights; with tensor parallelism each rank keeps its slice: rows of q/k/v and
 // gate/up (column-parallel, by heads / FFN channels), columns of o and down (row-parallel).
 extern "C" int flexllm_model_load_layer(flexllm_model* m, int layer, const flexllm_layer_weights* w, void* stream) {
-    FLEXLLM_REQUIRE(m && w && layer >= 0 && layer < m->cfg.layers);
+    FLEXLLM_REQUIRE(m && !m->fam && w && layer >= 0 && layer < m->cfg.layers);
     FLEXLLM_REQUIRE(w->wq && w->wk && w->wv && w->wo && w->wg && w->wu && w->wd && w->sq && w->sk && w->sv && w->so && w->sg &&
                     w->su && w->sd && w->gamma0 && w->gamma1 && w->a_s);
     cudaStream_t st = (cudaStream_t)stream;
@@ -304,7 +290,7 @@ extern "C" int flexllm_model_load_layer(flexllm_model* m, int layer, const flexl
 
 extern "C" int flexllm_model_load_head(flexllm_model* m, const int8_t* lm_w, const float* lm_s, const float* gamma_final,
                                        const float* cos_t, const float* sin_t, int table_len, void* stream) {
-    FLEXLLM_REQUIRE(m && lm_w && lm_s && gamma_final && cos_t && sin_t && table_len >= m->table_len);
+    FLEXLLM_REQUIRE(m && !m->fam && lm_w && lm_s && gamma_final && cos_t && sin_t && table_len >= m->table_len);
     cudaStream_t st = (cudaStream_t)stream;
     TRY(copy_any(m->lm_w, lm_w, (size_t)m->cfg.vocab * m->cfg.hidden, st));
     TRY(copy_any(m->lm_s, lm_s, (size_t)m->cfg.vocab * 4, st));
@@ -315,6 +301,13 @@ extern "C" int flexllm_model_load_head(flexllm_model* m, const int8_t* lm_w, con
     return FLEXLLM_OK;
 }
 
+// Token choice from m->logits [B][vocab] -> m->next (see run_head for col).
+static int choose_tokens(flexllm_model* m, int B, cudaStream_t st, const int32_t* col) {
+    const int V = m->cfg.vocab;
+    if (m->sample_k > 0) return topk_sample(m->logits, B, V, m->sample_lanes, m->sample_k, m->sample_rnd, col, m->next, nullptr, nullptr, st);
+    return flexllm_logits_argmax(m->logits, B, V, m->next, st);
+}
+
 // lm_head on the rows of xin [B][D] -> logits, argmax -> m->next
 // col: device pointer to the output column this head call fills (selects the row of sampling numbers), or
 // nullptr for column 0 (the prefill's token)
@@ -323,9 +316,7 @@ static int run_head(flexllm_model* m, const float* xin, int B, int order, cudaSt
     TRY(flexllm_rmsnorm_quant(xin, m->g_final, B, D, m->cfg.eps, order, nullptr, m->xq, m->xs, st));
     if (m->g == 1) {
         TRY(flexllm_linear_decode_i8(m->xq, m->xs, m->lm_w, m->lm_s, B, V, D, nullptr, m->logits, st));
-        if (m->sample_k > 0) TRY(topk_sample(m->logits, B, V, m->sample_lanes, m->sample_k, m->sample_rnd, col, m->next, nullptr, nullptr, st));
-        else TRY(flexllm_logits_argmax(m->logits, B, V, m->next, st));
-        return FLEXLLM_OK;
+        return choose_tokens(m, B, st, col);
     }
     if (m->sample_k > 0) return FLEXLLM_ENOTSUP;      // sampling needs the whole vocabulary on one GPU
     // vocab-parallel: this rank's rows of the (replicated) lm_head, local argmax, gather, select
@@ -516,8 +507,110 @@ static int prefill_any(flexllm_model* m, const int32_t* tokens, const float* emb
     return FLEXLLM_OK;
 }
 
+// ---- the step every family shares: the next tokens of the live sequences, from the cache that earlier steps left -------
+// Logits of the given rows (host indices into the rows of the last chunk) -> out [n][vocab] (host or device).
+static int rows_to_logits(flexllm_model* m, const int32_t* rows_host, int n, float* out, cudaStream_t st) {
+    const int D = m->cfg.hidden, V = m->cfg.vocab;
+    for (int i = 0; i < n; i += m->logits_rows) {
+        const int k = n - i < m->logits_rows ? n - i : m->logits_rows;
+        TRY(copy_any(m->rows, rows_host + i, (size_t)k * 4, st));
+        if (m->fam) {
+            TRY(m->fam->logits(m, m->rows, k, m->logits, st));
+        } else {
+            gather_rows_kernel<<<k, 256, 0, st>>>(m->x, m->rows, D, m->xlast);
+            TRY(launch_status());
+            TRY(flexllm_rmsnorm_quant(m->xlast, m->g_final, k, D, m->cfg.eps, FLEXLLM_NORM_PREFILL, nullptr, m->xq, m->xs, st));
+            TRY(flexllm_linear_decode_i8(m->xq, m->xs, m->lm_w, m->lm_s, k, V, D, nullptr, m->logits, st));
+        }
+        if (out) TRY(copy_any(out + (size_t)i * V, m->logits, (size_t)k * V * 4, st));
+    }
+    return FLEXLLM_OK;
+}
+
+static int extend_any(flexllm_model* m, const int32_t* tokens, int B, int n, const int32_t* want, int n_want, float* logits, bool pick,
+                      cudaStream_t st) {
+    const int base = m->pos;
+    int Sc = n;
+    std::vector<int32_t> rows;
+    for (int c0 = 0; c0 < n; c0 += m->cfg.max_prefill) {
+        Sc = n - c0 < m->cfg.max_prefill ? n - c0 : m->cfg.max_prefill;
+        if (m->fam) TRY(m->fam->forward(m, tokens, B, n, c0, Sc, st));
+        else TRY(prefill_chunk(m, tokens - base, nullptr, B, n, base + c0, Sc, st));       // indexes tokens by position
+        // wanted rows of this chunk, in runs that are consecutive in the output
+        for (int i = 0; i < n_want;) {
+            rows.clear();
+            int j = i;
+            for (; j < n_want; j++) {
+                const int b = want[j] / n, t = want[j] % n;
+                if (t < c0 || t >= c0 + Sc) break;
+                rows.push_back(b * Sc + t - c0);
+            }
+            if (j == i) { i++; continue; }
+            TRY(rows_to_logits(m, rows.data(), j - i, logits + (size_t)i * m->cfg.vocab, st));
+            i = j;
+        }
+        add_ctx_kernel<<<1, 64, 0, st>>>(m->ctx, B, Sc);
+        TRY(launch_status());
+    }
+    if (pick) {
+        rows.clear();
+        for (int b = 0; b < B; b++) rows.push_back(b * Sc + Sc - 1);
+        TRY(rows_to_logits(m, rows.data(), B, nullptr, st));
+        TRY(choose_tokens(m, B, st, nullptr));
+    }
+    m->B = B; m->pos = base + n; m->S = m->pos; m->last_chunk = Sc; m->rows_mode = false;
+    return FLEXLLM_OK;
+}
+
+extern "C" int flexllm_model_reset(flexllm_model* m, void* stream) {
+    FLEXLLM_REQUIRE(m);
+    fill_ctx_kernel<<<1, 64, 0, (cudaStream_t)stream>>>(m->ctx, 64, 0);
+    m->B = 0; m->pos = 0; m->S = 0;
+    return launch_status();
+}
+
+extern "C" int flexllm_model_extend(flexllm_model* m, const int32_t* tokens, int B, int n, const int32_t* want_host, int n_want,
+                                    float* logits, int32_t* next_out, void* stream) {
+    FLEXLLM_REQUIRE(m && tokens && B > 0 && B <= m->cfg.max_batch && n > 0 && (long)m->pos + n <= m->cfg.max_ctx);
+    FLEXLLM_REQUIRE(m->pos == 0 || B == m->B);                           // the same sequences as in the steps before
+    FLEXLLM_REQUIRE(n_want >= 0 && (n_want == 0 || (want_host && logits)));
+    for (int i = 0; i < n_want; i++) FLEXLLM_REQUIRE(want_host[i] >= 0 && want_host[i] < B * n);
+    if (m->fam) TRY(m->fam->check_loaded());
+    else if (m->g != 1 || m->pos % 128 || n % 16 || (n > m->cfg.max_prefill && m->cfg.max_prefill % 128)) return FLEXLLM_ENOTSUP;
+    TRY(extend_any(m, tokens, B, n, want_host, n_want, logits, next_out != nullptr, (cudaStream_t)stream));
+    if (next_out) TRY(copy_any(next_out, m->next, (size_t)B * 4, (cudaStream_t)stream));
+    return FLEXLLM_OK;
+}
+
+extern "C" int flexllm_model_extend_host(flexllm_model* m, const int32_t* tokens_host, int B, int n, const int32_t* want_host, int n_want,
+                                         float* logits_host, int32_t* next_host, void* stream) {
+    FLEXLLM_REQUIRE(m && tokens_host && B > 0 && B <= m->cfg.max_batch && n > 0 && (long)m->pos + n <= m->cfg.max_ctx);
+    for (long i = 0; i < (long)B * n; i++) FLEXLLM_REQUIRE(tokens_host[i] >= 0 && tokens_host[i] < m->cfg.vocab);
+    cudaStream_t st = (cudaStream_t)stream;
+    TRY(copy_any(m->tokens, tokens_host, (size_t)B * n * 4, st));
+    TRY(flexllm_model_extend(m, m->tokens, B, n, want_host, n_want, logits_host, next_host, stream));
+    FLEXLLM_CHECK_CUDA(cudaStreamSynchronize(st));
+    return gemm_check_error_flag();
+}
+
+extern "C" int flexllm_model_load_tensor(flexllm_model* m, const char* name, int dtype, int ndim, const int64_t* shape, const void* data, void* stream) {
+    FLEXLLM_REQUIRE(m && m->fam && name && ndim > 0 && shape && data);
+    return m->fam->load_tensor(m, name, dtype, ndim, shape, data, (cudaStream_t)stream);
+}
+
+extern "C" int flexllm_model_set_trace(flexllm_model* m, float* trace, size_t floats) {
+    FLEXLLM_REQUIRE(m);
+    return m->fam ? m->fam->set_trace(trace, floats) : FLEXLLM_ENOTSUP;
+}
+
 extern "C" int flexllm_model_prefill(flexllm_model* m, const int32_t* tokens, int B, int S, int32_t* next_out, void* stream) {
     FLEXLLM_REQUIRE(m && tokens && B > 0 && B <= m->cfg.max_batch && S > 0 && S <= m->cfg.max_ctx);
+    if (m->fam) {
+        TRY(m->fam->check_loaded());
+        TRY(flexllm_model_reset(m, stream));
+        TRY(extend_any(m, tokens, B, S, nullptr, 0, nullptr, true, (cudaStream_t)stream));
+        return next_out ? copy_any(next_out, m->next, (size_t)B * 4, (cudaStream_t)stream) : FLEXLLM_OK;
+    }
     if (S % 16 != 0) return FLEXLLM_ENOTSUP;
     if (S > m->cfg.max_prefill && m->cfg.max_prefill % 128 != 0) return FLEXLLM_ENOTSUP;     // chunks start at multiples of 128
     cudaStream_t st = (cudaStream_t)stream;
@@ -532,7 +625,7 @@ extern "C" int flexllm_model_prefill(flexllm_model* m, const int32_t* tokens, in
 extern "C" int flexllm_model_prefill_embeds(flexllm_model* m, const float* embeds, int B, int S, int n_valid, int32_t* next_out,
                                             void* stream) {
     FLEXLLM_REQUIRE(m && embeds && B > 0 && B <= m->cfg.max_batch && S > 0 && S <= m->cfg.max_ctx && n_valid > 0 && n_valid <= S);
-    if (m->g != 1 || S % 16 != 0) return FLEXLLM_ENOTSUP;
+    if (m->fam || m->g != 1 || S % 16 != 0) return FLEXLLM_ENOTSUP;
     if (S > m->cfg.max_prefill && m->cfg.max_prefill % 128 != 0) return FLEXLLM_ENOTSUP;
     FLEXLLM_REQUIRE(S - n_valid < (S > m->cfg.max_prefill ? S - (S - 1) / m->cfg.max_prefill * m->cfg.max_prefill : S));   // the last valid row lies in the last chunk
     return prefill_any(m, nullptr, embeds, B, S, n_valid, next_out, (cudaStream_t)stream);
@@ -541,6 +634,7 @@ extern "C" int flexllm_model_prefill_embeds(flexllm_model* m, const float* embed
 // Embedding rows of n token ids (tied embeddings: row t = (float)lm_head_q[t] * lm_head_s[t]): tokens [n] -> out [n][hidden].
 extern "C" int flexllm_model_embed_tokens(flexllm_model* m, const int32_t* tokens, int n, float* out, void* stream) {
     FLEXLLM_REQUIRE(m && tokens && out && n >= 0);
+    if (m->fam) return FLEXLLM_ENOTSUP;
     if (n == 0) return FLEXLLM_OK;
     embed_kernel<<<n, 256, 0, (cudaStream_t)stream>>>(tokens, m->lm_w, m->lm_s, m->cfg.hidden, m->cfg.vocab, out, device_error_flag(), 1, 0, 1, 0L);
     return launch_status();
@@ -553,7 +647,7 @@ extern "C" int flexllm_model_embed_tokens(flexllm_model* m, const int32_t* token
 static int mega_prepare(flexllm_model* m) {
     if (m->mega_state >= 0) return FLEXLLM_OK;
     m->mega_state = 0;
-    if (m->g != 1) return FLEXLLM_OK;
+    if (m->g != 1 || m->fam) return FLEXLLM_OK;
     std::vector<MegaLayerView> lv(m->cfg.layers);
     for (int l = 0; l < m->cfg.layers; l++) {
         const LayerW& w = m->L[l];
@@ -584,6 +678,13 @@ static int decode_step(flexllm_model* m, cudaStream_t st) {
     return rc;
 }
 static int decode_step_body(flexllm_model* m, cudaStream_t st) {
+    if (m->fam) {
+        TRY(m->fam->forward(m, m->next, m->B, 1, 0, 1, st));
+        TRY(m->fam->logits(m, nullptr, m->B, m->logits, st));
+        TRY(choose_tokens(m, m->B, st, m->state));
+        launch_k(step_bookkeeping_kernel, dim3(1), dim3(64), 0, st, (const int32_t*)m->next, m->B, m->out_tokens, m->state, m->ctx, 1);
+        return launch_status();
+    }
     const int D = m->cfg.hidden, HQ = m->HQl, HKV = m->HKVl, F = m->cfg.ffn;
     const int QKV = (HQ + 2 * HKV) * 64;
     const int B = m->B;
@@ -725,6 +826,24 @@ extern "C" int flexllm_model_set_sampling(flexllm_model* m, int lanes, int top_k
     if (m->graph) { cudaGraphExecDestroy(m->graph); m->graph = nullptr; }      // the captured step holds the old choice
     if (m->mega) mega_set_sampling(m->mega, m->sample_lanes, m->sample_k, m->sample_rnd);
     return FLEXLLM_OK;
+}
+
+// The same with the numbers rnd_host [n_new][B] in host memory, copied into a buffer of the model's own.
+extern "C" int flexllm_model_set_sampling_host(flexllm_model* m, int lanes, int top_k, const float* rnd_host, int n_new, int B) {
+    FLEXLLM_REQUIRE(m && top_k >= 0);
+    if (top_k == 0) return flexllm_model_set_sampling(m, 0, 0, nullptr);
+    FLEXLLM_REQUIRE(rnd_host && n_new > 0 && B > 0 && B <= m->cfg.max_batch);
+    const size_t n = (size_t)n_new * B;
+    if (n > m->own_rnd_floats) {
+        TRY(flexllm_model_set_sampling(m, 0, 0, nullptr));                     // drops the graph that holds the old buffer
+        FLEXLLM_CHECK_CUDA(cudaDeviceSynchronize());
+        if (m->own_rnd) cudaFree(m->own_rnd);
+        m->own_rnd = nullptr; m->own_rnd_floats = 0;
+        FLEXLLM_CHECK_CUDA(cudaMalloc(&m->own_rnd, n * 4));
+        m->own_rnd_floats = n;
+    }
+    FLEXLLM_CHECK_CUDA(cudaMemcpy(m->own_rnd, rnd_host, n * 4, cudaMemcpyHostToDevice));
+    return flexllm_model_set_sampling(m, lanes, top_k, m->own_rnd);
 }
 
 extern "C" int flexllm_model_limits(const flexllm_model* m, int* max_batch, int* max_prefill, int* max_ctx) {

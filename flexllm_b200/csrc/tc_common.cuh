@@ -124,6 +124,19 @@ __device__ __forceinline__ void umma_i8(uint32_t tmem_d, uint64_t adesc, uint64_
         ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate), "r"(0u)
         : "memory");
 }
+// Instruction descriptor for kind::f16 with bf16 operands (both K-major) and an fp32 accumulator.
+__host__ __device__ constexpr uint32_t umma_idesc_bf16(int M, int N) {
+    return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(N >> 3) << 17) | ((uint32_t)(M >> 4) << 24);
+}
+// D[tmem] (+)= A[smem] * B[smem]^T, one 128 x N x 16 bf16 step (32 bytes of K). Issued by ONE thread.
+__device__ __forceinline__ void umma_bf16(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p;\n\t"
+        "setp.ne.b32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}"
+        ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate), "r"(0u)
+        : "memory");
+}
 // Arrive on `bar` once every MMA issued so far by this thread has finished.
 __device__ __forceinline__ void umma_commit(uint32_t bar) {
     asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
@@ -167,5 +180,11 @@ int make_tmap_2d_u8_box(CUtensorMap* out, const void* base, uint64_t rows, uint6
 // one box = `kch` consecutive 128-byte chunks of `box_rows` rows, i.e. kch standard 128-byte-swizzled
 // tiles back to back in shared memory, fetched as kch*128 contiguous bytes per row.
 int make_tmap_3d_u8(CUtensorMap* out, const void* base, uint64_t rows, uint64_t row_bytes, uint32_t box_rows, uint32_t kch);
+// Row-major [outer][mid] rows of row_bytes bytes (the rows of one `outer` index back to back): a box of {128 bytes, box_mid rows,
+// box_outer} lands as box_outer * box_mid standard 128-byte-swizzled rows, outer-major.
+int make_tmap_rows3_u8(CUtensorMap* out, const void* base, uint64_t outer, uint64_t mid, uint64_t row_bytes, uint32_t box_outer,
+                       uint32_t box_mid);
+// make_tmap_2d_u8 / make_tmap_3d_u8 (kch != 0) behind a cache keyed by pointer and shape
+int cached_tmap_u8(CUtensorMap* out, const void* base, uint64_t rows, uint64_t row_bytes, uint32_t box_rows, uint32_t kch);
 
 }  // namespace flexllm

@@ -9,29 +9,9 @@ import ctypes as C
 import torch
 
 from . import _lib
-
-_handle = None
-
-
-class FlexLLMError(RuntimeError):
-    def __init__(self, fn, status):
-        l = lib()
-        msg = l.flexllm_status_string(status).decode()
-        super().__init__(f"{fn} failed: {msg} (status {status}, cuda error {l.flexllm_last_cuda_error()})")
-        self.status = status
-
-
-def lib():
-    global _handle
-    if _handle is None:
-        _handle = _lib.load()
-    return _handle
-
-
-def _check(fn, st):
-    if st != 0:
-        raise FlexLLMError(fn, st)
-
+from .models import HostModel
+from .runtime import FlexLLMError, lib  # noqa: F401
+from .runtime import check as _check
 
 def _ptr(t):
     if t is None:
@@ -249,6 +229,26 @@ def dec_Sampling_Layer(logits, rnd, lanes=32, top_k=5, details=False):
     _call("flexllm_topk_sample", _ptr(logits), B, V, lanes, top_k, _ptr(rnd), _ptr(idx), _ptr(ti) if details else None,
           _ptr(tv) if details else None)
     return (idx, ti, tv) if details else idx
+
+
+# ------------------------------------------------------------------------------ floating-point path
+def linear_float(a, w, bias=None, K=None, gelu_gate=False, out_f32=False):
+    """a [M,lda] bf16 or fp32, w [N,ldw] bf16 (columns from K on zero) -> [M,N] (gelu_gate: [M,N/2])."""
+    M, N = a.shape[0], w.shape[0]
+    dt = _lib.BF16 if a.dtype == torch.bfloat16 else _lib.F32
+    y = torch.empty((M, N // 2 if gelu_gate else N), dtype=torch.float32 if out_f32 else a.dtype, device=a.device)
+    _call("flexllm_linear_float", dt, _ptr(a), a.shape[1], _ptr(w), w.shape[1], _ptr(bias), M, N, a.shape[1] if K is None else K,
+          1 if gelu_gate else 0, _ptr(y), y.shape[1], 1 if out_f32 else 0)
+    return y
+
+
+def sandwich_norm(x, D, eps, y=None, gain_post=None, add_vec=None, gain_pre=None, dtype=torch.float32):
+    """In place x += rms(y) * gain_post, x += add_vec; returns h = rms(x) * gain_pre (or None). Rows zero-padded from D on."""
+    h = torch.zeros(x.shape, dtype=dtype, device=x.device) if gain_pre is not None else None
+    dt = _lib.BF16 if dtype == torch.bfloat16 else _lib.F32
+    _call("flexllm_sandwich_norm", dt, _ptr(x), x.shape[1], x.shape[0], D, float(eps), _ptr(y), y.shape[1] if y is not None else 0,
+          _ptr(gain_post), _ptr(add_vec), _ptr(gain_pre), _ptr(h), x.shape[1])
+    return h
 
 
 # ------------------------------------------------------------------------------ MHA_i8xi8
@@ -483,29 +483,46 @@ class TensorParallel:
         return out
 
 
-class Model:
+class Model(HostModel):
     """Whole-model runner (SpinQuant_Prefilling + SpinQuant_Decoding graphs). Weights are given as
     CUDA or CPU torch tensors (the library copies them; with `tp` every rank passes the full weights
-    and keeps its slice)."""
+    and keeps its slice). `Model.adopt(handle)` wraps a model of any other family."""
 
     def __init__(self, layers, hidden, heads_q, heads_kv, ffn, vocab, max_batch, max_prefill, max_ctx, eps=1e-5, tp=None):
         import math
         self.cfg = _lib.ModelConfig(layers, hidden, heads_q, heads_kv, ffn, vocab, eps, float(torch.tensor(math.sqrt(ffn), dtype=torch.float32)),
                                     max_batch, max_prefill, max_ctx)
         self._h = C.c_void_p()
-        self.tp = tp
+        self.tp, self.vocab = tp, vocab
         _check("flexllm_model_create_tp", lib().flexllm_model_create_tp(C.byref(self._h), C.byref(self.cfg), tp._h if tp else None))
 
-    def close(self):
-        if self._h:
-            lib().flexllm_model_destroy(self._h)
-            self._h = C.c_void_p()
+    @classmethod
+    def adopt(cls, host_model):
+        """The torch front end of a model made by models.load / models.create (which gives up its handle)."""
+        m = cls.__new__(cls)
+        m.tp, m._h, m.vocab = None, host_model._h, host_model.vocab
+        host_model._h = C.c_void_p()
+        return m
 
-    def __del__(self):
-        try:
-            self.close()
-        except Exception:
-            pass
+    def load_tensor(self, name, t):
+        """A bf16 tensor (CPU or CUDA) of a decoder-family model."""
+        assert t.dtype == torch.bfloat16
+        shape = (C.c_int64 * t.dim())(*t.shape)
+        _check("flexllm_model_load_tensor", lib().flexllm_model_load_tensor(self._h, name.encode(), _lib.BF16, t.dim(), shape, self._p(t), _stream()))
+        torch.cuda.current_stream().synchronize()
+
+    def extend(self, tokens, want=(), next_token=False):
+        """The next tokens [B,n] (CUDA int32) of the live sequences. Returns (logits [len(want), vocab] | None, next [B] | None)."""
+        B, n = tokens.shape
+        lg = torch.empty((len(want), self.vocab), dtype=torch.float32, device=tokens.device) if len(want) else None
+        nx = torch.empty((B,), dtype=torch.int32, device=tokens.device) if next_token else None
+        w = (C.c_int32 * max(1, len(want)))(*want)
+        _check("flexllm_model_extend", lib().flexllm_model_extend(self._h, _ptr(tokens), B, n, w, len(want), _ptr(lg), _ptr(nx), _stream()))
+        return lg, nx
+
+    def set_trace(self, buf=None):
+        """fp32 CUDA tensor [layer runs, B*n, width] that the following steps fill, or None."""
+        _check("flexllm_model_set_trace", lib().flexllm_model_set_trace(self._h, _ptr(buf), buf.numel() if buf is not None else 0))
 
     @staticmethod
     def _p(t):

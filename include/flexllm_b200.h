@@ -42,6 +42,10 @@ extern "C" {
 #define FLEXLLM_EDEVDATA (-7)  /* a token id or context length in DEVICE memory was out of range (clamped) */
 #define FLEXLLM_EIO (-8)       /* a parameter file could not be opened, or holds fewer values than asked for */
 
+/* Element types of the floating-point model path. */
+#define FLEXLLM_F32 0
+#define FLEXLLM_BF16 1
+
 /* RMSNorm summation orders (Modules/LayerNorm.h:82-130 prefill, :263-321 decode). */
 #define FLEXLLM_NORM_PREFILL 0 /* 4 interleaved partial sums over the whole row          */
 #define FLEXLLM_NORM_DECODE8 8 /* 8 contiguous chunks, 4 interleaved partial sums in each */
@@ -220,6 +224,11 @@ FLEXLLM_API int flexllm_mha_i8xi8_prefill_online(const int8_t* q, const float* q
  * ------------------------------------------------------------------------------------------- */
 typedef struct flexllm_kv_cache flexllm_kv_cache;
 FLEXLLM_API int flexllm_kv_cache_create(flexllm_kv_cache** out, int layers, int n_pages, int hkv, int page);
+/* Floating-point flavour (elem_bytes 2 = bf16, 4 = fp32): every layer has its own shape; K pages [n_pages][hkv][page][kdim],
+ * V pages [n_pages][hkv][vdim][page], no scales. destroy / reset / pools serve both flavours (pools: cast k and v; ks, vs NULL). */
+typedef struct { int hkv, kdim, vdim; } flexllm_kv_shape;
+FLEXLLM_API int flexllm_kv_cache_create_float(flexllm_kv_cache** out, int layers, int n_pages, const flexllm_kv_shape* shapes, int page,
+                                              int elem_bytes);
 FLEXLLM_API int flexllm_kv_cache_destroy(flexllm_kv_cache* c);
 FLEXLLM_API int flexllm_kv_cache_reset(flexllm_kv_cache* c, void* stream);
 /* raw device pointers of one layer's pools (for tests and zero-copy hand-off) */
@@ -320,6 +329,64 @@ FLEXLLM_API int flexllm_model_prefill_embeds(flexllm_model* m, const float* embe
 /* Embedding rows (tied embeddings) of n token ids: tokens [n] (device) -> out [n][hidden] fp32 (device). */
 FLEXLLM_API int flexllm_model_embed_tokens(flexllm_model* m, const int32_t* tokens, int n, float* out, void* stream);
 
+/* The next n tokens of each of the B live sequences, from the cache that earlier steps left (all sequences advance together;
+ * after flexllm_model_reset they start at position 0). tokens [B][n] (device). want_host[i] in [0, B*n) names a token of this
+ * call, row i of logits (host or device, [n_want][vocab] fp32) receives its logits; next_out (optional, device or host) the
+ * token chosen at the last position of every sequence, from which flexllm_model_begin / _decode go on. Steps of any length for
+ * the decoder family; the W8A8 Llama extends from multiples of 128 by multiples of 16. */
+FLEXLLM_API int flexllm_model_extend(flexllm_model* m, const int32_t* tokens, int B, int n, const int32_t* want_host, int n_want,
+                                     float* logits, int32_t* next_out, void* stream);
+/* The same with every buffer in host memory; synchronises and checks the device status. */
+FLEXLLM_API int flexllm_model_extend_host(flexllm_model* m, const int32_t* tokens_host, int B, int n, const int32_t* want_host, int n_want,
+                                          float* logits_host, int32_t* next_host, void* stream);
+/* Ends the live sequences: their pages are free for the next ones. */
+FLEXLLM_API int flexllm_model_reset(flexllm_model* m, void* stream);
+
+/* Decoder family with floating-point weights (the Pibidra design; no counterpart in the reference). Per layer
+ *     x += norm1b(attention(norm1(x)));   x += norm2b(down(gelu_tanh(gate h) * up h)), h = norm2(x)     (ff 0: no second part)
+ * with norm(x) = x / sqrt(mean x^2 + eps) * (1 + w); attention: see flexllm_attn_window. Layers loop_start .. loop_stop-1
+ * run loop_times times with the same weights (0: no loop); before pass t the vector loop.step[t], and from the second pass
+ * on also the embedding output, is added to x. Every layer run has its own cache. The pages of a sequence are a ring that
+ * holds the widest window and one chunk of max_prefill tokens, so memory does not grow with max_ctx.
+ * dtype FLEXLLM_BF16: bf16 products and activations, fp32 residual stream, norms, scores and softmax; FLEXLLM_F32: all fp32.
+ * The model is an ordinary flexllm_model: prefill (any length), begin, decode, generate_host, set_sampling, extend. */
+typedef struct {
+    int heads, kv_heads, dim, vdim;       /* attention: query heads, key/value heads, query/key size, value size */
+    int window, bias_max;                 /* i sees j with 0 <= i - j < window; distance at which the bias table saturates */
+    float scale, softcap;                 /* softcap 0: none */
+    int ff;                               /* feed-forward size, 0: none */
+} flexllm_decoder_layer;
+typedef struct {
+    int layers, width, vocab;
+    float eps, embed_scale;
+    int loop_start, loop_stop, loop_times;
+    int max_batch, max_prefill, max_ctx;
+    int dtype;
+    const flexllm_decoder_layer* layer;   /* [layers] */
+} flexllm_decoder_config;
+FLEXLLM_API int flexllm_model_create_decoder(flexllm_model** out, const flexllm_decoder_config* cfg);
+/* One bf16 weight tensor by name (host or device memory, dense; linear weights [out][in]): embed, head, final.norm, loop.step,
+ * l<i>.norm1 / norm1b / norm2 / norm2b, l<i>.mix.{q,k,v}[.b], .q.norm, .k.norm, .rel, .g, .o, l<i>.mlp.{gate,up,down}.
+ * Steps are refused (FLEXLLM_EINVAL) until every tensor is there. */
+FLEXLLM_API int flexllm_model_load_tensor(flexllm_model* m, const char* name, int dtype, int ndim, const int64_t* shape, const void* data,
+                                          void* stream);
+/* Every tensor of a .safetensors file that the model knows, by name. */
+FLEXLLM_API int flexllm_model_load_safetensors(flexllm_model* m, const char* path, void* stream);
+/* Tests: the following steps also store the residual stream after every layer run, [layer runs][B*n][width] fp32 (device;
+ * NULL turns it off). */
+FLEXLLM_API int flexllm_model_set_trace(flexllm_model* m, float* trace, size_t floats);
+
+/* Operators of that family.
+ * linear_float: y[m][n] = sum_k a[m][k] w[n][k] (+ bias[n]); a of type dtype [M][lda], w bf16 [N][ldw], lda and ldw multiples of 8
+ * and >= K rounded up to 8 (w zero and a finite from K on). gelu_gate: the rows of w alternate in blocks of 16 gate and 16 up
+ * rows, y[m][f] = gelu_tanh(gate) * up, N = 2 F, N % 32 == 0. y of type dtype, or fp32 (y_f32).
+ * sandwich_norm: x += y / rms(y) * gain_post (y NULL: nothing); x += add_vec; h (type dtype) = x / rms(x) * gain_pre. Rows are
+ * padded with zeros to multiples of 4. */
+FLEXLLM_API int flexllm_linear_float(int dtype, const void* a, long lda, const void* w, long ldw, const float* bias, int M, int N, int K,
+                                     int gelu_gate, void* y, long ldy, int y_f32, void* stream);
+FLEXLLM_API int flexllm_sandwich_norm(int dtype, float* x, long ldx, int M, int D, float eps, const float* y, long ldy, const float* gain_post,
+                                      const float* add_vec, const float* gain_pre, void* h, long ldh, void* stream);
+
 /* ---------------------------------------------------------------------------------------------
  * HMT long-context plug-in (Modules/HMT.h; HMT_SpinQuant_Llama_32_1B/): the prompt is processed in segments of seg_len
  * tokens through the same prefill path; per segment a summary pass over [T, first sum_len tokens, T] queries a ring of
@@ -345,6 +412,9 @@ FLEXLLM_API int flexllm_hmt_prefill(flexllm_hmt* h, const float* embeds, int T, 
  * output column c -- the reference's rand_seeds_mmap, one number per decode step (SpinQuant_Decoding_mem_opt.h:934-937).
  * The token feedback stays on the device in both decode paths. Single GPU only. */
 FLEXLLM_API int flexllm_model_set_sampling(flexllm_model* m, int lanes, int top_k, const float* rnd);
+
+/* The same with rnd_host [n_new][B] in host memory (copied). */
+FLEXLLM_API int flexllm_model_set_sampling_host(flexllm_model* m, int lanes, int top_k, const float* rnd_host, int n_new, int B);
 
 /* Measurement aid: the prefill GEMM's TMA -> shared memory -> tcgen05.mma kind::i8 -> TMEM pipeline on
  * a [M][K] x [N][K] problem with an epilogue that reads the accumulators and stores nothing. Its rate is
