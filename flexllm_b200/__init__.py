@@ -15,4 +15,5 @@ from . import _lib
 def __getattr__(name):          # the operators (and with them torch) are imported when first asked for
     if name.startswith("__"):
         raise AttributeError(name)
-    return getattr(importlib.import_module(".ops", __name__), name)
+    ops = importlib.import_module(".ops", __name__)
+    return ops if name == "ops" else getattr(ops, name)

@@ -84,6 +84,11 @@ SIGNATURES = {
     "flexllm_model_set_trace": [_P, _P, _SZ],
     "flexllm_linear_float": [_I, _P, _L, _P, _L, _P, _I, _I, _I, _I, _P, _L, _I, _P],
     "flexllm_sandwich_norm": [_I, _P, _L, _I, _I, _F, _P, _L, _P, _P, _P, _P, _L, _P],
+    "flexllm_attn_window_row": [_P],
+    "flexllm_attn_window_bias_floats": [_P],
+    "flexllm_attn_window_bias": [_P, _P, _I, _I, _P, _P],
+    "flexllm_attn_window_workspace": [_P, _I, _I],
+    "flexllm_attn_window": [_I, _P, _I, _P, _P, _P, _P, _P, _F, _P, _I, _P, _I, _I, _I, _P, _L, _P, _SZ, _P],
     "flexllm_hmt_create": [_P, _P, _P, _I, _P, _P, _P],
     "flexllm_hmt_destroy": [_P],
     "flexllm_hmt_prefill": [_P, _P, _I, _P, _P, _P],
@@ -114,6 +119,15 @@ class DecoderConfig(C.Structure):
                 ("loop_times", _I), ("max_batch", _I), ("max_prefill", _I), ("max_ctx", _I), ("dtype", _I), ("layer", C.POINTER(DecoderLayer))]
 
 
+class KvShape(C.Structure):
+    _fields_ = [("hkv", _I), ("kdim", _I), ("vdim", _I)]
+
+
+class AttnWindowShape(C.Structure):
+    _fields_ = [("heads", _I), ("kv_heads", _I), ("dim", _I), ("vdim", _I), ("window", _I), ("sink", _I), ("gate", _I), ("scale", _F),
+                ("softcap", _F), ("eps", _F)]
+
+
 class CkptLayerBuffers(C.Structure):
     _fields_ = ([(n, _P) for n in ("wq", "wk", "wv", "wo", "wg", "wu", "wd")] + [(n, _P) for n in ("sq", "sk", "sv", "so", "sg", "su", "sd")] +
                 [(n, _P) for n in ("sumq", "sumk", "sumv", "sumo", "sumg", "sumu", "sumd")] + [(n, _P) for n in ("gamma0", "gamma1", "a_s")])
@@ -128,7 +142,8 @@ class LayerWeights(C.Structure):
                                   "gamma0", "gamma1", "a_s")]
 
 RESTYPES = {"flexllm_status_string": C.c_char_p, "flexllm_launch_count": C.c_ulonglong, "flexllm_mha_prefill_workspace": C.c_size_t,
-            "flexllm_mha_decode_workspace": C.c_size_t, "flexllm_mlp_block_workspace": C.c_size_t}
+            "flexllm_mha_decode_workspace": C.c_size_t, "flexllm_mlp_block_workspace": C.c_size_t,
+            "flexllm_attn_window_row": C.c_long, "flexllm_attn_window_bias_floats": C.c_size_t, "flexllm_attn_window_workspace": C.c_size_t}
 
 
 def load():

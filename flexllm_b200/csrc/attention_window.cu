@@ -10,11 +10,11 @@
 //   prompts, bf16          : attn_prepare_kernel, then attn_window_prefill_kernel on tcgen05
 //   prompts, otherwise     : attn_prepare_kernel, then attn_row_kernel row by row
 // The sink is a score of 0, so max(0, largest score) is a valid softmax shift; without a sink the running maximum is.
-#include <math.h>
-
-#include <atomic>
+#include <cmath>
+#include <vector>
 
 #include "float_common.cuh"
+#include "kv_cache.h"
 #include "tc_common.cuh"
 
 namespace flexllm {
@@ -676,6 +676,37 @@ size_t attn_window_ws_floats(int max_batch, int G, int R, int dv) {
     return n * (size_t)R * (dv + 2);
 }
 
+void attn_layout(AttnShape* s, bool gate) {
+    s->dkp = (int)up_to(s->dk, 8);
+    s->q_off = 0;
+    s->k_off = (int)up_to((long)s->H * s->dk, 8);
+    s->v_off = s->k_off + (int)up_to((long)s->G * s->dk, 8);
+    const int end = s->v_off + (int)up_to((long)s->G * s->dv, 8);
+    s->g_off = gate ? end : -1;
+    s->ld = gate ? end + up_to((long)s->H * s->dv, 8) : end;
+}
+
+// Row of the distance table for distance n: exact below half the rows, logarithmic up to bias_max from there on. A quotient
+// of logarithms that is an integer in exact arithmetic must not fall below it by rounding.
+static int distance_bucket(int n, int rows, int bias_max) {
+    const int half = rows / 2;
+    if (n < half) return n;
+    if (half == 0 || bias_max <= half) return rows - 1;
+    const double v = std::log((double)n / half) / std::log((double)bias_max / half) * (rows - half);
+    const double b = half + std::floor(v + 1e-9);
+    return b < rows - 1 ? (int)b : rows - 1;
+}
+
+void attn_bias_table(const AttnShape& s, const float* table, int rows, int bias_max, float* out) {
+    const int R = s.H / s.G;
+    const size_t n = 2 * (size_t)kBiasPad + s.window;
+    for (size_t i = 0; i < (size_t)s.H * n; i++) out[i] = -INFINITY;
+    for (int d = 0; d < s.window; d++) {
+        const int bk = distance_bucket(d, rows, bias_max);
+        for (int h = 0; h < s.H; h++) out[((h / R) * n + kBiasPad + d) * R + h % R] = table[(size_t)bk * s.H + h];
+    }
+}
+
 template <class T> int attn_window(const AttnCall& c, cudaStream_t st) {
     TRY_RC(check_call(c));
     if (c.Sc == 1) return run_row<T, true>(c, st);
@@ -691,3 +722,62 @@ template int attn_window<float>(const AttnCall&, cudaStream_t);
 template int attn_window<bf16>(const AttnCall&, cudaStream_t);
 
 }  // namespace flexllm
+
+using namespace flexllm;
+
+// ---- C ABI, see include/flexllm_b200.h
+namespace {
+bool make_shape(const flexllm_attn_window_shape* a, AttnShape* s) {
+    if (!a || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->dim <= 0 || a->vdim <= 0 || a->window <= 0) return false;
+    *s = AttnShape();
+    s->H = a->heads; s->G = a->kv_heads; s->dk = a->dim; s->dv = a->vdim; s->window = a->window;
+    s->scale = a->scale; s->softcap = a->softcap; s->sink = a->sink ? 1 : 0;
+    attn_layout(s, a->gate != 0);
+    return true;
+}
+struct WindowWs { size_t ws_floats, counters, q, total; };      // byte offsets of the counters and of the q scratch
+WindowWs window_ws(const AttnShape& s, int B, int n) {
+    WindowWs w;
+    w.ws_floats = attn_window_ws_floats(B, s.G, s.H / s.G, s.dv);
+    w.counters = (w.ws_floats * 4 + 255) / 256 * 256;
+    w.q = w.counters + ((size_t)B * s.G * 4 + 255) / 256 * 256;
+    w.total = w.q + (size_t)B * n * s.H * s.dkp * 4 + 256;
+    return w;
+}
+}  // namespace
+
+extern "C" long flexllm_attn_window_row(const flexllm_attn_window_shape* a) { AttnShape s; return make_shape(a, &s) ? s.ld : 0; }
+extern "C" size_t flexllm_attn_window_bias_floats(const flexllm_attn_window_shape* a) { AttnShape s; return make_shape(a, &s) ? attn_bias_floats(s) : 0; }
+extern "C" size_t flexllm_attn_window_workspace(const flexllm_attn_window_shape* a, int B, int n) {
+    AttnShape s;
+    return make_shape(a, &s) && B > 0 && n > 0 ? window_ws(s, B, n).total : 0;
+}
+extern "C" int flexllm_attn_window_bias(const flexllm_attn_window_shape* a, const float* table_host, int rows, int bias_max, float* bias, void* stream) {
+    AttnShape s;
+    FLEXLLM_REQUIRE(make_shape(a, &s) && table_host && rows > 0 && bias);
+    std::vector<float> t(attn_bias_floats(s));
+    attn_bias_table(s, table_host, rows, bias_max, t.data());
+    FLEXLLM_CHECK_CUDA(cudaMemcpyAsync(bias, t.data(), t.size() * 4, cudaMemcpyHostToDevice, (cudaStream_t)stream));
+    return cuda_status(cudaStreamSynchronize((cudaStream_t)stream));
+}
+extern "C" int flexllm_attn_window(int dtype, flexllm_kv_cache* kv, int layer, const flexllm_attn_window_shape* a, const void* proj,
+                                   const float* q_gain, const float* k_gain, const float* bias, float bias_abs, const int32_t* page_table,
+                                   int max_pages, const int32_t* ctx, int max_ctx, int B, int n, void* out, long ldo, void* workspace,
+                                   size_t workspace_bytes, void* stream) {
+    AttnCall c = {};
+    FLEXLLM_REQUIRE(make_shape(a, &c.s) && kv && layer >= 0 && layer < kv->layers && B > 0 && n > 0);
+    FLEXLLM_REQUIRE(dtype == FLEXLLM_F32 || dtype == FLEXLLM_BF16);
+    FLEXLLM_REQUIRE(kv->elem_bytes == (dtype == FLEXLLM_BF16 ? 2 : 4));
+    const flexllm_kv_shape& ks = kv->shape[layer];
+    FLEXLLM_REQUIRE(ks.hkv == c.s.G && ks.kdim == c.s.dkp && ks.vdim == c.s.dv && ldo >= (long)c.s.H * c.s.dv);
+    const WindowWs w = window_ws(c.s, B, n);
+    FLEXLLM_REQUIRE(workspace && aligned(workspace, 256) && workspace_bytes >= w.total && aligned(proj, 16) && aligned(out, 16));
+    c.proj = proj; c.q_gain = q_gain; c.k_gain = k_gain; c.eps = a->eps; c.bias = bias; c.bias_max_abs = bias_abs;
+    c.k_pool = kv->k + kv->k_off[layer]; c.v_pool = kv->v + kv->v_off[layer]; c.n_pages = kv->n_pages;
+    c.page_table = page_table; c.max_pages = max_pages; c.ctx = ctx; c.max_pos = max_ctx; c.B = B; c.Sc = n;
+    c.ws = (float*)workspace; c.ws_floats = w.ws_floats; c.counters = (int*)((char*)workspace + w.counters); c.n_counters = B * c.s.G;
+    c.q = (char*)workspace + w.q; c.out = out; c.ldo = ldo;
+    cudaStream_t st = (cudaStream_t)stream;
+    FLEXLLM_CHECK_CUDA(cudaMemsetAsync(c.counters, 0, (size_t)c.n_counters * 4, st));
+    return dtype == FLEXLLM_BF16 ? attn_window<bf16>(c, st) : attn_window<float>(c, st);
+}

@@ -140,5 +140,10 @@ struct AttnCall {
 // bf16 shapes it covers, row by row otherwise).
 template <class T> int attn_window(const AttnCall& c, cudaStream_t st);
 size_t attn_window_ws_floats(int max_batch, int G, int R, int dv);
+// Fills in the derived members: dkp, the columns of the fused projection (parts padded to multiples of 8) and its row length.
+void attn_layout(AttnShape* s, bool gate);
+// The bias table of AttnCall::bias on the host, from a table [rows][H] of learned biases by bucketed distance.
+void attn_bias_table(const AttnShape& s, const float* table, int rows, int bias_max, float* out);
+inline size_t attn_bias_floats(const AttnShape& s) { return (size_t)s.H * (2 * kBiasPad + s.window); }
 
 }  // namespace flexllm

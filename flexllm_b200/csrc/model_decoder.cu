@@ -32,17 +32,6 @@ struct DecLayer {
     float bias_max = 0.0f;
 };
 
-// Row of the distance table for distance n: exact below half the rows, logarithmic up to bias_max from there on. A quotient
-// of logarithms that is an integer in exact arithmetic must not fall below it by rounding.
-int distance_bucket(int n, int rows, int bias_max) {
-    const int half = rows / 2;
-    if (n < half) return n;
-    if (half == 0 || bias_max <= half) return rows - 1;
-    const double v = std::log((double)n / half) / std::log((double)bias_max / half) * (rows - half);
-    const int b = half + (int)std::floor(v + 1e-9);
-    return b < rows - 1 ? b : rows - 1;
-}
-
 float bf16_to_float(uint16_t v) { uint32_t u = (uint32_t)v << 16; float f; memcpy(&f, &u, 4); return f; }
 
 struct Want { std::string name; std::vector<int64_t> shape; bool loaded; };
@@ -115,15 +104,11 @@ class DecoderFamily : public ModelFamily {
             l.c = specs[i];
             const flexllm_decoder_layer& a = l.c;
             AttnShape& s = l.s;
-            s.H = a.heads; s.G = a.kv_heads; s.dk = a.dim; s.dv = a.vdim; s.dkp = (int)up_to(a.dim, 8);
+            s.H = a.heads; s.G = a.kv_heads; s.dk = a.dim; s.dv = a.vdim;
             s.window = a.window < cfg.max_ctx + 1 ? a.window : cfg.max_ctx + 1;      // nothing is further away than that
             s.scale = a.scale; s.softcap = a.softcap; s.sink = 1;
-            s.q_off = 0;
-            s.k_off = (int)up_to((long)s.H * s.dk, 8);
-            s.v_off = s.k_off + (int)up_to((long)s.G * s.dk, 8);
-            s.g_off = s.v_off + (int)up_to((long)s.G * s.dv, 8);
-            l.proj_n = s.g_off + (int)up_to((long)s.H * s.dv, 8);
-            s.ld = l.proj_n;
+            attn_layout(&s, true);
+            l.proj_n = (int)s.ld;
             l.ffp = (int)up_to(a.ff, 16);
             max_window = s.window > max_window ? s.window : max_window;
             max_proj = l.proj_n > max_proj ? l.proj_n : max_proj;
@@ -138,7 +123,7 @@ class DecoderFamily : public ModelFamily {
             TRY(alloc(&l.n1b, (size_t)ldD * 4));
             TRY(alloc(&l.q_gain, (size_t)s.H * s.dk * 4));
             TRY(alloc(&l.k_gain, (size_t)s.G * s.dk * 4));
-            TRY(alloc(&l.bias, (size_t)s.H * (2 * kBiasPad + s.window) * 4));
+            TRY(alloc(&l.bias, attn_bias_floats(s) * 4));
             const std::string p = "l" + std::to_string(i) + ".", m = p + "mix.";
             want(p + "norm1", {D});
             want(p + "norm1b", {D});
@@ -234,14 +219,10 @@ class DecoderFamily : public ModelFamily {
     int put_distance_bias(DecLayer& l, const void* src, int rows, cudaStream_t st) {
         std::vector<float> t;
         TRY(get_floats(src, (long)rows * l.s.H, 0.0f, &t, st));
-        const int R = l.s.H / l.s.G, W = l.s.window, n = 2 * kBiasPad + W;
-        std::vector<float> out((size_t)l.s.H * n, -INFINITY);
         l.bias_max = 0.0f;
         for (float v : t) l.bias_max = std::fmax(l.bias_max, std::fabs(v));
-        for (int d = 0; d < W; d++) {
-            const int bk = distance_bucket(d, rows, l.c.bias_max);
-            for (int hd = 0; hd < l.s.H; hd++) out[((size_t)(hd / R) * n + kBiasPad + d) * R + hd % R] = t[(size_t)bk * l.s.H + hd];
-        }
+        std::vector<float> out(attn_bias_floats(l.s));
+        attn_bias_table(l.s, t.data(), rows, l.c.bias_max, out.data());
         return put_floats(l.bias, out, st);
     }
 

@@ -387,6 +387,26 @@ FLEXLLM_API int flexllm_linear_float(int dtype, const void* a, long lda, const v
 FLEXLLM_API int flexllm_sandwich_norm(int dtype, float* x, long ldx, int M, int D, float eps, const float* y, long ldy, const float* gain_post,
                                       const float* add_vec, const float* gain_pre, void* h, long ldh, void* stream);
 
+/* Windowed grouped-query attention on one layer of a floating-point cache, B sequences x n new tokens at positions ctx[b]..:
+ *   q, k = rms norm of the whole q (k) projection * gain;  s = softcap * tanh(scale * (q . k) / softcap) + bias[head][i - j]
+ *   for 0 <= i - j < window;  p = exp(s) / (sink + sum exp(s));  out = (sum p v) * logistic(gate)
+ * The new keys and values are appended to the cache first. proj: rows of q | k | v | gate, each part padded to a multiple of 8
+ * columns, row length flexllm_attn_window_row(shape) (gate 0: no gate part); cache element type = dtype, kdim = dim rounded up
+ * to 8. bias: flexllm_attn_window_bias_floats(shape) floats in device memory made by flexllm_attn_window_bias from a table
+ * [rows][heads] in host memory: distance d < rows/2 uses row d, larger ones min(rows-1, rows/2 + floor(ln(d/(rows/2)) /
+ * ln(bias_max/(rows/2)) * (rows - rows/2))); bias_abs: its largest magnitude. max_ctx: largest position the page table covers.
+ * out [B*n][ldo] of type dtype, ldo >= heads * vdim. n == 1 is the decode form. */
+typedef struct { int heads, kv_heads, dim, vdim, window, sink, gate; float scale, softcap, eps; } flexllm_attn_window_shape;
+FLEXLLM_API long flexllm_attn_window_row(const flexllm_attn_window_shape* s);
+FLEXLLM_API size_t flexllm_attn_window_bias_floats(const flexllm_attn_window_shape* s);
+FLEXLLM_API int flexllm_attn_window_bias(const flexllm_attn_window_shape* s, const float* table_host, int rows, int bias_max, float* bias,
+                                         void* stream);
+FLEXLLM_API size_t flexllm_attn_window_workspace(const flexllm_attn_window_shape* s, int B, int n);
+FLEXLLM_API int flexllm_attn_window(int dtype, flexllm_kv_cache* c, int layer, const flexllm_attn_window_shape* s, const void* proj,
+                                    const float* q_gain, const float* k_gain, const float* bias, float bias_abs,
+                                    const int32_t* page_table, int max_pages, const int32_t* ctx, int max_ctx, int B, int n, void* out,
+                                    long ldo, void* workspace, size_t workspace_bytes, void* stream);
+
 /* ---------------------------------------------------------------------------------------------
  * HMT long-context plug-in (Modules/HMT.h; HMT_SpinQuant_Llama_32_1B/): the prompt is processed in segments of seg_len
  * tokens through the same prefill path; per segment a summary pass over [T, first sum_len tokens, T] queries a ring of

@@ -43,7 +43,7 @@ def bucket(n, rows, bias_max):
     half = rows // 2
     if n < half:
         return n
-    if bias_max <= half:
+    if half == 0 or bias_max <= half:
         return rows - 1
     return min(rows - 1, half + math.floor(math.log(n / half) / math.log(bias_max / half) * (rows - half)))
 
@@ -69,6 +69,25 @@ def sink_softmax(s):
     return e / (math.exp(-m) + e.sum())
 
 
+def head_outputs(q, k, v, table, mx, sink=True):
+    """q [S, H, dk], k [S, G, dk], v [S, G, dv] (normed already) -> [S, H, dv]. mx: window (mask.size), scale, softcap, bias_max."""
+    S, H, _ = q.shape
+    G, size = k.shape[1], mx["mask"]["size"]
+    bias = np.stack([distance_bias(table, mx["bias_max"], n) for n in range(min(size, S))])           # [distance, H]
+    o = np.zeros((S, H, v.shape[2]), F)
+    for i in range(S):
+        keys = np.array(window_keys(i, size))
+        for hd in range(H):
+            g = hd // (H // G)
+            s = k[keys, g] @ q[i, hd] * mx["scale"]
+            if mx["softcap"]:
+                s = softcapped(s, mx["softcap"])
+            s = s + bias[i - keys, hd]
+            p = sink_softmax(s) if sink else np.exp(s - s.max()) / np.exp(s - s.max()).sum()
+            o[i, hd] = p @ v[keys, g]
+    return o
+
+
 def attention(h, t, pre, mx, eps):
     """The mixer on h [S, width]; t: tensors, pre: 'l<i>.mix.'."""
     S = h.shape[0]
@@ -78,19 +97,8 @@ def attention(h, t, pre, mx, eps):
     v = linear(t[pre + "v"], h, t[pre + "v.b"])
     q = norm_plain(q, t[pre + "q.norm"], eps).reshape(S, H, dk)      # the norm runs over all heads at once
     k = norm_plain(k, t[pre + "k.norm"], eps).reshape(S, G, dk)
-    v = v.reshape(S, G, dv)
-    o = np.zeros((S, H, dv), F)
-    for i in range(S):
-        keys = window_keys(i, mx["mask"]["size"])
-        lo = keys[0]
-        bias = np.stack([distance_bias(t[pre + "rel"], mx["bias_max"], i - j) for j in keys])      # [keys, H]
-        for hd in range(H):
-            g = hd // (H // G)
-            s = k[lo:i + 1, g] @ q[i, hd] * mx["scale"]
-            s = softcapped(s, mx["softcap"]) + bias[:, hd]
-            o[i, hd] = sink_softmax(s) @ v[lo:i + 1, g]
-    o = o.reshape(S, H * dv) * sigmoid(linear(t[pre + "g"], h))
-    return linear(t[pre + "o"], o)
+    o = head_outputs(q, k, v.reshape(S, G, dv), t[pre + "rel"], mx).reshape(S, H * dv)
+    return linear(t[pre + "o"], o * sigmoid(linear(t[pre + "g"], h)))
 
 
 def feed_forward(h, t, pre):
