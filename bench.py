@@ -577,6 +577,12 @@ def micro(args):
         synthetic.load_random_weights(m, max_ctx=1040, seed=0, **cfg2)
         tok = torch.randint(0, CFG["vocab"], (8, 1024), dtype=torch.int32).cuda()
         fn = lambda: m.prefill(tok)
+    elif name in ("pibidra_prefill", "pibidra_decode"):      # two layers of the Llama's sizes: every kernel of the family at its model shapes
+        S, B = 1024, 8 if name == "pibidra_prefill" else 4
+        m = pibidra_model(F, torch, PIBIDRA_SIZES["llama1b"], B, S, S + 64, layers=2)
+        tok = torch.randint(0, CFG["vocab"], (B, S), dtype=torch.int32).cuda()
+        m.prefill(tok); m.begin(32)
+        fn = (lambda: m.prefill(tok)) if name == "pibidra_prefill" else (lambda: m.decode(4, False))
     elif name == "decode_step":         # whole-model decode steps (one persistent kernel each) at a short context: small enough for ncu
         S, n = 128, 6
         m = F.Model(max_batch=BATCH, max_prefill=S, max_ctx=S + 16, **CFG)
@@ -600,6 +606,199 @@ def micro(args):
         fn()
     e1.record(); torch.cuda.synchronize()
     print(json.dumps({"micro": name, "ms": e0.elapsed_time(e1) / 3}))
+
+
+# ------------------------------------------------------------------------------------ the Pibidra family
+# layers of the sizes of real models, random weights; window 1024 so that a prompt of 1024 is as wide as the Llama's causal
+# attention. The first size is the Llama's own (its closest existing model); the others have heads of 128.
+PIBIDRA_SIZES = {
+    "llama1b": dict(layers=16, width=2048, heads=32, kv_heads=8, dim=64, vdim=64, ff=8192, vocab=128256, window=1024),
+    "wide": dict(layers=8, width=4096, heads=32, kv_heads=8, dim=128, vdim=128, ff=14336, vocab=128256, window=1024),
+    "small": dict(layers=12, width=1024, heads=8, kv_heads=2, dim=128, vdim=128, ff=4096, vocab=32000, window=512),
+}
+
+
+def pibidra_model(F, torch, z, max_batch, max_prefill, max_ctx, layers=None, seed=0):
+    """A model of size z with random bf16 weights, made on the device."""
+    from flexllm_b200 import models
+    L = layers or z["layers"]
+    layer = {"type": "attention", "mixer": dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"], vdim=z["vdim"], mask={"size": z["window"]},
+                                               bias_max=z["window"], softcap=30.0, scale=z["dim"] ** -0.5), "mlp": {"kind": "dense", "ff": z["ff"]}}
+    cfg = {"architecture": "Pibidra", "embedding": {"scale": 1.0}, "layers": [layer] * L, "norm": {"eps": 1e-5}, "vocab": z["vocab"], "width": z["width"]}
+    m = F.Model.adopt(models.create(cfg, max_batch, max_prefill, max_ctx, "bfloat16"))
+    g = torch.Generator(device="cuda").manual_seed(seed)
+    D, H, G, dk, dv, ff, V = z["width"], z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["ff"], z["vocab"]
+    rn = lambda *sh, s=1.0: (torch.randn(sh, device="cuda", generator=g) * s).to(torch.bfloat16)
+    m.load_tensor("embed", rn(V, D)); m.load_tensor("head", rn(V, D, s=D ** -0.5)); m.load_tensor("final.norm", rn(D, s=0.1))
+    for i in range(L):
+        p = "l%d." % i
+        for n in ("norm1", "norm1b", "norm2", "norm2b"):
+            m.load_tensor(p + n, rn(D, s=0.1))
+        for n, r in (("q", H * dk), ("k", G * dk), ("v", G * dv)):
+            m.load_tensor(p + "mix." + n, rn(r, D, s=D ** -0.5)); m.load_tensor(p + "mix." + n + ".b", rn(r, s=0.1))
+        m.load_tensor(p + "mix.q.norm", 1 + rn(H * dk, s=0.1)); m.load_tensor(p + "mix.k.norm", 1 + rn(G * dk, s=0.1))
+        m.load_tensor(p + "mix.rel", rn(32, H, s=0.5)); m.load_tensor(p + "mix.g", rn(H * dv, D, s=D ** -0.5))
+        m.load_tensor(p + "mix.o", rn(D, H * dv, s=(H * dv) ** -0.5))
+        m.load_tensor(p + "mlp.gate", rn(ff, D, s=D ** -0.5)); m.load_tensor(p + "mlp.up", rn(ff, D, s=D ** -0.5))
+        m.load_tensor(p + "mlp.down", rn(D, ff, s=ff ** -0.5))
+    return m
+
+
+def pibidra_work(z, B, S, ctx):
+    """(prefill FLOPs of B prompts of S, bytes one decode step of B sequences at context ctx has to read)."""
+    D, H, G, dk, dv, ff, V, W, L = (z[k] for k in ("width", "heads", "kv_heads", "dim", "vdim", "ff", "vocab", "window", "layers"))
+    w = D * (H * dk + G * dk + G * dv + H * dv) + H * dv * D + 3 * D * ff
+    pairs = sum(min(i + 1, W) for i in range(S))
+    flops = 2.0 * B * S * L * w + 2.0 * B * L * H * (dk + dv) * pairs + 2.0 * B * V * D
+    return flops, 2.0 * (L * w + V * D) + 2.0 * L * B * min(ctx, W) * G * (dk + dv)
+
+
+def event_ms(torch, fn, n, warm=3):
+    for i in range(warm):
+        fn(i)
+    torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record()
+    for i in range(n):
+        fn(i)
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) / n
+
+
+def graph_ms(torch, fn, n=40):
+    """Mean device time of fn(i, stream), replayed n times from a CUDA graph."""
+    side = torch.cuda.Stream()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.stream(side):
+        for i in range(3):
+            fn(i)
+        side.synchronize()
+        with torch.cuda.graph(graph, stream=side):
+            for i in range(n):
+                fn(i)
+        graph.replay(); side.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(side); graph.replay(); e1.record(side)
+        side.synchronize()
+    return e0.elapsed_time(e1) / n
+
+
+def pibidra_kernels(F, torch, peaks):
+    """The family's kernels beside the like kernels of the W8A8 Llama at the Llama's layer sizes: time and fraction of the
+    roofline (bf16 products against the measured bf16 peak, int8 ones against twice that; bytes against the copy rate)."""
+    hbm, tf = peaks.get("hbm_gbs") or 6650.0, peaks.get("bf16_tflops") or 1590.0
+    out = {}
+
+    def note(name, ms, flops=0.0, nbytes=0.0, peak_tf=tf):
+        floor = max(flops / peak_tf / 1e9, nbytes / hbm / 1e6)
+        out[name] = {"us": round(ms * 1e3, 2), "roofline": round(floor / ms, 4)}
+
+    bf = lambda *sh: torch.randn(sh, device="cuda").to(torch.bfloat16)
+    i8 = lambda *sh: torch.randint(-127, 128, sh, dtype=torch.int8, device="cuda")
+    rnd = lambda *sh: torch.rand(sh, device="cuda") * 0.01 + 0.001
+    # products: prompts (8192 rows) and decoding (1, 4, 32 rows; more weight sets than L2 holds)
+    for N, K in ((6144, 2048), (2048, 2048), (16384, 2048), (2048, 8192)):
+        M = 8192
+        a, w, aq, wq, st, sc = bf(M, K), bf(N, K), i8(M, K), i8(N, K), rnd(M), rnd(N)
+        glu = N == 16384
+        note(f"prompt bf16 {M}x{N}x{K}" + (" gated gelu" if glu else ""), event_ms(torch, lambda i: F.linear_float(a, w, gelu_gate=glu), 20), 2.0 * M * N * K,
+             2.0 * (M * K + N * K + M * (N // 2 if glu else N)))
+        note(f"prompt int8 {M}x{N}x{K}", event_ms(torch, lambda i: F.pref_Linear_Layer_i8xi8(aq, st, wq, sc), 20), 2.0 * M * N * K, M * K + N * K + 4.0 * M * N, 2 * tf)
+        del a, aq
+        nset = max(2, int(300e6 // (N * K)) + 1)
+        ws, wqs = [bf(N, K) for _ in range(nset // 2 + 1)], [i8(N, K) for _ in range(nset)]
+        for B in (1, 4, 32):
+            a, aq, st = bf(B, K), i8(B, K), rnd(B)
+            note(f"decode bf16 {B}x{N}x{K}", graph_ms(torch, lambda i: F.linear_float(a, ws[i % len(ws)], gelu_gate=glu, out_f32=not glu)), 2.0 * B * N * K, 2.0 * N * K)
+            note(f"decode int8 {B}x{N}x{K}", graph_ms(torch, lambda i: F.dec_Linear_Layer_i8xi8(aq, st, wqs[i % nset], sc)), 2.0 * B * N * K, 1.0 * N * K, 2 * tf)
+        del ws, wqs
+    # norms of 32768 rows
+    x, y, g = torch.randn((32768, 2048), device="cuda"), torch.randn((32768, 2048), device="cuda"), torch.ones(2048, device="cuda")
+    note("norms 32768x2048 (x += norm(y), h = norm(x))", event_ms(torch, lambda i: F.sandwich_norm(x, 2048, 1e-5, y, g, None, g, torch.bfloat16), 20), 0, 32768 * 2048 * 14.0)
+    note("int8 Llama rmsnorm + quantiser 32768x2048", event_ms(torch, lambda i: F.pref_Layer_Norm(x, g, quant=True, want_y=False), 20), 0, 32768 * 2048 * 5.0)
+    # attention: prompts of 4 x 1024, decoding of 64 sequences at context 4096 (window 4096)
+    H, G, dk = 32, 8, 64
+    B, S = 4, 1024
+    mk = lambda B, S, W: F.WindowAttention(H, G, dk, dk, W, dk ** -0.5, 30.0, torch.randn((32, H)), W, torch.ones(H * dk, device="cuda"), torch.ones(G * dk, device="cuda"),
+                                           torch.arange(B * (S // 64 + 1), dtype=torch.int32, device="cuda").reshape(B, -1), B * (S // 64 + 1), S)
+    op = mk(B, S, S)
+    proj, ctx = bf(B * S, op.row), torch.zeros(B, dtype=torch.int32, device="cuda")
+    fl = 4.0 * B * H * dk * S * (S + 1) / 2
+    note(f"prompt attention {B}x{S} (norms, append, attention, gate)", event_ms(torch, lambda i: op(proj, ctx), 20), fl)
+    op.close()
+    q, k, v = i8(B, S, H, 64), i8(B, S, G, 64), i8(B, S, G, 64)
+    qs, ks, vs = rnd(B, S, H), rnd(B, S, G), rnd(B, S, G)
+    from flexllm_b200 import synthetic
+    cs, sn = (torch.from_numpy(t).cuda() for t in synthetic.rope_table(4200))
+    a_s = torch.full((H,), 0.05 / 255, device="cuda")
+    note(f"int8 Llama prompt attention {B}x{S}", event_ms(torch, lambda i: F.MHA_i8xi8_Prefilling(q, qs, k, ks, v, vs, cs, sn, a_s), 20), fl, 0, 2 * tf)
+    B, S = 64, 4096
+    op = mk(B, S, S)
+    proj, ctx = bf(B, op.row), torch.full((B,), S - 1, dtype=torch.int32, device="cuda")
+    note(f"decode attention {B} sequences, {S} keys", event_ms(torch, lambda i: op(proj, ctx), 20), 0, 2.0 * B * S * G * 2 * dk)
+    op.close()
+    cache = F.KVCache(1, B * (S // 64 + 1), G)
+    pt = torch.arange(B * (S // 64 + 1), dtype=torch.int32, device="cuda").reshape(B, -1)
+    q, k, v, qs, ks = i8(B, H, 64), i8(B, G, 64), i8(B, G, 64), rnd(B, H), rnd(B, G)
+    note(f"int8 Llama decode attention {B} sequences, {S} keys",
+         event_ms(torch, lambda i: F.MHA_i8xi8_Decoding(cache, 0, q, qs, k, ks, v, ks, cs, sn, a_s, pt, ctx, S), 20), 0, 1088.0 * B * S)
+    cache.close()
+    return out
+
+
+def pibidra_arm(args):
+    """python bench.py --design pibidra: prefill and decode throughput of the Pibidra family at a few sizes, the W8A8 Llama at
+    the size they share, and the kernels of both. One JSON line."""
+    import torch
+    import flexllm_b200 as F
+    from flexllm_b200 import synthetic
+    torch.cuda.set_device(0)
+    F.lib()
+    try:
+        peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
+    except Exception:
+        peaks = {}
+    hbm, tf = peaks.get("hbm_gbs") or 6650.0, peaks.get("bf16_tflops_sustained") or 1400.0
+    sampler = ClockSampler(0); sampler.start(); sampler.mark()
+    S, n_dec = 1024, 64
+    line = {"metric": "pibidra_prefill_decode", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic, random weights", "n_gpus": 1, "sizes": {},
+            "config": {"prefill_len": S, "decode_steps": n_dec, "window": "as listed", "l2": "weights exceed the 126 MB L2 (small: 0.4 GB); no flush"}}
+
+    def measure(m, vocab, B):
+        tok = torch.randint(0, vocab, (B, S), dtype=torch.int32).cuda()
+        pre = event_ms(torch, lambda i: m.prefill(tok), max(2, args.steps), warm=args.warmup)
+        m.prefill(tok); m.begin(2 * n_dec + 8)
+        m.decode(8, True); torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record(); m.decode(n_dec, True); e1.record(); torch.cuda.synchronize()
+        return pre, e0.elapsed_time(e1) / n_dec
+
+    for name, z in PIBIDRA_SIZES.items():
+        rows = {}
+        for B in (1, 4, 32):
+            m = pibidra_model(F, torch, z, B, S, S + 2 * n_dec + 16)
+            pre, dec = measure(m, z["vocab"], B)
+            m.close()
+            fl, by = pibidra_work(z, B, S, S + n_dec // 2)
+            rows["batch%d" % B] = {"prefill_ms": round(pre, 3), "prefill_tokens_per_s": round(B * S / pre * 1e3), "prefill_tflops_frac": round(fl / pre / 1e9 / tf, 3),
+                                   "decode_ms": round(dec, 4), "decode_tokens_per_s": round(B / dec * 1e3), "decode_hbm_frac": round(by / dec / 1e6 / hbm, 3)}
+        line["sizes"][name] = dict(shape=z, **rows)
+    rows = {}
+    for B in (1, 4, 32):
+        m = F.Model(max_batch=B, max_prefill=S, max_ctx=S + 2 * n_dec + 16, **CFG)
+        synthetic.load_random_weights(m, max_ctx=S + 2 * n_dec + 16, seed=0, **CFG)
+        pre, dec = measure(m, CFG["vocab"], B)
+        m.close()
+        rows["batch%d" % B] = {"prefill_ms": round(pre, 3), "prefill_tokens_per_s": round(B * S / pre * 1e3), "decode_ms": round(dec, 4),
+                               "decode_tokens_per_s": round(B / dec * 1e3),
+                               "prefill_tops_frac": round(prefill_ops(B) / pre / 1e9 / (2 * tf), 3), "decode_hbm_frac": round(decode_step_bytes(B) / dec / 1e6 / hbm, 3)}
+    line["int8_llama_same_size"] = rows
+    line["value"] = line["sizes"]["llama1b"]["batch32"]["decode_tokens_per_s"]
+    if not args.no_extras:
+        line["kernels"] = pibidra_kernels(F, torch, peaks)
+    line["clocks"] = sampler.stop()
+    print(json.dumps(line))
 
 
 def gpu_arm(args):
@@ -821,15 +1020,20 @@ def main():
                     help="N > 1: headline partition - tensor parallel over the N GPUs with a fixed total batch of 32 (default: the "
                          "partition the workload names), or independent batch-parallel replicas; the other one is reported under "
                          "other_partition")
+    ap.add_argument("--design", default="llama", choices=["llama", "pibidra"],
+                    help="pibidra: throughput of that model family at a few sizes beside the W8A8 Llama (one GPU) instead of the headline workload")
     ap.add_argument("--decode-len", type=int, default=NEW)
     ap.add_argument("--no-extras", action="store_true", help="skip roofline kernel timing and the CPU baseline")
     ap.add_argument("--micro", default=None, help="run one kernel on a small case and exit (attn_prefill, attn_prefill_online, gemm_prefill, "
-                                                  "gemm_prefill_k8192, decode_linear, gemv_b1, decode_attention, swiglu_fht, rmsnorm_prefill, prefill_small, decode_step)")
+                                                  "gemm_prefill_k8192, decode_linear, gemv_b1, decode_attention, swiglu_fht, rmsnorm_prefill, prefill_small, decode_step, pibidra_prefill, pibidra_decode)")
     args = ap.parse_args()
     globals()["NEW"] = args.decode_len
     args.warmup = max(args.warmup, 0)
     if args.micro:
         micro(args)
+        return
+    if args.design == "pibidra":
+        pibidra_arm(args)
         return
     if args.impl == "reference":
         if env_int("RANK", 0) == 0:

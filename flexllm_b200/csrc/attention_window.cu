@@ -6,7 +6,8 @@
 // window), so that a masked key costs nothing extra. Scores, weights and sums are fp32.
 //
 // Cache pages hold 64 tokens, K [page][G][64][dkp] and V transposed [page][G][dv][64] (as the int8 cache does).
-//   one token per sequence : attn_row_kernel<FUSED>: norms, append and attention in one launch, keys split over CTAs
+//   one token per sequence : attn_decode_mma_kernel (bf16), else attn_row_kernel<FUSED>: norms, append and attention in one
+//                            launch, keys split over CTAs
 //   prompts, bf16          : attn_prepare_kernel, then attn_window_prefill_kernel on tcgen05
 //   prompts, otherwise     : attn_prepare_kernel, then attn_row_kernel row by row
 // The sink is a score of 0, so max(0, largest score) is a valid softmax shift; without a sink the running maximum is.
@@ -26,6 +27,7 @@ namespace {
 constexpr int PG = 64;                     // tokens per page
 constexpr int TILE_PAGES = 4;              // pages per key tile of the row kernel
 constexpr int TILE_KEYS = TILE_PAGES * PG;
+constexpr long kDecodeCtas = 1776;         // CTAs the decode form aims at: four waves of three per SM
 
 // Start position of sequence b; a value that would leave the page-table row is clamped and reported.
 __device__ __forceinline__ int start_pos(const AttnCall& c, int b, int* error_flag) {
@@ -35,6 +37,37 @@ __device__ __forceinline__ int start_pos(const AttnCall& c, int b, int* error_fl
         pos = pos < 0 ? 0 : c.max_pos - (c.Sc - 1);
     }
     return pos;
+}
+
+// This thread's share (NT threads) of the sum of squares of n elements at a 16-byte aligned address.
+template <int NT, class T> __device__ __forceinline__ float share_sumsq(const T* p, int n, int tid) {
+    float s = 0.0f;
+    const int nv = n >> 3;
+    for (int i = tid; i < nv; i += NT) {
+        float f[8];
+        load8(p + 8 * i, f);
+#pragma unroll
+        for (int e = 0; e < 8; e++) s = __fmaf_rn(f[e], f[e], s);
+    }
+    for (int i = (nv << 3) + tid; i < n; i += NT) { const float v = to_f(p[i]); s = __fmaf_rn(v, v, s); }
+    return s;
+}
+// Normed elements e0 .. e0+7 of a head whose first element is j0 of the projection at src (j0 + e0 is 8-aligned when dk is a
+// multiple of 8); zero from dk on.
+template <class T> __device__ __forceinline__ void normed8(const T* src, const float* gain, int j0, int e0, int dk, float r, float (&f)[8]) {
+    if ((dk & 7) == 0) {
+        load8(src + j0 + e0, f);
+        const float4 a = load4(gain + j0 + e0), b = load4(gain + j0 + e0 + 4);
+        f[0] = (f[0] * r) * a.x; f[1] = (f[1] * r) * a.y; f[2] = (f[2] * r) * a.z; f[3] = (f[3] * r) * a.w;
+        f[4] = (f[4] * r) * b.x; f[5] = (f[5] * r) * b.y; f[6] = (f[6] * r) * b.z; f[7] = (f[7] * r) * b.w;
+    } else {
+#pragma unroll
+        for (int e = 0; e < 8; e++) f[e] = e0 + e < dk ? (to_f(src[j0 + e0 + e]) * r) * gain[j0 + e0 + e] : 0.0f;
+    }
+}
+template <class T> __device__ __forceinline__ void store8(T* p, const float (&f)[8]) {
+    store4(p, make_float4(f[0], f[1], f[2], f[3]));
+    store4(p + 4, make_float4(f[4], f[5], f[6], f[7]));
 }
 
 // ---------------------------------------------------------------------------------------------------------------
@@ -52,21 +85,23 @@ __global__ void __launch_bounds__(256) attn_prepare_kernel(const AttnCall c, int
         const int pos = start_pos(c, b, error_flag) + m % c.Sc;
         const T* src = (const T*)c.proj + (long)m * s.ld;
         const int nq = s.H * s.dk, nk = s.G * s.dk;
-        float sq = 0.0f, sk = 0.0f;
-        for (int i = tid; i < nq; i += 256) { const float v = to_f(src[s.q_off + i]); sq = __fmaf_rn(v, v, sq); }
-        for (int i = tid; i < nk; i += 256) { const float v = to_f(src[s.k_off + i]); sk = __fmaf_rn(v, v, sk); }
-        const float2 ss = block_sum2<256>(sq, sk, red);
+        const float2 ss = block_sum2<256>(share_sumsq<256>(src + s.q_off, nq, tid), share_sumsq<256>(src + s.k_off, nk, tid), red);
         const float rq = 1.0f / sqrtf(ss.x / (float)nq + c.eps), rk = 1.0f / sqrtf(ss.y / (float)nk + c.eps);
         T* q = (T*)c.q + (long)m * s.H * s.dkp;
-        for (int i = tid; i < s.H * s.dkp; i += 256) {
-            const int h = i / s.dkp, e = i - h * s.dkp, j = h * s.dk + e;
-            q[i] = from_f<T>(e < s.dk ? (to_f(src[s.q_off + j]) * rq) * c.q_gain[j] : 0.0f);
+        const int nv = s.dkp >> 3;                                  // 8-element blocks per head
+        for (int i = tid; i < s.H * nv; i += 256) {
+            const int h = i / nv, e0 = (i - h * nv) * 8;
+            float f[8];
+            normed8(src + s.q_off, c.q_gain, h * s.dk, e0, s.dk, rq, f);
+            store8(q + (long)i * 8, f);
         }
         const long page = c.page_table[(long)b * c.max_pages + pos / PG];
         T* kp = (T*)c.k_pool + (page * s.G * PG + (pos & (PG - 1))) * s.dkp;
-        for (int i = tid; i < s.G * s.dkp; i += 256) {
-            const int g = i / s.dkp, e = i - g * s.dkp, j = g * s.dk + e;
-            kp[(long)g * PG * s.dkp + e] = from_f<T>(e < s.dk ? (to_f(src[s.k_off + j]) * rk) * c.k_gain[j] : 0.0f);
+        for (int i = tid; i < s.G * nv; i += 256) {
+            const int g = i / nv, e0 = (i - g * nv) * 8;
+            float f[8];
+            normed8(src + s.k_off, c.k_gain, g * s.dk, e0, s.dk, rk, f);
+            store8(kp + (long)g * PG * s.dkp + e0, f);
         }
         return;
     }
@@ -131,10 +166,7 @@ __global__ void __launch_bounds__(256) attn_row_kernel(const AttnCall c, int L, 
     const long kh = (long)PG * s.dkp, vh = (long)PG * s.dv;          // one head of a page
     if (FUSED) {
         const int nq = s.H * s.dk, nk = s.G * s.dk;
-        float sq = 0.0f, sk = 0.0f;
-        for (int i = tid; i < nq; i += 256) { const float v = to_f(prow[s.q_off + i]); sq = __fmaf_rn(v, v, sq); }
-        for (int i = tid; i < nk; i += 256) { const float v = to_f(prow[s.k_off + i]); sk = __fmaf_rn(v, v, sk); }
-        const float2 ss = block_sum2<256>(sq, sk, red);
+        const float2 ss = block_sum2<256>(share_sumsq<256>(prow + s.q_off, nq, tid), share_sumsq<256>(prow + s.k_off, nk, tid), red);
         const float rq = 1.0f / sqrtf(ss.x / (float)nq + c.eps), rk = 1.0f / sqrtf(ss.y / (float)nk + c.eps);
         for (int i = tid; i < R * s.dkp; i += 256) {
             const int r = i / s.dkp, e = i - r * s.dkp, j = (g * R + r) * s.dk + e;
@@ -333,6 +365,202 @@ __global__ void __launch_bounds__(256) attn_row_kernel(const AttnCall c, int L, 
 }
 
 // ---------------------------------------------------------------------------------------------------------------
+// Decoding, bf16, up to 8 query heads per key/value head: the fused form of the row kernel with warp-level bf16 MMAs.
+// A CTA takes one (sequence, key/value head) and a share of its key tiles of 128 keys (two pages):
+//   scores: warp w has keys 16 w .. 16 w + 15 of the tile on the 16-row side, the query heads on the 8-column side
+//   values: dimensions on the 16-row side (V^T page rows), heads on the 8-column side, the tile's keys as the inner index,
+//           cut into KS slices when there are fewer than 8 blocks of 16 dimensions (MPW blocks per warp)
+// Every operand row is read with 16-byte loads: lane % 4 holds elements 8 c .. 8 c + 7 of each 32, i.e. the inner index is
+// permuted, the same way in both operands. K of the next tile and V of this one are in flight during the arithmetic. The
+// scores are bounded (see the prompt kernel), so exp(s) needs no running maximum and splits just add up.
+struct DecodeArgs { AttnCall c; float a2, b2, shift2; int tiles_max; int* error_flag; };
+constexpr int DT_KEYS = 128, DT_PS = DT_KEYS + 8;      // keys per tile, row pitch of the weights in shared memory
+
+__host__ __device__ inline size_t decode_smem(int dkp, int dv, int KS, int tiles_max) {
+    // page ids, q [8][dkp + 8], weights [2][8][DT_PS], sums [8][8], outputs [KS][8][dv]
+    return (size_t)((2 * tiles_max + 3) & ~3) * 4 + 8 * (size_t)(dkp + 8) * 2 + 2 * 8 * DT_PS * 2 + 64 * 4 + (size_t)KS * 8 * dv * 4;
+}
+
+template <int DKC, int KS, int MPW>
+__global__ void __launch_bounds__(256, DKC == 8 || MPW == 2 ? 1 : 2) attn_decode_mma_kernel(const __grid_constant__ DecodeArgs a) {
+    constexpr int MTP = MPW == 2 ? 8 : 8 / KS;             // warps along the dimensions
+    constexpr int NCH = 4 / KS;                            // 32-key chunks of a warp's slice
+    extern __shared__ __align__(16) uint8_t raw[];
+    __shared__ float red[16];
+    __shared__ int last_sm;
+    const AttnCall& c = a.c;
+    const AttnShape& s = c.s;
+    const int R = s.H / s.G;
+    int* pt_sm = reinterpret_cast<int*>(raw);
+    bf16* q_sm = reinterpret_cast<bf16*>(raw + (size_t)((2 * a.tiles_max + 3) & ~3) * 4);
+    bf16* p_sm = q_sm + 8 * (s.dkp + 8);
+    float* l_sm = reinterpret_cast<float*>(p_sm + 2 * 8 * DT_PS);
+    float* o_sm = l_sm + 64;
+    const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lr = lane >> 2, lc = lane & 3;
+    const int split = blockIdx.x, n_split = gridDim.x, g = blockIdx.y, b = blockIdx.z;
+    pdl_sync();
+    const int pos = start_pos(c, b, a.error_flag);
+    const int lo = max(0, pos - s.window + 1);
+    const int p_lo = lo / PG, n_pg = pos / PG - p_lo + 1, n_tiles = (n_pg + 1) / 2;
+    const int t_beg = (int)((long)split * n_tiles / n_split), t_end = (int)((long)(split + 1) * n_tiles / n_split);
+    const int32_t* pt = c.page_table + (long)b * c.max_pages + p_lo;
+    const bf16* prow = (const bf16*)c.proj + (long)b * s.ld;
+    const long kh = (long)PG * s.dkp, vh = (long)PG * s.dv;
+    for (int i = tid; i < 2 * (t_end - t_beg); i += 256) pt_sm[i] = 2 * t_beg + i < n_pg ? pt[2 * t_beg + i] : -1;
+    const int nq = s.H * s.dk, nk = s.G * s.dk, nv = s.dkp >> 3;
+    const float2 ss = block_sum2<256>(share_sumsq<256>(prow + s.q_off, nq, tid), share_sumsq<256>(prow + s.k_off, nk, tid), red);
+    const float rq = 1.0f / sqrtf(ss.x / (float)nq + c.eps), rk = 1.0f / sqrtf(ss.y / (float)nk + c.eps);
+    for (int i = tid; i < 8 * nv; i += 256) {
+        const int r = i / nv, e0 = (i - r * nv) * 8;
+        float f[8] = {0, 0, 0, 0, 0, 0, 0, 0};
+        if (r < R) normed8(prow + s.q_off, c.q_gain, (g * R + r) * s.dk, e0, s.dk, rq, f);
+        store8(q_sm + r * (s.dkp + 8) + e0, f);
+    }
+    if (split == n_split - 1) {
+        const long page = pt[n_pg - 1];
+        const int slot = pos & (PG - 1);
+        bf16* kp = (bf16*)c.k_pool + (page * s.G + g) * kh + (long)slot * s.dkp;
+        for (int i = tid; i < nv; i += 256) {
+            float f[8];
+            normed8(prow + s.k_off, c.k_gain, g * s.dk, i * 8, s.dk, rk, f);
+            store8(kp + i * 8, f);
+        }
+        bf16* vp = (bf16*)c.v_pool + (page * s.G + g) * vh + slot;
+        for (int d = tid; d < s.dv; d += 256) vp[(long)d * PG] = prow[s.v_off + g * s.dv + d];
+    }
+    __syncthreads();
+
+    uint4 qb[DKC];
+#pragma unroll
+    for (int ch = 0; ch < DKC; ch++) {
+        const int e = ch * 32 + lc * 8;
+        qb[ch] = e < s.dkp ? *reinterpret_cast<const uint4*>(q_sm + lr * (s.dkp + 8) + e) : make_uint4(0, 0, 0, 0);
+    }
+    uint4 kr[DKC][2];
+    auto load_k = [&](int t) {
+        const int page = pt_sm[2 * (t - t_beg) + (warp >> 2)];
+        const bf16* kp = (const bf16*)c.k_pool + ((long)page * s.G + g) * kh + (long)((warp & 3) * 16 + lr) * s.dkp + lc * 8;
+#pragma unroll
+        for (int ch = 0; ch < DKC; ch++) {
+            const bool in = page >= 0 && ch * 32 + lc * 8 < s.dkp;
+#pragma unroll
+            for (int h = 0; h < 2; h++)
+                kr[ch][h] = in ? *reinterpret_cast<const uint4*>(kp + (long)h * 8 * s.dkp + ch * 32) : make_uint4(0, 0, 0, 0);
+        }
+    };
+    const int mt = warp % MTP, slice = warp / MTP;
+    const bool pv_on = slice < KS;
+    float acc[MPW][4] = {};
+    float lsum[2] = {0.0f, 0.0f};
+    const float* bias_g = c.bias + (long)g * (2 * kBiasPad + s.window) * R;
+    const float badd = s.softcap * kLog2e - a.shift2;
+    if (t_beg < t_end) load_k(t_beg);
+    for (int t = t_beg; t < t_end; t++) {
+        uint4 vr[MPW][NCH][2];
+        if (pv_on) {
+#pragma unroll
+            for (int ch = 0; ch < NCH; ch++) {
+                const int key = slice * (DT_KEYS / KS) + ch * 32;          // of the tile
+                const int page = pt_sm[2 * (t - t_beg) + (key >> 6)];
+                const bf16* vp = (const bf16*)c.v_pool + ((long)page * s.G + g) * vh + (key & 63) + lc * 8;
+#pragma unroll
+                for (int m = 0; m < MPW; m++)
+#pragma unroll
+                    for (int h = 0; h < 2; h++) {
+                        const int d = (mt + 8 * m) * 16 + lr + 8 * h;
+                        vr[m][ch][h] = page >= 0 && d < s.dv ? *reinterpret_cast<const uint4*>(vp + (long)d * PG) : make_uint4(0, 0, 0, 0);
+                    }
+            }
+        }
+        // biases of this thread's two keys and two heads (-inf: masked, or no such head)
+        const int d0 = pos - ((p_lo + 2 * t) * PG + warp * 16 + lr);
+        float bi[2][2];
+#pragma unroll
+        for (int h = 0; h < 2; h++)
+#pragma unroll
+            for (int u = 0; u < 2; u++)
+                bi[h][u] = lc * 2 + u < R ? bias_g[(long)(d0 - 8 * h + kBiasPad) * R + lc * 2 + u] : -INFINITY;
+        float sc[4] = {0.0f, 0.0f, 0.0f, 0.0f};
+#pragma unroll
+        for (int ch = 0; ch < DKC; ch++) {
+            mma_bf16(sc, kr[ch][0].x, kr[ch][1].x, kr[ch][0].y, kr[ch][1].y, qb[ch].x, qb[ch].y);
+            mma_bf16(sc, kr[ch][0].z, kr[ch][1].z, kr[ch][0].w, kr[ch][1].w, qb[ch].z, qb[ch].w);
+        }
+        if (t + 1 < t_end) load_k(t + 1);
+        bf16* pb = p_sm + (t & 1) * 8 * DT_PS + warp * 16 + lr;
+#pragma unroll
+        for (int h = 0; h < 2; h++)
+#pragma unroll
+            for (int u = 0; u < 2; u++) {
+                const float s2 = __fmaf_rn(a.b2, rcp_fast(1.0f + ex2_fast(sc[2 * h + u] * a.a2)), __fmaf_rn(bi[h][u], kLog2e, badd));
+                const float p = ex2_fast(s2);
+                lsum[u] += p;
+                pb[(lc * 2 + u) * DT_PS + 8 * h] = __float2bfloat16_rn(p);
+            }
+        __syncthreads();
+        if (pv_on) {
+            const bf16* pr = p_sm + (t & 1) * 8 * DT_PS + lr * DT_PS + slice * (DT_KEYS / KS) + lc * 8;
+#pragma unroll
+            for (int ch = 0; ch < NCH; ch++) {
+                const uint4 pw = *reinterpret_cast<const uint4*>(pr + ch * 32);
+#pragma unroll
+                for (int m = 0; m < MPW; m++) {
+                    mma_bf16(acc[m], vr[m][ch][0].x, vr[m][ch][1].x, vr[m][ch][0].y, vr[m][ch][1].y, pw.x, pw.y);
+                    mma_bf16(acc[m], vr[m][ch][0].z, vr[m][ch][1].z, vr[m][ch][0].w, vr[m][ch][1].w, pw.z, pw.w);
+                }
+            }
+        }
+    }
+    // sums over the warps' keys, outputs over the slices
+#pragma unroll
+    for (int o = 4; o < 32; o <<= 1)
+#pragma unroll
+        for (int u = 0; u < 2; u++) lsum[u] += __shfl_xor_sync(0xffffffffu, lsum[u], o);
+    if (lr == 0) { l_sm[warp * 8 + lc * 2] = lsum[0]; l_sm[warp * 8 + lc * 2 + 1] = lsum[1]; }
+    if (pv_on)
+#pragma unroll
+        for (int m = 0; m < MPW; m++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                const int d = (mt + 8 * m) * 16 + lr + 8 * (i >> 1);
+                if (d < s.dv) o_sm[((long)slice * 8 + lc * 2 + (i & 1)) * s.dv + d] = acc[m][i];
+            }
+    __syncthreads();
+    auto head_l = [&](int r) { float v = 0.0f; for (int w = 0; w < 8; w++) v += l_sm[w * 8 + r]; return v; };
+    auto head_o = [&](int r, int d) { float v = 0.0f; for (int k = 0; k < KS; k++) v += o_sm[((long)k * 8 + r) * s.dv + d]; return v; };
+    const float sink = s.sink ? ex2_fast(-a.shift2) : 0.0f;
+    const long stride = (long)R * (s.dv + 1);
+    float* part = c.ws + ((long)b * s.G + g) * n_split * stride;
+    if (n_split > 1) {
+        float* mine = part + split * stride;
+        for (int i = tid; i < R; i += 256) mine[i] = head_l(i);
+        for (int i = tid; i < R * s.dv; i += 256) mine[R + i] = head_o(i / s.dv, i % s.dv);
+        __threadfence();
+        __syncthreads();
+        int* cnt = c.counters + (long)b * s.G + g;
+        if (tid == 0) last_sm = atomicAdd(cnt, 1) == n_split - 1;
+        __syncthreads();
+        if (!last_sm) return;
+        __threadfence();
+        if (tid == 0) *cnt = 0;
+    }
+    bf16* out = (bf16*)c.out + (long)b * c.ldo + (long)g * R * s.dv;
+    for (int i = tid; i < R * s.dv; i += 256) {
+        const int r = i / s.dv;
+        float l = sink, v = 0.0f;
+        if (n_split > 1) {
+#pragma unroll 4
+            for (int k = 0; k < n_split; k++) { l += __ldcg(part + k * stride + r); v += __ldcg(part + k * stride + R + i); }
+        } else {
+            l += head_l(r); v = head_o(r, i - r * s.dv);
+        }
+        v /= l;
+        if (s.g_off >= 0) v *= sigmoid_f<true>(to_f(prow[s.g_off + (long)g * R * s.dv + i]));
+        out[i] = __float2bfloat16_rn(v);
+    }
+}
+
+// ---------------------------------------------------------------------------------------------------------------
 // Prompt attention on the tensor cores. A CTA takes TQ = 128 / R consecutive positions x the R query heads of one key/value
 // head (row = position * R + head: the heads of a group share the K and V tiles, and a small window wastes few keys), and
 // walks the key pages its window reaches. The scores are bounded by softcap + max|bias|, so the softmax shift is a constant
@@ -474,19 +702,29 @@ __global__ void __launch_bounds__(192, 2) attn_window_prefill_kernel(const __gri
         // biases of key tile j, in log2 units with the constants of the score formula folded in; masked keys stay -inf.
         // Entry (t + 63 - key) * R + r belongs to position t, head r: consecutive rows read consecutive words.
         const float badd = s.softcap * kLog2e - a.shift2;
-        auto stage_bias = [&](int j) {
+        // The values of the next tile travel through registers, so that their latency hides behind this tile's arithmetic.
+        constexpr int NB = 9;                                            // (TQ + 63) * R <= 1136 for R <= 16
+        float nb[NB];
+        auto fetch_bias = [&](int j) {
             const int dmin = q0 - (pg_lo + j) * PG - 63;                 // distance of the first entry
             const float* src = bias_g + (long)(dmin + kBiasPad) * R;
-            float* dst = bias_sm + (j & 1) * bias_stride;
-            for (int i = rr; i < n_bias; i += 128) dst[i] = __fmaf_rn(src[i], kLog2e, badd);
+#pragma unroll
+            for (int i = 0; i < NB; i++) nb[i] = rr + 128 * i < n_bias ? src[rr + 128 * i] : 0.0f;
         };
+        auto stage_bias = [&](int j) {
+            float* dst = bias_sm + (j & 1) * bias_stride;
+#pragma unroll
+            for (int i = 0; i < NB; i++)
+                if (rr + 128 * i < n_bias) dst[rr + 128 * i] = __fmaf_rn(nb[i], kLog2e, badd);
+        };
+        fetch_bias(0);
         stage_bias(0);
         float l = 0.0f;
         bool ok = true;
         for (int j = 0; j < n_kt; j++) {
             const int sb = j & 1, pb = a.p_bufs == 2 ? sb : 0;
             named_sync<1, 128>();                                        // tile j's biases are in place; j - 1's reads are over
-            if (j + 1 < n_kt) stage_bias(j + 1);
+            if (j + 1 < n_kt) fetch_bias(j + 1);
             const float* bs = bias_sm + sb * bias_stride + rr + 63 * R;
             if (ok && !wait_bar(bar_sf + 8 * sb, (uint32_t)((j >> 1) & 1))) ok = false;
             if (ok && !wait_bar(bar_pe + 8 * pb, (uint32_t)((a.p_bufs == 2 ? j >> 1 : j) & 1) ^ 1u)) ok = false;
@@ -494,33 +732,43 @@ __global__ void __launch_bounds__(192, 2) attn_window_prefill_kernel(const __gri
             tc_fence_after();
             uint8_t* prow = base_ptr + o.p + pb * 16384 + rr * 128;
             const uint32_t tS = tmem_base + sb * PF_S_COLS + lane_addr;
-#pragma unroll
-            for (int cc = 0; cc < 4; cc++) {
-                uint32_t v[16];
-                tmem_ld_32x16(tS + cc * 16, v);
-                tmem_ld_wait();
+            auto chunk = [&](const uint32_t (&v)[16], int cc) {
                 uint32_t pk[8];
 #pragma unroll
                 for (int i = 0; i < 16; i += 2) {
-                    float p[2];
-#pragma unroll
-                    for (int u = 0; u < 2; u++) {
-                        const float bi = bs[-(cc * 16 + i + u) * R];
-                        const float x = __uint_as_float(v[i + u]) * a.a2;
-                        // softcap * tanh(z) = softcap - 2 softcap / (1 + e^(2 z)); all in log2 units
-                        const float s2 = __fmaf_rn(a.b2, rcp_fast(1.0f + ex2_fast(x)), bi);
-                        p[u] = ex2_fast(s2);
-                    }
-                    l += p[0] + p[1];
-                    pk[i >> 1] = bf_pack(p[0], p[1]);
+                    // softcap * tanh(z) = softcap - 2 softcap / (1 + e^(2 z)), in log2 units; the two reciprocals of a pair
+                    // come from one: 1/x = y / (x y). The clamp (tanh is 1 there) keeps the product finite.
+                    const float e0 = 1.0f + ex2_fast(fminf(__uint_as_float(v[i]) * a.a2, 60.0f));
+                    const float e1 = 1.0f + ex2_fast(fminf(__uint_as_float(v[i + 1]) * a.a2, 60.0f));
+                    const float rc = rcp_fast(e0 * e1) * a.b2;
+                    const float p0 = ex2_fast(__fmaf_rn(rc, e1, bs[-(cc * 16 + i) * R]));
+                    const float p1 = ex2_fast(__fmaf_rn(rc, e0, bs[-(cc * 16 + i + 1) * R]));
+                    l += p0 + p1;
+                    pk[i >> 1] = bf_pack(p0, p1);
                 }
                 *reinterpret_cast<uint4*>(prow + (((2 * cc) ^ (rr & 7)) << 4)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
                 *reinterpret_cast<uint4*>(prow + (((2 * cc + 1) ^ (rr & 7)) << 4)) = make_uint4(pk[4], pk[5], pk[6], pk[7]);
-            }
-            fence_proxy_async_smem();
+            };
+            uint32_t va[16], vb[16];
+            tmem_ld_32x16(tS, va);
+            tmem_ld_wait();
+            tmem_ld_32x16(tS + 16, vb);
+            chunk(va, 0);
+            tmem_ld_wait();
+            tmem_ld_32x16(tS + 32, va);
+            chunk(vb, 1);
+            tmem_ld_wait();
+            tmem_ld_32x16(tS + 48, vb);
+            chunk(va, 2);
+            tmem_ld_wait();
             tc_fence_before();
             __syncwarp();
-            if (lane == 0) { mbar_arrive(bar_pf + 8 * pb); mbar_arrive(bar_se + 8 * sb); }
+            if (lane == 0) mbar_arrive(bar_se + 8 * sb);                 // the scores are in registers: the next product may start
+            chunk(vb, 3);
+            fence_proxy_async_smem();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(bar_pf + 8 * pb);
+            if (j + 1 < n_kt) stage_bias(j + 1);
         }
         if (ok) ok = wait_bar(bar_o, 0);
         if (ok) {
@@ -611,19 +859,62 @@ template <class T, bool FUSED> int run_row(const AttnCall& c, cudaStream_t st) {
 #undef FLEXLLM_ROW
 }
 
+// Constants of the score formula in log2 units for the kernels that rely on bounded scores; false when the bound is missing
+// (no softcap) or so wide that sums could vanish below the smallest floats.
+bool bounded_scores(const AttnCall& c, float* a2, float* b2, float* shift2) {
+    const AttnShape& s = c.s;
+    if (s.softcap <= 0.0f) return false;
+    const float bound2 = (s.softcap + c.bias_max_abs) * kLog2e;
+    *shift2 = bound2 > 100.0f ? bound2 - 100.0f : 0.0f;
+    *a2 = s.scale / s.softcap * 2.0f * kLog2e; *b2 = -2.0f * s.softcap * kLog2e;
+    return *shift2 <= (s.sink ? 80.0f : 20.0f);
+}
+
+template <int DKC, int KS, int MPW> int launch_decode(DecodeArgs& a, int splits, cudaStream_t st) {
+    const AttnCall& c = a.c;
+    const size_t smem = decode_smem(c.s.dkp, c.s.dv, KS, a.tiles_max);
+    auto kern = attn_decode_mma_kernel<DKC, KS, MPW>;
+    if (smem > 200 * 1024) return FLEXLLM_ENOTSUP;
+    TRY_RC(set_smem((const void*)kern, smem));
+    launch_k(kern, dim3(splits, c.s.G, c.B), dim3(256), smem, st, a);
+    return launch_status();
+}
+template <int DKC> int pick_decode(DecodeArgs& a, int splits, cudaStream_t st) {
+    const int dv = a.c.s.dv;
+    if (dv <= 32) return launch_decode<DKC, 4, 1>(a, splits, st);
+    if (dv <= 64) return launch_decode<DKC, 2, 1>(a, splits, st);
+    if (dv <= 128) return launch_decode<DKC, 1, 1>(a, splits, st);
+    return launch_decode<DKC, 1, 2>(a, splits, st);
+}
+// FLEXLLM_ENOTSUP: the row kernel takes the call.
+int run_decode(const AttnCall& c, cudaStream_t st) {
+    const AttnShape& s = c.s;
+    DecodeArgs a;
+    a.c = c; a.error_flag = device_error_flag();
+    if (s.H / s.G > 8 || s.dkp > 256 || s.dv > 256 || c.B > 65535 || !bounded_scores(c, &a.a2, &a.b2, &a.shift2)) return FLEXLLM_ENOTSUP;
+    const int reach = s.window < c.max_pos + 1 ? s.window : c.max_pos + 1;
+    const int tiles = (reach + 2 * PG - 2) / PG / 2 + 1;
+    const long ctas = (long)c.B * s.G;
+    long splits = (kDecodeCtas + ctas - 1) / ctas;
+    if (splits > tiles / 2) splits = tiles / 2;
+    const long per = ctas * (s.H / s.G) * (s.dv + 1);
+    if (splits * per > (long)c.ws_floats) splits = (long)c.ws_floats / per;
+    if (splits < 1 || ctas > c.n_counters || !c.ws) splits = 1;
+    a.tiles_max = (int)((tiles + splits - 1) / splits + 1);
+    if (s.dkp <= 64) return pick_decode<2>(a, (int)splits, st);
+    if (s.dkp <= 128) return pick_decode<4>(a, (int)splits, st);
+    return pick_decode<8>(a, (int)splits, st);
+}
+
 // Whether the tensor-core kernel covers the call (bf16 only).
 bool prefill_covers(const AttnCall& c, PrefillArgs* a) {
     const AttnShape& s = c.s;
     a->c = c;
     a->R = s.H / s.G; a->TQ = a->R <= 16 ? 128 / a->R : 0;
     if (a->R > 16 || s.dkp > 256 || s.dv > 256) return false;
-    if (s.softcap <= 0.0f) return false;                                  // no bound on the scores: running maximum needed
-    const float bound2 = (s.softcap + c.bias_max_abs) * kLog2e;
-    a->shift2 = bound2 > 100.0f ? bound2 - 100.0f : 0.0f;
-    if (a->shift2 > (s.sink ? 80.0f : 20.0f)) return false;               // sums could vanish below the smallest floats
+    if (!bounded_scores(c, &a->a2, &a->b2, &a->shift2)) return false;
     a->kc = (s.dkp + 63) / 64; a->vrows = (s.dv + 15) / 16 * 16;
     a->n_qt = (c.Sc + a->TQ - 1) / a->TQ;
-    a->a2 = s.scale / s.softcap * 2.0f * kLog2e; a->b2 = -2.0f * s.softcap * kLog2e;
     a->o_col = 2 * PF_S_COLS;
     int cols = 32;
     while (cols < a->o_col + a->vrows) cols *= 2;
@@ -650,6 +941,8 @@ int run_prefill(const PrefillArgs& a, cudaStream_t st) {
     return launch_status();
 }
 
+template <class T> int run_tensor_decode(const AttnCall&, cudaStream_t) { return FLEXLLM_ENOTSUP; }
+template <> int run_tensor_decode<bf16>(const AttnCall& c, cudaStream_t st) { return run_decode(c, st); }
 template <class T> bool run_tensor_prefill(const AttnCall&, cudaStream_t, int*) { return false; }
 template <> bool run_tensor_prefill<bf16>(const AttnCall& c, cudaStream_t st, int* rc) {
     PrefillArgs a;
@@ -670,10 +963,8 @@ int check_call(const AttnCall& c) {
 }  // namespace
 
 size_t attn_window_ws_floats(int max_batch, int G, int R, int dv) {
-    // splits * CTAs never exceeds twice the SM count plus one CTA row
     const size_t ctas = (size_t)max_batch * G;
-    const size_t n = 2u * 160u > ctas ? 2u * 160u : ctas;
-    return n * (size_t)R * (dv + 2);
+    return ((size_t)kDecodeCtas + ctas) * R * (dv + 2);
 }
 
 void attn_layout(AttnShape* s, bool gate) {
@@ -709,7 +1000,10 @@ void attn_bias_table(const AttnShape& s, const float* table, int rows, int bias_
 
 template <class T> int attn_window(const AttnCall& c, cudaStream_t st) {
     TRY_RC(check_call(c));
-    if (c.Sc == 1) return run_row<T, true>(c, st);
+    if (c.Sc == 1) {
+        const int rc = run_tensor_decode<T>(c, st);
+        return rc == FLEXLLM_ENOTSUP ? run_row<T, true>(c, st) : rc;
+    }
     FLEXLLM_REQUIRE(c.q);
     const int v_pages = (c.Sc + PG - 2) / PG + 1;
     launch_k(attn_prepare_kernel<T>, dim3(c.B * c.Sc + c.B * c.s.G * v_pages), dim3(256), 0, st, c, v_pages, device_error_flag());

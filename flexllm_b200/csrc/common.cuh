@@ -57,6 +57,23 @@ inline void launch_k(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t smem,
     cudaLaunchKernelEx(&cfg, kern, KArgs(args)...);
 }
 
+// The same with the grid's CTAs in clusters of `cluster` along x.
+template <class... KArgs, class... Args>
+inline void launch_cluster(void (*kern)(KArgs...), dim3 grid, dim3 block, int cluster, size_t smem, cudaStream_t st, Args... args) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = grid; cfg.blockDim = block; cfg.dynamicSmemBytes = smem; cfg.stream = st;
+    cudaLaunchAttribute at[2];
+    at[0].id = cudaLaunchAttributeClusterDimension;
+    at[0].val.clusterDim.x = cluster; at[0].val.clusterDim.y = 1; at[0].val.clusterDim.z = 1;
+    cfg.attrs = at; cfg.numAttrs = 1;
+    if (g_pdl) {
+        at[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        at[1].val.programmaticStreamSerializationAllowed = 1;
+        cfg.numAttrs = 2;
+    }
+    cudaLaunchKernelEx(&cfg, kern, KArgs(args)...);
+}
+
 #define FLEXLLM_CHECK_CUDA(expr)                                   \
     do {                                                           \
         int _st = ::flexllm::cuda_status((expr));                  \

@@ -373,9 +373,19 @@ __global__ void __launch_bounds__(1024) argmax_kernel(const float* __restrict__ 
     const float* l = logits + (long)blockIdx.x * V;
     float best = -INFINITY;
     int bi = 0x7fffffff;
-    for (long v = threadIdx.x; v < V; v += blockDim.x) {
-        float t = l[v];
-        if (t > best || bi == 0x7fffffff) { best = t; bi = (int)v; }   // strided scan visits increasing v
+    // strided scan in increasing v; eight loads in flight
+    long v = threadIdx.x;
+    for (; v + 7L * blockDim.x < V; v += 8L * blockDim.x) {
+        float t[8];
+#pragma unroll
+        for (int i = 0; i < 8; i++) t[i] = l[v + (long)i * blockDim.x];
+#pragma unroll
+        for (int i = 0; i < 8; i++)
+            if (t[i] > best || bi == 0x7fffffff) { best = t[i]; bi = (int)(v + (long)i * blockDim.x); }
+    }
+    for (; v < V; v += blockDim.x) {
+        const float t = l[v];
+        if (t > best || bi == 0x7fffffff) { best = t; bi = (int)v; }
     }
     auto better = [](float a, int ai, float b, int bi2) { return a > b || (a == b && ai < bi2); };
 #pragma unroll

@@ -4,12 +4,12 @@
 // producer warp (128-byte-swizzled K-major tiles), one MMA-issuing thread, four epilogue warps on a
 // double-buffered TMEM accumulator.
 //   prompts: A = activations (128-row side), B = weights (BN rows)
-//   decode : A = weights, B = activations (M <= 64), split over K; the splits' fp32 partial sums go to slabs
-//            and the last arriver adds them in split order, so the result does not depend on timing
+//   decode : A = weights, B = activations (M <= 64), split over K within a thread-block cluster: each CTA leaves its
+//            fp32 partial tile in shared memory and the cluster's CTAs add them, a share of the tokens each, over
+//            distributed shared memory and in rank order, so the result does not depend on timing
 // Epilogue: optional bias, optional gated GELU (weight rows alternating in blocks of 16 gate / 16 up rows),
 // fp32 or bf16 output.
 #include <atomic>
-#include <mutex>
 
 #include "float_common.cuh"
 #include "tc_common.cuh"
@@ -27,7 +27,6 @@ struct GemmBfArgs {
     float* y32; bf16* y16;
     const float* bias;                 // per output channel (row of the weights)
     int glu, vec;                      // vec: rows of the output are 16-byte aligned
-    float* slabs; int* counters;       // split-K: [ksplit][rowsB][rowsA] partial sums, zeroed arrival counters
     int* error_flag;
 };
 
@@ -78,6 +77,22 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tcgen05_kernel(const __grid_
     tc_fence_after();
     const uint32_t tmem_base = *tmem_base_slot;
     pdl_sync();
+
+    // decode form: one value of token `tok`, weight row rowA (this lane's; row0: the warp's first); a warp store covers 32 channels
+    auto emit = [&](float v, int tok, int rowA, int row0, float bA) {
+        v += bA;
+        if (args.glu) {
+            const float up = __shfl_xor_sync(0xffffffffu, v, 16);
+            if (lane < 16 && rowA < args.rowsA) {
+                const float r = gelu_tanh_f<true>(v) * up;
+                const long o = (long)tok * args.ldo + (row0 >> 1) + lane;
+                if (args.y16) args.y16[o] = __float2bfloat16_rn(r); else args.y32[o] = r;
+            }
+        } else if (rowA < args.rowsA) {
+            const long o = (long)tok * args.ldo + rowA;
+            if (args.y16) args.y16[o] = __float2bfloat16_rn(v); else args.y32[o] = v;
+        }
+    };
 
     if (warp == 0) {
         if (lane == 0) {
@@ -245,21 +260,8 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tcgen05_kernel(const __grid_
                 __syncwarp();
                 if (lane == 0) mbar_arrive(bar_tempty + 8 * as);
             } else {
-                // lane = weight row, columns = tokens: a warp store covers 32 channels of one token
-                auto emit = [&](float v, int tok) {
-                    v += bA;
-                    if (args.glu) {
-                        const float up = __shfl_xor_sync(0xffffffffu, v, 16);
-                        if (lane < 16 && rowA_ok) {
-                            const float r = gelu_tanh_f<true>(v) * up;
-                            const long o = (long)tok * args.ldo + (row0 >> 1) + lane;
-                            if (args.y16) args.y16[o] = __float2bfloat16_rn(r); else args.y32[o] = r;
-                        }
-                    } else if (rowA_ok) {
-                        const long o = (long)tok * args.ldo + rowA;
-                        if (args.y16) args.y16[o] = __float2bfloat16_rn(v); else args.y32[o] = v;
-                    }
-                };
+                // lane = weight row, columns = tokens
+                float* part = reinterpret_cast<float*>(ring_ptr);
 #pragma unroll
                 for (int c = 0; c < BN / 16; c++) {
                     uint32_t v[16];
@@ -268,45 +270,39 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tcgen05_kernel(const __grid_
 #pragma unroll
                     for (int j = 0; j < 16; j++) {
                         const int tok = tb * BN + c * 16 + j;
-                        if (tok < args.rowsB) {
-                            if (args.ksplit > 1) {
-                                if (rowA_ok) args.slabs[((long)split * args.rowsB + tok) * args.rowsA + rowA] = __uint_as_float(v[j]);
-                            } else {
-                                emit(__uint_as_float(v[j]), tok);
-                            }
-                        }
+                        if (args.ksplit > 1) part[(c * 16 + j) * 128 + q * 32 + lane] = __uint_as_float(v[j]);
+                        else if (tok < args.rowsB) emit(__uint_as_float(v[j]), tok, rowA, row0, bA);
                     }
                 }
                 tc_fence_before();
                 __syncwarp();
                 if (lane == 0) mbar_arrive(bar_tempty + 8 * as);
-                if (args.ksplit > 1) {
-                    __threadfence();
-                    __syncwarp();
-                    int last = 0;
-                    if (lane == 0) last = (atomicAdd(args.counters + ta * 4 + q, 1) == args.ksplit - 1);
-                    last = __shfl_sync(0xffffffffu, last, 0);
-                    if (last) {
-                        __threadfence();
-                        for (int t0 = 0; t0 < args.rowsB; t0 += 8) {
-                            float s[8];
-#pragma unroll
-                            for (int j = 0; j < 8; j++) s[j] = 0.0f;
-                            for (int k = 0; k < args.ksplit; k++)
-#pragma unroll
-                                for (int j = 0; j < 8; j++)
-                                    if (rowA_ok && t0 + j < args.rowsB) s[j] += __ldcg(args.slabs + ((long)k * args.rowsB + t0 + j) * args.rowsA + rowA);
-#pragma unroll
-                            for (int j = 0; j < 8; j++)
-                                if (t0 + j < args.rowsB) emit(s[j], t0 + j);
-                        }
-                        if (lane == 0) args.counters[ta * 4 + q] = 0;
-                    }
-                }
             }
         }
     }
 
+    if (SWAP && args.ksplit > 1) {
+        // every CTA of the cluster has one tile, the same for all of them: the partial tiles are in the rings (their MMAs
+        // have finished reading), and CTA r adds up tokens r, r + ksplit, ...
+        tc_fence_before();
+        cluster_sync();
+        if (warp >= 2 && !*abort_flag) {
+            const int q = warp & 3, ta = blockIdx.x / args.ksplit, r = blockIdx.x % args.ksplit;
+            const int row0 = ta * 128 + q * 32, rowA = row0 + lane;
+            const float bA = (args.bias && rowA < args.rowsA) ? args.bias[rowA] : 0.0f;
+            for (int tok = r; tok < args.rowsB; tok += args.ksplit) {
+                float p[8];
+#pragma unroll
+                for (int k = 0; k < 8; k++)
+                    p[k] = k < args.ksplit ? ld_cluster_f32(cluster_addr(ring + (uint32_t)(tok * 128 + q * 32 + lane) * 4u, k)) : 0.0f;
+                float s = p[0];
+#pragma unroll
+                for (int k = 1; k < 8; k++) s += p[k];
+                emit(s, tok, rowA, row0, bA);
+            }
+        }
+        cluster_sync();                      // nobody leaves while its partial tile may still be read
+    }
     tc_fence_before();
     __syncthreads();
     if (*abort_flag) {
@@ -317,36 +313,6 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tcgen05_kernel(const __grid_
         __syncthreads();
     }
     if (warp == 1) { tc_fence_after(); tmem_dealloc(tmem_base, Cfg::TMEM_COLS); }
-}
-
-// Split-K slabs and counters, one set per device, allocated by the first decode-form call on the device (outside any
-// stream capture) and kept: captured graphs hold it by address. Counters are zero between launches. Calls that can
-// overlap on the GPU must be serialised by the caller, as for the int8 decode layer's scratch.
-constexpr size_t kSlabFloats = (size_t)160 * 128 * 64;      // tiles * splits <= number of SMs, 128 channels x 64 tokens each
-constexpr int kSlabCounters = 4096;
-struct SlabScratch { std::mutex mu; void* p = nullptr; };
-SlabScratch g_slabs[kMaxDevices];
-
-int slab_get(float** slabs, int** counters, cudaStream_t st) {
-    const int dev = current_device();
-    if (dev < 0) return FLEXLLM_ECUDA;
-    SlabScratch& s = g_slabs[dev];
-    std::lock_guard<std::mutex> lk(s.mu);
-    if (!s.p) {
-        cudaStreamCaptureStatus cap = cudaStreamCaptureStatusNone;
-        FLEXLLM_CHECK_CUDA(cudaStreamIsCapturing(st, &cap));
-        if (cap != cudaStreamCaptureStatusNone) return FLEXLLM_EINVAL;
-        void* p = nullptr;
-        cudaError_t e = cudaMalloc(&p, kSlabFloats * 4 + kSlabCounters * 4);
-        if (e != cudaSuccess) { g_last_cuda_error = (int)e; return e == cudaErrorMemoryAllocation ? FLEXLLM_ENOMEM : FLEXLLM_ECUDA; }
-        e = cudaMemset(p, 0, kSlabFloats * 4 + kSlabCounters * 4);
-        if (e == cudaSuccess) e = cudaDeviceSynchronize();
-        if (e != cudaSuccess) { cudaFree(p); return cuda_status(e); }
-        s.p = p;
-    }
-    *slabs = (float*)s.p;
-    *counters = (int*)((float*)s.p + kSlabFloats);
-    return FLEXLLM_OK;
 }
 
 template <int BN, bool SWAP, int KCH>
@@ -367,6 +333,11 @@ int launch(const bf16* A, int rowsA, long ldA, const bf16* B, int rowsB, long ld
         attr_set[dev].store(true, std::memory_order_release);
     }
     const int total = g.tilesA * g.tilesB * g.ksplit;
+    if (SWAP && g.ksplit > 1) {
+        // one tile per CTA, the splits of a tile form a cluster
+        launch_cluster(kern, dim3(total), dim3(192), g.ksplit, (size_t)Cfg::SMEM_BYTES, st, ta, tb, g);
+        return launch_status();
+    }
     const int grid = total < gemm_sm_count() ? total : gemm_sm_count();
     launch_k(kern, dim3(grid), dim3(192), (size_t)Cfg::SMEM_BYTES, st, ta, tb, g);
     return launch_status();
@@ -399,19 +370,14 @@ int gemm_bf16_decode(const bf16* a, long lda, const bf16* w, long ldw, const flo
     // K blocks per pipeline stage: longer contiguous runs per weight row and TMA request
     // ... as long as the splits that give every SM work keep two steps each
     const int kb = (K + 63) / 64, tiles = (N + 127) / 128;
-    int want = gemm_sm_count() / tiles;
-    if (want < 1 || tiles * 4 > kSlabCounters) want = 1;
+    int ks = 1;
+    while (ks < 8 && tiles * ks * 2 <= gemm_sm_count() && kb >= 4 * ks) ks *= 2;
     int kch = 1;
     if (lda % 64 == 0 && ldw % 64 == 0) {
-        if (kb % 4 == 0 && kb / 4 >= 2 * want) kch = 4;
-        else if (kb % 2 == 0 && kb / 2 >= 2 * want) kch = 2;
+        if (kb % 4 == 0 && kb / 4 >= 2 * ks) kch = 4;
+        else if (kb % 2 == 0 && kb / 2 >= 2 * ks) kch = 2;
     }
-    const int steps = kb / kch;
-    int ks = want;
-    if (ks > steps / 2) ks = steps / 2;
-    if (ks < 1) ks = 1;
     g.ksplit = ks;
-    if (ks > 1) TRY_RC(slab_get(&g.slabs, &g.counters, st));
 #define FLEXLLM_DEC(BN_, KCH_) return launch<BN_, true, KCH_>(w, N, ldw, a, M, lda, K, g, st)
     if (M > 32) { if (kch == 4) FLEXLLM_DEC(64, 4); if (kch == 2) FLEXLLM_DEC(64, 2); FLEXLLM_DEC(64, 1); }
     if (M > 16) { if (kch == 4) FLEXLLM_DEC(32, 4); if (kch == 2) FLEXLLM_DEC(32, 2); FLEXLLM_DEC(32, 1); }

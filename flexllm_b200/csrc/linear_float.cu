@@ -1,6 +1,6 @@
-// Linear layers of the floating-point model path that do not need the tensor cores, and the choice between
-// the forms: a weight-streaming GEMV for a few tokens (T = bf16 or float activations, bf16 weights), the
-// tcgen05 GEMMs for more (gemm_bf16.cu), and a tiled fp32 GEMM for the 32-bit mode.
+// Linear layers of the floating-point model path apart from the tcgen05 GEMMs (gemm_bf16.cu), and the choice between the
+// forms: a weight-streaming GEMV for one or two tokens (T = bf16 or float activations, bf16 weights), its warp-MMA form for
+// more, and a tiled fp32 GEMM for the 32-bit mode.
 #include "float_common.cuh"
 
 namespace flexllm {
@@ -133,6 +133,102 @@ __global__ void __launch_bounds__(128) gemv_float_kernel(const T* __restrict__ a
     }
 }
 
+// A few tokens, bf16: weight streaming with warp-level bf16 MMAs. A CTA takes RT blocks of 16 weight rows (the MMA's row side;
+// GLU: one gate and one up block), its eight warps share K; the tokens are the column side, NT blocks of 8. Rows of both
+// operands are read straight from memory with 16-byte loads: lane % 4 holds elements 8 c .. 8 c + 7 of every 32, i.e. the inner
+// index is permuted, the same way on both sides. The warps' partial sums are added in warp order.
+template <int NT, int RT, bool GLU>
+__global__ void __launch_bounds__(256) skinny_mma_kernel(const bf16* __restrict__ a, long lda, const bf16* __restrict__ w, long ldw,
+                                                         const float* __restrict__ bias, int M, int N, int kv, float* y32, bf16* y16, long ldy) {
+    constexpr int G = NT * RT >= 4 ? 2 : 4;                 // 32-element chunks per step
+    __shared__ float part[8][RT * 16][NT * 8 + 1];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lr = lane >> 2, lc = lane & 3;
+    const int row0 = blockIdx.x * RT * 16;
+    const int n_ch = (kv + 3) >> 2;                         // kv: 8-element vectors per row
+    const int c_beg = (int)((long)warp * n_ch / 8), c_end = (int)((long)(warp + 1) * n_ch / 8);
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    const bf16* wr[RT][2];
+#pragma unroll
+    for (int r = 0; r < RT; r++)
+#pragma unroll
+        for (int h = 0; h < 2; h++) wr[r][h] = w + (long)min(row0 + r * 16 + h * 8 + lr, N - 1) * ldw + lc * 8;
+    uint4 wv[G][RT][2], nx[G][RT][2];
+    auto load_w = [&](uint4 (&v)[G][RT][2], int c) {
+#pragma unroll
+        for (int g = 0; g < G; g++)
+#pragma unroll
+            for (int r = 0; r < RT; r++)
+#pragma unroll
+                for (int h = 0; h < 2; h++)
+                    v[g][r][h] = (c + g < c_end && (c + g) * 4 + lc < kv) ? ldg_stream16(wr[r][h] + (long)(c + g) * 32) : zero;
+    };
+    load_w(nx, c_beg);
+    pdl_sync();
+    float acc[RT][NT][4] = {};
+    for (int c = c_beg; c < c_end; c += G) {
+#pragma unroll
+        for (int g = 0; g < G; g++)
+#pragma unroll
+            for (int r = 0; r < RT; r++)
+#pragma unroll
+                for (int h = 0; h < 2; h++) wv[g][r][h] = nx[g][r][h];
+        uint4 av[G][NT];
+#pragma unroll
+        for (int g = 0; g < G; g++)
+#pragma unroll
+            for (int t = 0; t < NT; t++)
+                av[g][t] = (t * 8 + lr < M && c + g < c_end && (c + g) * 4 + lc < kv)
+                               ? *reinterpret_cast<const uint4*>(a + (long)(t * 8 + lr) * lda + (long)(c + g) * 32 + lc * 8) : zero;
+        load_w(nx, c + G);
+#pragma unroll
+        for (int g = 0; g < G; g++)
+#pragma unroll
+            for (int r = 0; r < RT; r++)
+#pragma unroll
+                for (int t = 0; t < NT; t++) {
+                    mma_bf16(acc[r][t], wv[g][r][0].x, wv[g][r][1].x, wv[g][r][0].y, wv[g][r][1].y, av[g][t].x, av[g][t].y);
+                    mma_bf16(acc[r][t], wv[g][r][0].z, wv[g][r][1].z, wv[g][r][0].w, wv[g][r][1].w, av[g][t].z, av[g][t].w);
+                }
+    }
+#pragma unroll
+    for (int r = 0; r < RT; r++)
+#pragma unroll
+        for (int t = 0; t < NT; t++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) part[warp][r * 16 + lr + 8 * (i >> 1)][t * 8 + lc * 2 + (i & 1)] = acc[r][t][i];
+    __syncthreads();
+    auto total = [&](int row, int tok) {
+        float v = part[0][row][tok];
+#pragma unroll
+        for (int k = 1; k < 8; k++) v += part[k][row][tok];
+        const int n = row0 + row;
+        return v + (bias && n < N ? bias[n] : 0.0f);
+    };
+    constexpr int OUT = GLU ? 16 : RT * 16;                 // output columns of the CTA
+    const int n0 = GLU ? row0 >> 1 : row0, n_out = GLU ? N >> 1 : N;
+    for (int i = threadIdx.x; i < OUT * M; i += 256) {
+        const int tok = i / OUT, o = i - tok * OUT;
+        if (n0 + o >= n_out) continue;
+        const float v = GLU ? gelu_tanh_f<true>(total(o, tok)) * total(RT * 16 - 16 + o, tok) : total(o, tok);
+        if (y32) y32[(long)tok * ldy + n0 + o] = v;
+        else y16[(long)tok * ldy + n0 + o] = __float2bfloat16_rn(v);
+    }
+}
+
+template <int NT>
+int skinny_nt(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st) {
+    const int kv = (K + 7) / 8;
+    if (glu) launch_k(skinny_mma_kernel<NT, 2, true>, dim3((N + 31) / 32), dim3(256), 0, st, a, lda, w, ldw, bias, M, N, kv, y.f32, (bf16*)y.t, y.ld);
+    else if (N >= 148 * 4 * 16) launch_k(skinny_mma_kernel<NT, 2, false>, dim3((N + 31) / 32), dim3(256), 0, st, a, lda, w, ldw, bias, M, N, kv, y.f32, (bf16*)y.t, y.ld);
+    else launch_k(skinny_mma_kernel<NT, 1, false>, dim3((N + 15) / 16), dim3(256), 0, st, a, lda, w, ldw, bias, M, N, kv, y.f32, (bf16*)y.t, y.ld);
+    return launch_status();
+}
+int skinny_mma(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st) {
+    if (M <= 8) return skinny_nt<1>(a, lda, w, ldw, bias, M, N, K, glu, y, st);
+    if (M <= 16) return skinny_nt<2>(a, lda, w, ldw, bias, M, N, K, glu, y, st);
+    return skinny_nt<4>(a, lda, w, ldw, bias, M, N, K, glu, y, st);
+}
+
 template <class T, int BT, int R, int KS, bool GLU>
 int launch_gemv(const T* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, LinearOut y, cudaStream_t st) {
     const int kv = (K + 7) / 8;
@@ -153,12 +249,12 @@ int gemv_bt(const T* a, long lda, const bf16* w, long ldw, const float* bias, in
     return launch_gemv<T, BT, 2, 1, GLU>(a, lda, w, ldw, bias, M, N, K, y, st);
 }
 
-template <class T>
+template <class T>               // M <= 4 (bf16: M <= 2, more goes to the MMA forms)
 int gemv_any(const T* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st) {
 #define FLEXLLM_GEMV(BT_) return glu ? gemv_bt<T, BT_, true>(a, lda, w, ldw, bias, M, N, K, y, st) : gemv_bt<T, BT_, false>(a, lda, w, ldw, bias, M, N, K, y, st)
     if (M <= 1) FLEXLLM_GEMV(1);
-    if (M <= 2) FLEXLLM_GEMV(2);
-    FLEXLLM_GEMV(4);
+    if (sizeof(T) == 2 || M <= 2) FLEXLLM_GEMV(2);
+    FLEXLLM_GEMV(sizeof(T) == 2 ? 2 : 4);
 #undef FLEXLLM_GEMV
 }
 
@@ -227,10 +323,14 @@ int check(const void* a, long lda, const void* w, long ldw, int M, int N, int K,
 int linear_bf16(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st) {
     TRY_RC(check(a, lda, w, ldw, M, N, K, glu, y));
     if (M == 0) return FLEXLLM_OK;
-    if (M <= 4) {
+    // Measured on the layer shapes of 1B to 8B models: the scalar GEMV wins for one token (two for wide matrices), the
+    // tensor-core form where its 128-row tiles alone fill most SMs, the warp-MMA form for the narrow rest.
+    const bool wide = (N + 127) / 128 >= 100;
+    if ((M == 1 && K <= 12288) || (M == 2 && wide)) {
         const int rc = gemv_any<bf16>(a, lda, w, ldw, bias, M, N, K, glu, y, st);
         if (rc != FLEXLLM_ENOTSUP) return rc;
     }
+    if (M <= 16 ? !wide : M <= 32 && !wide && (long)N * K <= (17L << 20)) return skinny_mma(a, lda, w, ldw, bias, M, N, K, glu, y, st);
     if (M <= 64) return gemm_bf16_decode(a, lda, w, ldw, bias, M, N, K, glu, y, st);
     return gemm_bf16_prefill(a, lda, w, ldw, bias, M, N, K, glu, y, st);
 }
