@@ -21,6 +21,9 @@ int main() {
     if (pref_Linear_Layer_i4xi4(nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, 8, 64, 64) != FLEXLLM_EINVAL) return 7;
     HMT hmt; SpinQuantModel model;
     if (hmt.Prefilling(nullptr, 16) != FLEXLLM_EINVAL) return 8;
+    DecoderModel dec;
+    flexllm_decoder_config none = {};
+    if (dec.create(none) != FLEXLLM_EINVAL || dec.step(nullptr, 1, 1, nullptr, 0, nullptr) != FLEXLLM_EINVAL) return 9;
     std::printf("%s\n", status_string(FLEXLLM_EINVAL));
     return 0;
 }
