@@ -2,15 +2,17 @@
 //   q, k = rms norm over the whole projection, before the split into heads
 //   s    = softcap * tanh(scale * (q . k) / softcap) + bias[head][i - j]          0 <= i - j < window
 //   p    = exp(s) / (sink + sum exp(s)),   out = (sum p v) * logistic(gate)
-// Softcap, sink and gate are optional; the distance bias and the window are one table per layer (-inf outside the
-// window), so that a masked key costs nothing extra. Scores, weights and sums are fp32.
+// Norms, softcap, bias, sink (a score of 0, or one learned score per head) and gate are optional; the first `keep` positions may
+// stay visible behind the window; a call may use another layer's keys and values. A distance bias and the window are one
+// table per layer (-inf outside the window), so that a masked key costs nothing extra. Scores, weights and sums are fp32.
 //
 // Cache pages hold 64 tokens, K [page][G][64][dkp] and V transposed [page][G][dv][64] (as the int8 cache does).
 //   one token per sequence : attn_decode_mma_kernel (bf16), else attn_row_kernel<FUSED>: norms, append and attention in one
 //                            launch, keys split over CTAs
 //   prompts, bf16          : attn_prepare_kernel, then attn_window_prefill_kernel on tcgen05
 //   prompts, otherwise     : attn_prepare_kernel, then attn_row_kernel row by row
-// The sink is a score of 0, so max(0, largest score) is a valid softmax shift; without a sink the running maximum is.
+// Where softcap and bias bound the scores, the tensor-core forms use a constant softmax shift; otherwise (no softcap, no bias)
+// their ONLINE variants keep a running maximum, which starts at the sink's score.
 #include <cmath>
 #include <vector>
 
@@ -39,6 +41,22 @@ __device__ __forceinline__ int start_pos(const AttnCall& c, int b, int* error_fl
     return pos;
 }
 
+// Logical pages that a range of positions reads: the pages of the kept first positions, then those of the window.
+struct KeyPages {
+    int keep, lo, n;
+    __device__ __forceinline__ KeyPages(const AttnShape& s, int first, int last) {        // positions [first, last]
+        lo = max(0, first - s.window + 1) / PG;
+        keep = min((s.keep + PG - 1) / PG, lo);
+        n = keep + last / PG - lo + 1;
+    }
+    __device__ __forceinline__ int at(int i) const { return i < keep ? i : lo + i - keep; }
+};
+__device__ __forceinline__ bool sees(const AttnShape& s, int pos, int key) { return key <= pos && (pos - key < s.window || key < s.keep); }
+// Score of the sink of head h (-inf: none).
+__device__ __forceinline__ float sink_score(const AttnCall& c, int h) {
+    return c.s.sink == 2 ? c.sinks[h] : c.s.sink ? 0.0f : -INFINITY;
+}
+
 // This thread's share (NT threads) of the sum of squares of n elements at a 16-byte aligned address.
 template <int NT, class T> __device__ __forceinline__ float share_sumsq(const T* p, int n, int tid) {
     float s = 0.0f;
@@ -57,13 +75,21 @@ template <int NT, class T> __device__ __forceinline__ float share_sumsq(const T*
 template <class T> __device__ __forceinline__ void normed8(const T* src, const float* gain, int j0, int e0, int dk, float r, float (&f)[8]) {
     if ((dk & 7) == 0) {
         load8(src + j0 + e0, f);
+        if (!gain) return;
         const float4 a = load4(gain + j0 + e0), b = load4(gain + j0 + e0 + 4);
         f[0] = (f[0] * r) * a.x; f[1] = (f[1] * r) * a.y; f[2] = (f[2] * r) * a.z; f[3] = (f[3] * r) * a.w;
         f[4] = (f[4] * r) * b.x; f[5] = (f[5] * r) * b.y; f[6] = (f[6] * r) * b.z; f[7] = (f[7] * r) * b.w;
     } else {
 #pragma unroll
-        for (int e = 0; e < 8; e++) f[e] = e0 + e < dk ? (to_f(src[j0 + e0 + e]) * r) * gain[j0 + e0 + e] : 0.0f;
+        for (int e = 0; e < 8; e++) f[e] = e0 + e < dk ? (gain ? (to_f(src[j0 + e0 + e]) * r) * gain[j0 + e0 + e] : to_f(src[j0 + e0 + e])) : 0.0f;
     }
+}
+// Reciprocal root mean squares of the q and k projections of a row (1 without norms).
+template <class T> __device__ __forceinline__ float2 qk_rms(const AttnCall& c, const T* row, int tid, float* red) {
+    if (!c.q_gain) return make_float2(1.0f, 1.0f);
+    const int nq = c.s.H * c.s.dk, nk = c.s.G * c.s.dk;
+    const float2 ss = block_sum2<256>(share_sumsq<256>(row + c.s.q_off, nq, tid), share_sumsq<256>(row + c.s.k_off, nk, tid), red);
+    return make_float2(1.0f / sqrtf(ss.x / (float)nq + c.eps), 1.0f / sqrtf(ss.y / (float)nk + c.eps));
 }
 template <class T> __device__ __forceinline__ void store8(T* p, const float (&f)[8]) {
     store4(p, make_float4(f[0], f[1], f[2], f[3]));
@@ -84,9 +110,8 @@ __global__ void __launch_bounds__(256) attn_prepare_kernel(const AttnCall c, int
         const int m = blockIdx.x, b = m / c.Sc;
         const int pos = start_pos(c, b, error_flag) + m % c.Sc;
         const T* src = (const T*)c.proj + (long)m * s.ld;
-        const int nq = s.H * s.dk, nk = s.G * s.dk;
-        const float2 ss = block_sum2<256>(share_sumsq<256>(src + s.q_off, nq, tid), share_sumsq<256>(src + s.k_off, nk, tid), red);
-        const float rq = 1.0f / sqrtf(ss.x / (float)nq + c.eps), rk = 1.0f / sqrtf(ss.y / (float)nk + c.eps);
+        const float2 rms = qk_rms(c, src, tid, red);
+        const float rq = rms.x, rk = rms.y;
         T* q = (T*)c.q + (long)m * s.H * s.dkp;
         const int nv = s.dkp >> 3;                                  // 8-element blocks per head
         for (int i = tid; i < s.H * nv; i += 256) {
@@ -95,6 +120,7 @@ __global__ void __launch_bounds__(256) attn_prepare_kernel(const AttnCall c, int
             normed8(src + s.q_off, c.q_gain, h * s.dk, e0, s.dk, rq, f);
             store8(q + (long)i * 8, f);
         }
+        if (s.k_off < 0) return;
         const long page = c.page_table[(long)b * c.max_pages + pos / PG];
         T* kp = (T*)c.k_pool + (page * s.G * PG + (pos & (PG - 1))) * s.dkp;
         for (int i = tid; i < s.G * nv; i += 256) {
@@ -165,20 +191,19 @@ __global__ void __launch_bounds__(256) attn_row_kernel(const AttnCall c, int L, 
     const T* prow = (const T*)c.proj + (long)row * s.ld;
     const long kh = (long)PG * s.dkp, vh = (long)PG * s.dv;          // one head of a page
     if (FUSED) {
-        const int nq = s.H * s.dk, nk = s.G * s.dk;
-        const float2 ss = block_sum2<256>(share_sumsq<256>(prow + s.q_off, nq, tid), share_sumsq<256>(prow + s.k_off, nk, tid), red);
-        const float rq = 1.0f / sqrtf(ss.x / (float)nq + c.eps), rk = 1.0f / sqrtf(ss.y / (float)nk + c.eps);
+        const float2 rms = qk_rms(c, prow, tid, red);
+        const float rq = rms.x, rk = rms.y;
         for (int i = tid; i < R * s.dkp; i += 256) {
             const int r = i / s.dkp, e = i - r * s.dkp, j = (g * R + r) * s.dk + e;
-            q_sm[i] = e < s.dk ? (to_f(prow[s.q_off + j]) * rq) * c.q_gain[j] : 0.0f;
+            q_sm[i] = e < s.dk ? (to_f(prow[s.q_off + j]) * rq) * (c.q_gain ? c.q_gain[j] : 1.0f) : 0.0f;
         }
-        if (split == n_split - 1) {               // the split that holds the newest key appends it
+        if (s.k_off >= 0 && split == n_split - 1) {               // the split that holds the newest key appends it
             const long page = pt[pos / PG];
             const int slot = pos & (PG - 1);
             T* kp = (T*)c.k_pool + (page * s.G + g) * kh + (long)slot * s.dkp;
             for (int e = tid; e < s.dkp; e += 256) {
                 const int j = g * s.dk + e;
-                kp[e] = from_f<T>(e < s.dk ? (to_f(prow[s.k_off + j]) * rk) * c.k_gain[j] : 0.0f);
+                kp[e] = from_f<T>(e < s.dk ? (to_f(prow[s.k_off + j]) * rk) * (c.k_gain ? c.k_gain[j] : 1.0f) : 0.0f);
             }
             T* vp = (T*)c.v_pool + (page * s.G + g) * vh + slot;
             for (int d = tid; d < s.dv; d += 256) vp[(long)d * PG] = prow[s.v_off + g * s.dv + d];
@@ -188,18 +213,18 @@ __global__ void __launch_bounds__(256) attn_row_kernel(const AttnCall c, int L, 
         for (int i = tid; i < R * s.dkp; i += 256) q_sm[i] = to_f(q[i]);
     }
     for (int i = tid; i < R * s.dv; i += 256) o_sm[i] = 0.0f;
-    for (int i = tid; i < R; i += 256) { m_sm[i] = s.sink ? 0.0f : -INFINITY; l_sm[i] = 0.0f; }
+    for (int i = tid; i < R; i += 256) { m_sm[i] = sink_score(c, g * R + i); l_sm[i] = 0.0f; }
     __syncthreads();
 
-    const int lo = max(0, pos - s.window + 1);
-    const int p_lo = lo / PG, n_pg = pos / PG - p_lo + 1;
+    const KeyPages pages(s, pos, pos);
+    const int n_pg = pages.n;
     const int n_tiles = (n_pg + TILE_PAGES - 1) / TILE_PAGES;
     const int t_beg = (int)((long)split * n_tiles / n_split), t_end = (int)((long)(split + 1) * n_tiles / n_split);
-    const float* bias_g = c.bias + (long)g * (2 * kBiasPad + s.window) * R;
+    const float* bias_g = c.bias ? c.bias + (long)g * (2 * kBiasPad + s.window) * R : nullptr;
     const float inv_cap = s.softcap > 0.0f ? s.scale / s.softcap : 0.0f;
     const int kpw = 32 / L, sub = lane / L, ln = lane % L;            // keys per warp step, this lane's key and part
     for (int t = t_beg; t < t_end; t++) {
-        const int pg0 = p_lo + t * TILE_PAGES, npg = min(TILE_PAGES, n_pg - t * TILE_PAGES);
+        const int pg0 = t * TILE_PAGES, npg = min(TILE_PAGES, n_pg - t * TILE_PAGES);
         // ---- scores of the tile's keys
         for (int r0 = 0; r0 < R; r0 += RC) {
             float qr[RC][8];
@@ -210,7 +235,8 @@ __global__ void __launch_bounds__(256) attn_row_kernel(const AttnCall c, int L, 
                     for (int e = 0; e < 8; e++) qr[r][e] = (r0 + r < R && ln * 8 < s.dkp) ? q_sm[(r0 + r) * s.dkp + ln * 8 + e] : 0.0f;
 #pragma unroll 2
             for (int k = warp * kpw + sub; k < npg * PG; k += 8 * kpw) {
-                const T* kp = (const T*)c.k_pool + ((long)pt[pg0 + (k >> 6)] * s.G + g) * kh + (long)(k & (PG - 1)) * s.dkp;
+                const int lp = pages.at(pg0 + (k >> 6));                         // logical page
+                const T* kp = (const T*)c.k_pool + ((long)pt[lp] * s.G + g) * kh + (long)(k & (PG - 1)) * s.dkp;
                 float acc[RC];
 #pragma unroll
                 for (int r = 0; r < RC; r++) acc[r] = 0.0f;
@@ -236,19 +262,19 @@ __global__ void __launch_bounds__(256) attn_row_kernel(const AttnCall c, int L, 
                 for (int off = L >> 1; off > 0; off >>= 1)
 #pragma unroll
                     for (int r = 0; r < RC; r++) acc[r] += __shfl_xor_sync(0xffffffffu, acc[r], off);
-                const int d = pos - (pg0 * PG + k);
+                const int key = lp * PG + (k & (PG - 1));
 #pragma unroll
                 for (int r = 0; r < RC; r++)
                     if (r0 + r < R && ln == (r & (L - 1))) {
                         float v = -INFINITY;
-                        if (d >= 0 && d < s.window) {
+                        if (sees(s, pos, key)) {
                             if (s.softcap > 0.0f) {
                                 const float z = acc[r] * inv_cap;
                                 v = s.softcap * (FAST ? 1.0f - 2.0f * rcp_fast(1.0f + ex2_fast(z * (2.0f * kLog2e))) : tanhf(z));
                             } else {
                                 v = acc[r] * s.scale;
                             }
-                            v += bias_g[(long)(d + kBiasPad) * R + r0 + r];
+                            if (bias_g) v += bias_g[(long)(pos - key + kBiasPad) * R + r0 + r];
                         }
                         s_sm[(r0 + r) * TILE_KEYS + k] = v;
                     }
@@ -289,7 +315,7 @@ __global__ void __launch_bounds__(256) attn_row_kernel(const AttnCall c, int L, 
 #pragma unroll 4
                     for (int p = 0; p < npg; p++) {
                         float vf[8];
-                        load8((const T*)c.v_pool + ((long)pt[pg0 + p] * s.G + g) * vh + (long)d * PG + tv * 8, vf);
+                        load8((const T*)c.v_pool + ((long)pt[pages.at(pg0 + p)] * s.G + g) * vh + (long)d * PG + tv * 8, vf);
 #pragma unroll
                         for (int r = 0; r < RC; r++) {
                             if (r0 + r >= R) continue;
@@ -330,7 +356,7 @@ __global__ void __launch_bounds__(256) attn_row_kernel(const AttnCall c, int L, 
         if (!last_sm) return;
         __threadfence();
         for (int r = tid; r < R; r += 256) {
-            float m = s.sink ? 0.0f : -INFINITY;
+            float m = sink_score(c, g * R + r);
             for (int k = 0; k < n_split; k++) m = fmaxf(m, __ldcg(part + k * stride + r));
             float l = 0.0f;
             for (int k = 0; k < n_split; k++) {
@@ -357,7 +383,7 @@ __global__ void __launch_bounds__(256) attn_row_kernel(const AttnCall c, int L, 
     T* out = (T*)c.out + (long)row * c.ldo + (long)g * R * s.dv;
     for (int i = tid; i < R * s.dv; i += 256) {
         const int r = i / s.dv;
-        const float den = l_sm[r] + (s.sink ? expf(-m_sm[r]) : 0.0f);
+        const float den = l_sm[r] + (s.sink ? expf(sink_score(c, g * R + r) - m_sm[r]) : 0.0f);
         float v = o_sm[i] / den;
         if (s.g_off >= 0) v *= sigmoid_f<FAST>(to_f(prow[s.g_off + (long)g * R * s.dv + i]));
         out[i] = from_f<T>(v);
@@ -841,7 +867,7 @@ template <class T, bool FUSED> int run_row(const AttnCall& c, cudaStream_t st) {
     const long ctas = (long)c.B * c.Sc * s.G;
     if (ctas / s.G > 65535) return FLEXLLM_ENOTSUP;
     const int reach = s.window < c.max_pos + 1 ? s.window : c.max_pos + 1;
-    const int tiles = (reach + 2 * PG - 2) / PG / TILE_PAGES + 1;
+    const int tiles = ((reach + 2 * PG - 2) / PG + attn_keep_pages(s.keep)) / TILE_PAGES + 1;
     long splits = 1;
     if (FUSED && c.ws) {
         splits = 2L * gemm_sm_count() / ctas;
@@ -863,7 +889,7 @@ template <class T, bool FUSED> int run_row(const AttnCall& c, cudaStream_t st) {
 // (no softcap) or so wide that sums could vanish below the smallest floats.
 bool bounded_scores(const AttnCall& c, float* a2, float* b2, float* shift2) {
     const AttnShape& s = c.s;
-    if (s.softcap <= 0.0f) return false;
+    if (s.softcap <= 0.0f || !c.bias || s.keep || s.sink == 2) return false;
     const float bound2 = (s.softcap + c.bias_max_abs) * kLog2e;
     *shift2 = bound2 > 100.0f ? bound2 - 100.0f : 0.0f;
     *a2 = s.scale / s.softcap * 2.0f * kLog2e; *b2 = -2.0f * s.softcap * kLog2e;
@@ -953,9 +979,10 @@ template <> bool run_tensor_prefill<bf16>(const AttnCall& c, cudaStream_t st, in
 
 int check_call(const AttnCall& c) {
     const AttnShape& s = c.s;
-    FLEXLLM_REQUIRE(c.proj && c.q_gain && c.k_gain && c.bias && c.k_pool && c.v_pool && c.page_table && c.ctx && c.out);
+    FLEXLLM_REQUIRE(c.proj && !c.q_gain == !c.k_gain && c.k_pool && c.v_pool && c.page_table && c.ctx && c.out);
+    FLEXLLM_REQUIRE(s.keep >= 0 && (!c.bias || s.keep == 0) && (s.sink != 2 || c.sinks) && (s.k_off >= 0 || !c.q_gain));
     FLEXLLM_REQUIRE(s.H > 0 && s.G > 0 && s.H % s.G == 0 && s.dk > 0 && s.dv > 0 && s.window > 0 && s.dkp % 8 == 0 && s.dkp >= s.dk);
-    FLEXLLM_REQUIRE(s.ld % 8 == 0 && s.q_off % 8 == 0 && s.k_off % 8 == 0 && s.v_off % 8 == 0 && (s.g_off < 0 || s.g_off % 8 == 0));
+    FLEXLLM_REQUIRE(s.ld % 8 == 0 && s.q_off % 8 == 0 && (s.k_off < 0 || (s.k_off % 8 == 0 && s.v_off % 8 == 0)) && (s.g_off < 0 || s.g_off % 8 == 0));
     FLEXLLM_REQUIRE(c.B > 0 && c.Sc > 0 && c.max_pos >= c.Sc - 1 && c.max_pos < c.max_pages * PG && c.n_pages > 0);
     return FLEXLLM_OK;
 }
@@ -967,12 +994,16 @@ size_t attn_window_ws_floats(int max_batch, int G, int R, int dv) {
     return ((size_t)kDecodeCtas + ctas) * R * (dv + 2);
 }
 
-void attn_layout(AttnShape* s, bool gate) {
+void attn_layout(AttnShape* s, bool gate, bool own_kv) {
     s->dkp = (int)up_to(s->dk, 8);
     s->q_off = 0;
-    s->k_off = (int)up_to((long)s->H * s->dk, 8);
-    s->v_off = s->k_off + (int)up_to((long)s->G * s->dk, 8);
-    const int end = s->v_off + (int)up_to((long)s->G * s->dv, 8);
+    s->k_off = s->v_off = -1;
+    int end = (int)up_to((long)s->H * s->dk, 8);
+    if (own_kv) {
+        s->k_off = end;
+        s->v_off = s->k_off + (int)up_to((long)s->G * s->dk, 8);
+        end = s->v_off + (int)up_to((long)s->G * s->dv, 8);
+    }
     s->g_off = gate ? end : -1;
     s->ld = gate ? end + up_to((long)s->H * s->dv, 8) : end;
 }
@@ -1005,7 +1036,7 @@ template <class T> int attn_window(const AttnCall& c, cudaStream_t st) {
         return rc == FLEXLLM_ENOTSUP ? run_row<T, true>(c, st) : rc;
     }
     FLEXLLM_REQUIRE(c.q);
-    const int v_pages = (c.Sc + PG - 2) / PG + 1;
+    const int v_pages = c.s.k_off >= 0 ? (c.Sc + PG - 2) / PG + 1 : 0;
     launch_k(attn_prepare_kernel<T>, dim3(c.B * c.Sc + c.B * c.s.G * v_pages), dim3(256), 0, st, c, v_pages, device_error_flag());
     TRY_RC(launch_status());
     int rc = FLEXLLM_OK;

@@ -90,13 +90,16 @@ int gemm_sm_count();
 // ---------------------------------------------------------------------------- linear layers
 // y[m][n] = sum_k a[m][k] w[n][k] (+ bias[n]); a T [M][lda], w bf16 [N][ldw]. ldw and lda are multiples of 8 and at least
 // K rounded up to 8; the columns from K on are zero in w and finite in a.
-// glu: rows of w alternate in blocks of 16 (gate 0..15, up 0..15, gate 16..31, ...): y[m][f] = gelu_tanh(gate_f) * up_f, N = 2 F.
+// act, applied to the sums: kActGeluGate: rows of w alternate in blocks of 16 (gate 0..15, up 0..15, gate 16..31, ...),
+// y[m][f] = gelu_tanh(gate_f) * up_f, N = 2 F; kActRelu2: max(y, 0)^2.
+enum { kActNone = 0, kActGeluGate = 1, kActRelu2 = 2 };
+__device__ __forceinline__ float relu2_f(float v) { v = fmaxf(v, 0.0f); return v * v; }
 struct LinearOut { float* f32; void* t; long ld; };      // exactly one of f32 / t (type T) is set
-int linear_bf16(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st);
-int linear_f32(const float* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st);
+int linear_bf16(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int act, LinearOut y, cudaStream_t st);
+int linear_f32(const float* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int act, LinearOut y, cudaStream_t st);
 // tensor-core kernels behind linear_bf16
-int gemm_bf16_prefill(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st);
-int gemm_bf16_decode(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st);
+int gemm_bf16_prefill(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int act, LinearOut y, cudaStream_t st);
+int gemm_bf16_decode(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int act, LinearOut y, cudaStream_t st);
 
 // ---------------------------------------------------------------------------- norms around a sublayer
 // One pass over the rows of the residual stream, every step optional:
@@ -120,18 +123,21 @@ template <class T> int res_norm(const ResNormArgs& a, int rows, cudaStream_t st)
 constexpr int kBiasPad = 192;               // masked (-inf) distances on either side of the window in the bias tables
 struct AttnShape {
     int H, G, dk, dv, dkp;                  // heads, key/value heads, sizes; dkp = dk rounded up to 8 (rows of Q and of the K pages)
-    int window;                             // i sees j with 0 <= i - j < window
+    int window;                             // i sees j with 0 <= i - j < window ...
+    int keep;                               // ... and every j < keep (0 <= j <= i)
     float scale, softcap;                   // softcap 0: none
-    int sink;                               // 1: one extra score of 0 without a value in the denominator
-    int q_off, k_off, v_off, g_off;         // columns of the fused projection; g_off < 0: no output gate
+    int sink;                               // an extra score without a value in the denominator: 0 none, 1 a score of 0, 2 one per head
+    int q_off, k_off, v_off, g_off;         // columns of the fused projection; g_off < 0: no output gate; k_off < 0: no keys and
+                                            // values of its own (the pools are another layer's, nothing is appended)
     long ld;                                // its row length
 };
 struct AttnCall {
     AttnShape s;
     const void* proj;                       // fused projection, T [rows][s.ld]
-    const float *q_gain, *k_gain; float eps;   // norm over the whole q (k) projection before the split into heads
-    const float* bias;                      // [G][kBiasPad + window + kBiasPad][H / G]: bias by distance, -inf outside the window
-    float bias_max_abs;
+    const float *q_gain, *k_gain; float eps;   // norm over the whole q (k) projection before the split into heads; nullptr: none
+    const float* bias;                      // [G][kBiasPad + window + kBiasPad][H / G]: bias by distance, -inf outside the window;
+    float bias_max_abs;                     // nullptr: none
+    const float* sinks;                     // [H], sink == 2
     void *k_pool, *v_pool;                  // T pages of this layer: K [page][G][64][dkp], V^T [page][G][dv][64]
     long n_pages;
     const int32_t* page_table; int max_pages;
@@ -146,8 +152,10 @@ struct AttnCall {
 // bf16 shapes it covers, row by row otherwise).
 template <class T> int attn_window(const AttnCall& c, cudaStream_t st);
 size_t attn_window_ws_floats(int max_batch, int G, int R, int dv);
+// Pages of a sequence that the first `keep` positions occupy (they stay where they are when the other pages form a ring).
+inline int attn_keep_pages(int keep) { return (keep + 63) / 64; }
 // Fills in the derived members: dkp, the columns of the fused projection (parts padded to multiples of 8) and its row length.
-void attn_layout(AttnShape* s, bool gate);
+void attn_layout(AttnShape* s, bool gate, bool own_kv = true);
 // The bias table of AttnCall::bias on the host, from a table [rows][H] of learned biases by bucketed distance.
 void attn_bias_table(const AttnShape& s, const float* table, int rows, int bias_max, float* out);
 inline size_t attn_bias_floats(const AttnShape& s) { return (size_t)s.H * (2 * kBiasPad + s.window); }

@@ -7,7 +7,7 @@
 //   decode : A = weights, B = activations (M <= 64), split over K within a thread-block cluster: each CTA leaves its
 //            fp32 partial tile in shared memory and the cluster's CTAs add them, a share of the tokens each, over
 //            distributed shared memory and in rank order, so the result does not depend on timing
-// Epilogue: optional bias, optional gated GELU (weight rows alternating in blocks of 16 gate / 16 up rows),
+// Epilogue: optional bias, optional gated GELU (weight rows alternating in blocks of 16 gate / 16 up rows) or squared ReLU,
 // fp32 or bf16 output.
 #include <atomic>
 
@@ -26,7 +26,7 @@ struct GemmBfArgs {
     long ldo;
     float* y32; bf16* y16;
     const float* bias;                 // per output channel (row of the weights)
-    int glu, vec;                      // vec: rows of the output are 16-byte aligned
+    int glu, relu2, vec;               // vec: rows of the output are 16-byte aligned
     int* error_flag;
 };
 
@@ -89,6 +89,7 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tcgen05_kernel(const __grid_
                 if (args.y16) args.y16[o] = __float2bfloat16_rn(r); else args.y32[o] = r;
             }
         } else if (rowA < args.rowsA) {
+            if (args.relu2) v = relu2_f(v);
             const long o = (long)tok * args.ldo + rowA;
             if (args.y16) args.y16[o] = __float2bfloat16_rn(v); else args.y32[o] = v;
         }
@@ -200,9 +201,10 @@ __global__ void __launch_bounds__(192, 1) gemm_bf16_tcgen05_kernel(const __grid_
 #pragma unroll
                         for (int g = 0; g < 8; g++) {
                             const float4 b4 = *reinterpret_cast<const float4*>(bw + c * 32 + 4 * g);
-                            *reinterpret_cast<float4*>(stg + lane * 32 + ((g ^ s7) << 2)) =
-                                make_float4(__uint_as_float(v[4 * g]) + b4.x, __uint_as_float(v[4 * g + 1]) + b4.y,
-                                            __uint_as_float(v[4 * g + 2]) + b4.z, __uint_as_float(v[4 * g + 3]) + b4.w);
+                            float4 o4 = make_float4(__uint_as_float(v[4 * g]) + b4.x, __uint_as_float(v[4 * g + 1]) + b4.y,
+                                                    __uint_as_float(v[4 * g + 2]) + b4.z, __uint_as_float(v[4 * g + 3]) + b4.w);
+                            if (args.relu2) o4 = make_float4(relu2_f(o4.x), relu2_f(o4.y), relu2_f(o4.z), relu2_f(o4.w));
+                            *reinterpret_cast<float4*>(stg + lane * 32 + ((g ^ s7) << 2)) = o4;
                         }
                     }
                     __syncwarp();
@@ -343,18 +345,19 @@ int launch(const bf16* A, int rowsA, long ldA, const bf16* B, int rowsB, long ld
     return launch_status();
 }
 
-GemmBfArgs base_args(const float* bias, bool glu, const LinearOut& y) {
+GemmBfArgs base_args(const float* bias, int act, const LinearOut& y) {
     GemmBfArgs g = {};
-    g.ksplit = 1; g.ldo = y.ld; g.y32 = y.f32; g.y16 = (bf16*)y.t; g.bias = bias; g.glu = glu;
+    g.ksplit = 1; g.ldo = y.ld; g.y32 = y.f32; g.y16 = (bf16*)y.t; g.bias = bias;
+    g.glu = act == kActGeluGate; g.relu2 = act == kActRelu2;
     return g;
 }
 
 }  // namespace
 
-int gemm_bf16_prefill(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y,
+int gemm_bf16_prefill(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int act, LinearOut y,
                       cudaStream_t st) {
-    GemmBfArgs g = base_args(bias, glu, y);
-    const int n_out = glu ? N / 2 : N;
+    GemmBfArgs g = base_args(bias, act, y);
+    const int n_out = g.glu ? N / 2 : N;
     g.vec = y.t ? (y.ld % 8 == 0 && n_out % 8 == 0 && aligned(y.t, 16)) : (y.ld % 4 == 0 && n_out % 4 == 0 && aligned(y.f32, 16));
     // the widest tile that still gives every SM work
     const long tiles256 = (long)((M + 127) / 128) * ((N + 255) / 256);
@@ -363,10 +366,10 @@ int gemm_bf16_prefill(const bf16* a, long lda, const bf16* w, long ldw, const fl
     return launch<64, false, 1>(a, M, lda, w, N, ldw, K, g, st);
 }
 
-int gemm_bf16_decode(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y,
+int gemm_bf16_decode(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int act, LinearOut y,
                      cudaStream_t st) {
     if (M > 64) return FLEXLLM_ENOTSUP;
-    GemmBfArgs g = base_args(bias, glu, y);
+    GemmBfArgs g = base_args(bias, act, y);
     // K blocks per pipeline stage: longer contiguous runs per weight row and TMA request
     // ... as long as the splits that give every SM work keep two steps each
     const int kb = (K + 63) / 64, tiles = (N + 127) / 128;

@@ -24,7 +24,7 @@ template <bool GLU> __device__ __forceinline__ long weight_row(int n0, int r, in
 // KS = 4: the four warps share R rows, a quarter of K each.
 template <class T, int BT, int R, int KS, bool GLU>
 __global__ void __launch_bounds__(128) gemv_float_kernel(const T* __restrict__ a, long lda, const bf16* __restrict__ w, long ldw,
-                                                         const float* __restrict__ bias, int M, int n_out, int kv, float* y32, T* yt,
+                                                         const float* __restrict__ bias, int M, int n_out, int kv, int relu2, float* y32, T* yt,
                                                          long ldy) {
     extern __shared__ __align__(16) uint8_t a_raw[];
     T* a_sm = reinterpret_cast<T*>(a_raw);               // [BT][kv * 8]
@@ -126,6 +126,7 @@ __global__ void __launch_bounds__(128) gemv_float_kernel(const T* __restrict__ a
                 v = gelu_tanh_f<FAST>(gt) * up;
             } else {
                 v = acc[o][b] + (bias ? bias[n] : 0.0f);
+                if (relu2) v = relu2_f(v);
             }
             if (y32) y32[(long)b * ldy + n] = v;
             else yt[(long)b * ldy + n] = from_f<T>(v);
@@ -139,7 +140,7 @@ __global__ void __launch_bounds__(128) gemv_float_kernel(const T* __restrict__ a
 // index is permuted, the same way on both sides. The warps' partial sums are added in warp order.
 template <int NT, int RT, bool GLU>
 __global__ void __launch_bounds__(256) skinny_mma_kernel(const bf16* __restrict__ a, long lda, const bf16* __restrict__ w, long ldw,
-                                                         const float* __restrict__ bias, int M, int N, int kv, float* y32, bf16* y16, long ldy) {
+                                                         const float* __restrict__ bias, int M, int N, int kv, int relu2, float* y32, bf16* y16, long ldy) {
     constexpr int G = NT * RT >= 4 ? 2 : 4;                 // 32-element chunks per step
     __shared__ float part[8][RT * 16][NT * 8 + 1];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, lr = lane >> 2, lc = lane & 3;
@@ -209,28 +210,29 @@ __global__ void __launch_bounds__(256) skinny_mma_kernel(const bf16* __restrict_
     for (int i = threadIdx.x; i < OUT * M; i += 256) {
         const int tok = i / OUT, o = i - tok * OUT;
         if (n0 + o >= n_out) continue;
-        const float v = GLU ? gelu_tanh_f<true>(total(o, tok)) * total(RT * 16 - 16 + o, tok) : total(o, tok);
+        float v = GLU ? gelu_tanh_f<true>(total(o, tok)) * total(RT * 16 - 16 + o, tok) : total(o, tok);
+        if (!GLU && relu2) v = relu2_f(v);
         if (y32) y32[(long)tok * ldy + n0 + o] = v;
         else y16[(long)tok * ldy + n0 + o] = __float2bfloat16_rn(v);
     }
 }
 
 template <int NT>
-int skinny_nt(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st) {
-    const int kv = (K + 7) / 8;
-    if (glu) launch_k(skinny_mma_kernel<NT, 2, true>, dim3((N + 31) / 32), dim3(256), 0, st, a, lda, w, ldw, bias, M, N, kv, y.f32, (bf16*)y.t, y.ld);
-    else if (N >= 148 * 4 * 16) launch_k(skinny_mma_kernel<NT, 2, false>, dim3((N + 31) / 32), dim3(256), 0, st, a, lda, w, ldw, bias, M, N, kv, y.f32, (bf16*)y.t, y.ld);
-    else launch_k(skinny_mma_kernel<NT, 1, false>, dim3((N + 15) / 16), dim3(256), 0, st, a, lda, w, ldw, bias, M, N, kv, y.f32, (bf16*)y.t, y.ld);
+int skinny_nt(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int act, LinearOut y, cudaStream_t st) {
+    const int kv = (K + 7) / 8, r2 = act == kActRelu2;
+    if (act == kActGeluGate) launch_k(skinny_mma_kernel<NT, 2, true>, dim3((N + 31) / 32), dim3(256), 0, st, a, lda, w, ldw, bias, M, N, kv, r2, y.f32, (bf16*)y.t, y.ld);
+    else if (N >= 148 * 4 * 16) launch_k(skinny_mma_kernel<NT, 2, false>, dim3((N + 31) / 32), dim3(256), 0, st, a, lda, w, ldw, bias, M, N, kv, r2, y.f32, (bf16*)y.t, y.ld);
+    else launch_k(skinny_mma_kernel<NT, 1, false>, dim3((N + 15) / 16), dim3(256), 0, st, a, lda, w, ldw, bias, M, N, kv, r2, y.f32, (bf16*)y.t, y.ld);
     return launch_status();
 }
-int skinny_mma(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st) {
-    if (M <= 8) return skinny_nt<1>(a, lda, w, ldw, bias, M, N, K, glu, y, st);
-    if (M <= 16) return skinny_nt<2>(a, lda, w, ldw, bias, M, N, K, glu, y, st);
-    return skinny_nt<4>(a, lda, w, ldw, bias, M, N, K, glu, y, st);
+int skinny_mma(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int act, LinearOut y, cudaStream_t st) {
+    if (M <= 8) return skinny_nt<1>(a, lda, w, ldw, bias, M, N, K, act, y, st);
+    if (M <= 16) return skinny_nt<2>(a, lda, w, ldw, bias, M, N, K, act, y, st);
+    return skinny_nt<4>(a, lda, w, ldw, bias, M, N, K, act, y, st);
 }
 
 template <class T, int BT, int R, int KS, bool GLU>
-int launch_gemv(const T* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, LinearOut y, cudaStream_t st) {
+int launch_gemv(const T* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int relu2, LinearOut y, cudaStream_t st) {
     const int kv = (K + 7) / 8;
     const size_t smem = (size_t)BT * kv * 8 * sizeof(T);
     auto kern = gemv_float_kernel<T, BT, R, KS, GLU>;
@@ -238,20 +240,21 @@ int launch_gemv(const T* a, long lda, const bf16* w, long ldw, const float* bias
     if (smem > 48 * 1024) FLEXLLM_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     const int n_out = GLU ? N / 2 : N, out = GLU ? R / 2 : R;
     const int per_cta = KS == 1 ? 4 * out : out;
-    launch_k(kern, dim3((n_out + per_cta - 1) / per_cta), dim3(128), smem, st, a, lda, w, ldw, bias, M, n_out, kv, y.f32, (T*)y.t, y.ld);
+    launch_k(kern, dim3((n_out + per_cta - 1) / per_cta), dim3(128), smem, st, a, lda, w, ldw, bias, M, n_out, kv, relu2, y.f32, (T*)y.t, y.ld);
     return launch_status();
 }
 
 template <class T, int BT, bool GLU>
-int gemv_bt(const T* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, LinearOut y, cudaStream_t st) {
-    if (N >= 148 * 4 * 4 * 4) return launch_gemv<T, BT, 4, 1, GLU>(a, lda, w, ldw, bias, M, N, K, y, st);
-    if (N / 2 < 148 * 16 && K >= 1024) return launch_gemv<T, BT, 2, 4, GLU>(a, lda, w, ldw, bias, M, N, K, y, st);
-    return launch_gemv<T, BT, 2, 1, GLU>(a, lda, w, ldw, bias, M, N, K, y, st);
+int gemv_bt(const T* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int relu2, LinearOut y, cudaStream_t st) {
+    if (N >= 148 * 4 * 4 * 4) return launch_gemv<T, BT, 4, 1, GLU>(a, lda, w, ldw, bias, M, N, K, relu2, y, st);
+    if (N / 2 < 148 * 16 && K >= 1024) return launch_gemv<T, BT, 2, 4, GLU>(a, lda, w, ldw, bias, M, N, K, relu2, y, st);
+    return launch_gemv<T, BT, 2, 1, GLU>(a, lda, w, ldw, bias, M, N, K, relu2, y, st);
 }
 
 template <class T>               // M <= 4 (bf16: M <= 2, more goes to the MMA forms)
-int gemv_any(const T* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st) {
-#define FLEXLLM_GEMV(BT_) return glu ? gemv_bt<T, BT_, true>(a, lda, w, ldw, bias, M, N, K, y, st) : gemv_bt<T, BT_, false>(a, lda, w, ldw, bias, M, N, K, y, st)
+int gemv_any(const T* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int act, LinearOut y, cudaStream_t st) {
+#define FLEXLLM_GEMV(BT_) return act == kActGeluGate ? gemv_bt<T, BT_, true>(a, lda, w, ldw, bias, M, N, K, 0, y, st) \
+                                                     : gemv_bt<T, BT_, false>(a, lda, w, ldw, bias, M, N, K, act == kActRelu2, y, st)
     if (M <= 1) FLEXLLM_GEMV(1);
     if (sizeof(T) == 2 || M <= 2) FLEXLLM_GEMV(2);
     FLEXLLM_GEMV(sizeof(T) == 2 ? 2 : 4);
@@ -261,7 +264,7 @@ int gemv_any(const T* a, long lda, const bf16* w, long ldw, const float* bias, i
 // 32-bit mode, any M: 64 x 64 tile, 4 x 4 values per thread (columns 16 apart, so a thread of a gated layer holds the gate and
 // up values of its outputs), fp32 fused multiply-adds in increasing k.
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__ a, long lda, const bf16* __restrict__ w, long ldw,
-                                                       const float* __restrict__ bias, int M, int N, int K, int glu, float* __restrict__ y,
+                                                       const float* __restrict__ bias, int M, int N, int K, int act, float* __restrict__ y,
                                                        long ldy) {
     __shared__ float as[16][65], ws[16][65];
     pdl_sync();
@@ -291,7 +294,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
     for (int i = 0; i < 4; i++) {
         const int m = m0 + ty + 16 * i;
         if (m >= M) continue;
-        if (glu) {
+        if (act == kActGeluGate) {
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
                 const int rg = n0 + tx + 16 * j, ru = rg + 16;
@@ -304,13 +307,18 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* __restrict__
 #pragma unroll
             for (int j = 0; j < 4; j++) {
                 const int n = n0 + tx + 16 * j;
-                if (n < N) y[(long)m * ldy + n] = acc[i][j] + (bias ? bias[n] : 0.0f);
+                if (n < N) {
+                    const float v = acc[i][j] + (bias ? bias[n] : 0.0f);
+                    y[(long)m * ldy + n] = act == kActRelu2 ? relu2_f(v) : v;
+                }
             }
         }
     }
 }
 
-int check(const void* a, long lda, const void* w, long ldw, int M, int N, int K, bool glu, const LinearOut& y) {
+int check(const void* a, long lda, const void* w, long ldw, int M, int N, int K, int act, const LinearOut& y) {
+    const bool glu = act == kActGeluGate;
+    FLEXLLM_REQUIRE(act >= kActNone && act <= kActRelu2);
     FLEXLLM_REQUIRE(a && w && (y.f32 || y.t) && M >= 0 && N > 0 && K > 0);
     FLEXLLM_REQUIRE(lda % 8 == 0 && ldw % 8 == 0 && lda >= up_to(K, 8) && ldw >= up_to(K, 8) && aligned(a, 16) && aligned(w, 16));
     FLEXLLM_REQUIRE(!glu || N % 32 == 0);
@@ -320,30 +328,30 @@ int check(const void* a, long lda, const void* w, long ldw, int M, int N, int K,
 
 }  // namespace
 
-int linear_bf16(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st) {
-    TRY_RC(check(a, lda, w, ldw, M, N, K, glu, y));
+int linear_bf16(const bf16* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int act, LinearOut y, cudaStream_t st) {
+    TRY_RC(check(a, lda, w, ldw, M, N, K, act, y));
     if (M == 0) return FLEXLLM_OK;
     // Measured on the layer shapes of 1B to 8B models: the scalar GEMV wins for one token (two for wide matrices), the
     // tensor-core form where its 128-row tiles alone fill most SMs, the warp-MMA form for the narrow rest.
     const bool wide = (N + 127) / 128 >= 100;
     if ((M == 1 && K <= 12288) || (M == 2 && wide)) {
-        const int rc = gemv_any<bf16>(a, lda, w, ldw, bias, M, N, K, glu, y, st);
+        const int rc = gemv_any<bf16>(a, lda, w, ldw, bias, M, N, K, act, y, st);
         if (rc != FLEXLLM_ENOTSUP) return rc;
     }
-    if (M <= 16 ? !wide : M <= 32 && !wide && (long)N * K <= (17L << 20)) return skinny_mma(a, lda, w, ldw, bias, M, N, K, glu, y, st);
-    if (M <= 64) return gemm_bf16_decode(a, lda, w, ldw, bias, M, N, K, glu, y, st);
-    return gemm_bf16_prefill(a, lda, w, ldw, bias, M, N, K, glu, y, st);
+    if (M <= 16 ? !wide : M <= 32 && !wide && (long)N * K <= (17L << 20)) return skinny_mma(a, lda, w, ldw, bias, M, N, K, act, y, st);
+    if (M <= 64) return gemm_bf16_decode(a, lda, w, ldw, bias, M, N, K, act, y, st);
+    return gemm_bf16_prefill(a, lda, w, ldw, bias, M, N, K, act, y, st);
 }
 
-int linear_f32(const float* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, bool glu, LinearOut y, cudaStream_t st) {
-    TRY_RC(check(a, lda, w, ldw, M, N, K, glu, y));
+int linear_f32(const float* a, long lda, const bf16* w, long ldw, const float* bias, int M, int N, int K, int act, LinearOut y, cudaStream_t st) {
+    TRY_RC(check(a, lda, w, ldw, M, N, K, act, y));
     if (M == 0) return FLEXLLM_OK;
     if (M <= 4) {
-        const int rc = gemv_any<float>(a, lda, w, ldw, bias, M, N, K, glu, y, st);
+        const int rc = gemv_any<float>(a, lda, w, ldw, bias, M, N, K, act, y, st);
         if (rc != FLEXLLM_ENOTSUP) return rc;
     }
     float* out = y.f32 ? y.f32 : (float*)y.t;
-    launch_k(gemm_f32_kernel, dim3((N + 63) / 64, (M + 63) / 64), dim3(256), 0, st, a, lda, w, ldw, bias, M, N, K, glu ? 1 : 0, out, y.ld);
+    launch_k(gemm_f32_kernel, dim3((N + 63) / 64, (M + 63) / 64), dim3(256), 0, st, a, lda, w, ldw, bias, M, N, K, act, out, y.ld);
     return launch_status();
 }
 
@@ -353,10 +361,10 @@ using namespace flexllm;
 
 // See include/flexllm_b200.h.
 extern "C" int flexllm_linear_float(int dtype, const void* a, long lda, const void* w, long ldw, const float* bias, int M, int N, int K,
-                                    int gelu_gate, void* y, long ldy, int y_f32, void* stream) {
+                                    int act, void* y, long ldy, int y_f32, void* stream) {
     FLEXLLM_REQUIRE(dtype == FLEXLLM_F32 || dtype == FLEXLLM_BF16);
     LinearOut o = {y_f32 || dtype == FLEXLLM_F32 ? (float*)y : nullptr, y_f32 || dtype == FLEXLLM_F32 ? nullptr : y, ldy};
     if (dtype == FLEXLLM_BF16)
-        return linear_bf16((const bf16*)a, lda, (const bf16*)w, ldw, bias, M, N, K, gelu_gate != 0, o, (cudaStream_t)stream);
-    return linear_f32((const float*)a, lda, (const bf16*)w, ldw, bias, M, N, K, gelu_gate != 0, o, (cudaStream_t)stream);
+        return linear_bf16((const bf16*)a, lda, (const bf16*)w, ldw, bias, M, N, K, act, o, (cudaStream_t)stream);
+    return linear_f32((const float*)a, lda, (const bf16*)w, ldw, bias, M, N, K, act, o, (cudaStream_t)stream);
 }

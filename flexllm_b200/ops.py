@@ -232,13 +232,13 @@ def dec_Sampling_Layer(logits, rnd, lanes=32, top_k=5, details=False):
 
 
 # ------------------------------------------------------------------------------ floating-point path
-def linear_float(a, w, bias=None, K=None, gelu_gate=False, out_f32=False):
-    """a [M,lda] bf16 or fp32, w [N,ldw] bf16 (columns from K on zero) -> [M,N] (gelu_gate: [M,N/2])."""
+def linear_float(a, w, bias=None, K=None, gelu_gate=False, out_f32=False, relu2=False):
+    """a [M,lda] bf16 or fp32, w [N,ldw] bf16 (columns from K on zero) -> [M,N] (gelu_gate: [M,N/2]; relu2: squared ReLU)."""
     M, N = a.shape[0], w.shape[0]
     dt = _lib.BF16 if a.dtype == torch.bfloat16 else _lib.F32
     y = torch.empty((M, N // 2 if gelu_gate else N), dtype=torch.float32 if out_f32 else a.dtype, device=a.device)
     _call("flexllm_linear_float", dt, _ptr(a), a.shape[1], _ptr(w), w.shape[1], _ptr(bias), M, N, a.shape[1] if K is None else K,
-          1 if gelu_gate else 0, _ptr(y), y.shape[1], 1 if out_f32 else 0)
+          1 if gelu_gate else 2 if relu2 else 0, _ptr(y), y.shape[1], 1 if out_f32 else 0)
     return y
 
 

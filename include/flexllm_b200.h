@@ -378,12 +378,12 @@ FLEXLLM_API int flexllm_model_set_trace(flexllm_model* m, float* trace, size_t f
 
 /* Operators of that family.
  * linear_float: y[m][n] = sum_k a[m][k] w[n][k] (+ bias[n]); a of type dtype [M][lda], w bf16 [N][ldw], lda and ldw multiples of 8
- * and >= K rounded up to 8 (w zero and a finite from K on). gelu_gate: the rows of w alternate in blocks of 16 gate and 16 up
- * rows, y[m][f] = gelu_tanh(gate) * up, N = 2 F, N % 32 == 0. y of type dtype, or fp32 (y_f32).
+ * and >= K rounded up to 8 (w zero and a finite from K on). act 0: none; 1: the rows of w alternate in blocks of 16 gate and 16 up
+ * rows, y[m][f] = gelu_tanh(gate) * up, N = 2 F, N % 32 == 0; 2: y = max(y, 0)^2. y of type dtype, or fp32 (y_f32).
  * sandwich_norm: x += y / rms(y) * gain_post (y NULL: nothing); x += add_vec; h (type dtype) = x / rms(x) * gain_pre. Rows are
  * padded with zeros to multiples of 4. */
 FLEXLLM_API int flexllm_linear_float(int dtype, const void* a, long lda, const void* w, long ldw, const float* bias, int M, int N, int K,
-                                     int gelu_gate, void* y, long ldy, int y_f32, void* stream);
+                                     int act, void* y, long ldy, int y_f32, void* stream);
 FLEXLLM_API int flexllm_sandwich_norm(int dtype, float* x, long ldx, int M, int D, float eps, const float* y, long ldy, const float* gain_post,
                                       const float* add_vec, const float* gain_pre, void* h, long ldh, void* stream);
 
