@@ -119,6 +119,54 @@ struct ResNormArgs {
 };
 template <class T> int res_norm(const ResNormArgs& a, int rows, cudaStream_t st);
 
+// The same place in a model whose residual is a set of n streams mixed around every sublayer (hyper-connections), every step
+// optional:
+//   x_s (or the embedding of the row's token, in every stream) -> x_t <- sum_s mix[s][t] x_s + out[t] y -> [trace: sum of the streams]
+//   -> x stored -> h = rms(u) * gain, u = sum_s in[s] x_s
+constexpr int kMaxStreams = 8;
+struct HyperNormArgs {
+    float* x; long lds; int n, D; float eps;   // x [row][n][lds]
+    const int32_t* rows;                    // row r of the launch is row rows[r] of x (nullptr: r)
+    const int32_t* tok; int S, c0, Sc;      // token of row r: tok[(r / Sc) * S + c0 + r % Sc] ...
+    const bf16* emb; long lde; float emb_scale; int V; int* error_flag;      // ... when emb is given
+    const float* y; long ldy;               // sublayer output, nullptr: none
+    const float *mix, *out;                 // [n][n] (from, to), [n]
+    float* trace;                           // dense [rows][D]
+    const float* in;                        // [n]
+    const float* gain; void* h; long ldh;
+};
+template <class T> int hyper_norm(const HyperNormArgs& a, int rows, cudaStream_t st);
+
+// ---------------------------------------------------------------------------- state-space mixer (Mamba-2 form)
+// Between the projections: causal convolution and silu on x | B | C, recurrence per head, gate, grouped norm.
+struct SsmShape {
+    int H, P, N, G, taps, parts;            // heads, value size, state size, groups of B and C, convolution taps, parts of the norm
+    int P8, N8, Np;                         // sizes padded to 8 (per head / group: columns of the projection) and to 4 (state rows)
+    int inner, ch;                          // H * P8; channels of the convolution: inner + 2 G N8, in the order x | B | C
+    int x_off, dt_off;                      // columns of the fused projection: z 0.., x | B | C x_off.., dt dt_off..
+    long ld;                                // its row length
+};
+struct SsmCall {
+    SsmShape s;
+    const void* proj;                       // T [rows][s.ld]
+    const float *conv_w, *conv_b;           // [taps][ch] (last row: the current token), [ch]; 0 in the padding
+    const float *dt_bias, *A, *D;           // [H]; A = -exp(A_log)
+    const float* gain; float eps;           // [inner], 0 in the padding
+    float* state;                           // [slot][H][P][Np], zero in the padding
+    void* conv_state;                       // T [slot][taps][ch]: inputs of the convolution, position p in row p % taps
+    const int32_t* ctx;                     // position of the first of the call's Sc tokens per sequence (0: the state starts at zero)
+    int B, Sc;
+    void* xbc;                              // scratch T [rows][ch] (unused by the decode form)
+    void* y;                                // scratch T [rows][inner]: gated outputs before the norm
+    void* out;                              // T [rows][inner]
+};
+// Sc == 1: convolution, state update and gate in one kernel; else convolution, then the recurrence (bf16: in chunks on the tensor
+// cores, fp32: token by token). Then the norm. States and histories of the call's sequences are advanced.
+template <class T> int ssm_mixer(const SsmCall& c, cudaStream_t st);
+void ssm_layout(SsmShape* s);               // fills in the derived members
+bool ssm_supported(const SsmShape& s);
+inline size_t ssm_state_floats(const SsmShape& s) { return (size_t)s.H * s.P * s.Np; }
+
 // ---------------------------------------------------------------------------- windowed attention
 constexpr int kBiasPad = 192;               // masked (-inf) distances on either side of the window in the bias tables
 struct AttnShape {
