@@ -84,11 +84,17 @@ SIGNATURES = {
     "flexllm_model_set_trace": [_P, _P, _SZ],
     "flexllm_linear_float": [_I, _P, _L, _P, _L, _P, _I, _I, _I, _I, _P, _L, _I, _P],
     "flexllm_sandwich_norm": [_I, _P, _L, _I, _I, _F, _P, _L, _P, _P, _P, _P, _L, _P],
+    "flexllm_hyper_norm": [_I, _P, _L, _I, _I, _I, _F, _P, _L, _P, _P, _P, _P, _P, _L, _P],
+    "flexllm_ssm_row": [_P],
+    "flexllm_ssm_channels": [_P],
+    "flexllm_ssm_state_floats": [_P],
+    "flexllm_ssm_workspace": [_P, _I, _I],
+    "flexllm_ssm": [_I] + [_P] * 11 + [_I, _I, _P, _P, _SZ, _P],
     "flexllm_attn_window_row": [_P],
     "flexllm_attn_window_bias_floats": [_P],
     "flexllm_attn_window_bias": [_P, _P, _I, _I, _P, _P],
     "flexllm_attn_window_workspace": [_P, _I, _I],
-    "flexllm_attn_window": [_I, _P, _I, _P, _P, _P, _P, _P, _F, _P, _I, _P, _I, _I, _I, _P, _L, _P, _SZ, _P],
+    "flexllm_attn_window": [_I, _P, _I, _P, _P, _P, _P, _P, _F, _P, _P, _I, _P, _I, _I, _I, _P, _L, _P, _SZ, _P],
     "flexllm_hmt_create": [_P, _P, _P, _I, _P, _P, _P],
     "flexllm_hmt_destroy": [_P],
     "flexllm_hmt_prefill": [_P, _P, _I, _P, _P, _P],
@@ -125,7 +131,11 @@ class KvShape(C.Structure):
 
 class AttnWindowShape(C.Structure):
     _fields_ = [("heads", _I), ("kv_heads", _I), ("dim", _I), ("vdim", _I), ("window", _I), ("sink", _I), ("gate", _I), ("scale", _F),
-                ("softcap", _F), ("eps", _F)]
+                ("softcap", _F), ("eps", _F), ("keep_first", _I), ("shared_kv", _I)]
+
+
+class SsmShape(C.Structure):
+    _fields_ = [("heads", _I), ("vdim", _I), ("state", _I), ("groups", _I), ("conv", _I), ("norm_groups", _I), ("eps", _F)]
 
 
 class CkptLayerBuffers(C.Structure):
@@ -143,7 +153,8 @@ class LayerWeights(C.Structure):
 
 RESTYPES = {"flexllm_status_string": C.c_char_p, "flexllm_launch_count": C.c_ulonglong, "flexllm_mha_prefill_workspace": C.c_size_t,
             "flexllm_mha_decode_workspace": C.c_size_t, "flexllm_mlp_block_workspace": C.c_size_t,
-            "flexllm_attn_window_row": C.c_long, "flexllm_attn_window_bias_floats": C.c_size_t, "flexllm_attn_window_workspace": C.c_size_t}
+            "flexllm_attn_window_row": C.c_long, "flexllm_ssm_row": C.c_long, "flexllm_ssm_channels": C.c_long,
+            "flexllm_ssm_state_floats": C.c_size_t, "flexllm_ssm_workspace": C.c_size_t, "flexllm_attn_window_bias_floats": C.c_size_t, "flexllm_attn_window_workspace": C.c_size_t}
 
 
 def load():

@@ -1056,8 +1056,9 @@ bool make_shape(const flexllm_attn_window_shape* a, AttnShape* s) {
     if (!a || a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads || a->dim <= 0 || a->vdim <= 0 || a->window <= 0) return false;
     *s = AttnShape();
     s->H = a->heads; s->G = a->kv_heads; s->dk = a->dim; s->dv = a->vdim; s->window = a->window;
-    s->scale = a->scale; s->softcap = a->softcap; s->sink = a->sink ? 1 : 0;
-    attn_layout(s, a->gate != 0);
+    if (a->sink < 0 || a->sink > 2 || a->keep_first < 0) return false;
+    s->scale = a->scale; s->softcap = a->softcap; s->sink = a->sink; s->keep = a->keep_first;
+    attn_layout(s, a->gate != 0, !a->shared_kv);
     return true;
 }
 struct WindowWs { size_t ws_floats, counters, q, total; };      // byte offsets of the counters and of the q scratch
@@ -1086,8 +1087,8 @@ extern "C" int flexllm_attn_window_bias(const flexllm_attn_window_shape* a, cons
     return cuda_status(cudaStreamSynchronize((cudaStream_t)stream));
 }
 extern "C" int flexllm_attn_window(int dtype, flexllm_kv_cache* kv, int layer, const flexllm_attn_window_shape* a, const void* proj,
-                                   const float* q_gain, const float* k_gain, const float* bias, float bias_abs, const int32_t* page_table,
-                                   int max_pages, const int32_t* ctx, int max_ctx, int B, int n, void* out, long ldo, void* workspace,
+                                   const float* q_gain, const float* k_gain, const float* bias, float bias_abs, const float* sinks,
+                                   const int32_t* page_table, int max_pages, const int32_t* ctx, int max_ctx, int B, int n, void* out, long ldo, void* workspace,
                                    size_t workspace_bytes, void* stream) {
     AttnCall c = {};
     FLEXLLM_REQUIRE(make_shape(a, &c.s) && kv && layer >= 0 && layer < kv->layers && B > 0 && n > 0);
@@ -1097,7 +1098,7 @@ extern "C" int flexllm_attn_window(int dtype, flexllm_kv_cache* kv, int layer, c
     FLEXLLM_REQUIRE(ks.hkv == c.s.G && ks.kdim == c.s.dkp && ks.vdim == c.s.dv && ldo >= (long)c.s.H * c.s.dv);
     const WindowWs w = window_ws(c.s, B, n);
     FLEXLLM_REQUIRE(workspace && aligned(workspace, 256) && workspace_bytes >= w.total && aligned(proj, 16) && aligned(out, 16));
-    c.proj = proj; c.q_gain = q_gain; c.k_gain = k_gain; c.eps = a->eps; c.bias = bias; c.bias_max_abs = bias_abs;
+    c.proj = proj; c.q_gain = q_gain; c.k_gain = k_gain; c.eps = a->eps; c.bias = bias; c.bias_max_abs = bias_abs; c.sinks = sinks;
     c.k_pool = kv->k + kv->k_off[layer]; c.v_pool = kv->v + kv->v_off[layer]; c.n_pages = kv->n_pages;
     c.page_table = page_table; c.max_pages = max_pages; c.ctx = ctx; c.max_pos = max_ctx; c.B = B; c.Sc = n;
     c.ws = (float*)workspace; c.ws_floats = w.ws_floats; c.counters = (int*)((char*)workspace + w.counters); c.n_counters = B * c.s.G;

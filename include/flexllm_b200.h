@@ -381,29 +381,56 @@ FLEXLLM_API int flexllm_model_set_trace(flexllm_model* m, float* trace, size_t f
  * and >= K rounded up to 8 (w zero and a finite from K on). act 0: none; 1: the rows of w alternate in blocks of 16 gate and 16 up
  * rows, y[m][f] = gelu_tanh(gate) * up, N = 2 F, N % 32 == 0; 2: y = max(y, 0)^2. y of type dtype, or fp32 (y_f32).
  * sandwich_norm: x += y / rms(y) * gain_post (y NULL: nothing); x += add_vec; h (type dtype) = x / rms(x) * gain_pre. Rows are
- * padded with zeros to multiples of 4. */
+ * padded with zeros to multiples of 4.
+ * hyper_norm: x [M][streams][lds] fp32 residual streams; x_t <- sum_s mix[s][t] x_s + out[t] y (y NULL: nothing), then h (type dtype) =
+ * u / rms(u) * gain with u = sum_s in[s] x_s (gain NULL: nothing). mix [streams][streams] (from, to), out, in [streams], gain [D]:
+ * device fp32; streams <= 8; rows of x, y and h padded with zeros to multiples of 4. */
 FLEXLLM_API int flexllm_linear_float(int dtype, const void* a, long lda, const void* w, long ldw, const float* bias, int M, int N, int K,
                                      int act, void* y, long ldy, int y_f32, void* stream);
 FLEXLLM_API int flexllm_sandwich_norm(int dtype, float* x, long ldx, int M, int D, float eps, const float* y, long ldy, const float* gain_post,
                                       const float* add_vec, const float* gain_pre, void* h, long ldh, void* stream);
 
+FLEXLLM_API int flexllm_hyper_norm(int dtype, float* x, long lds, int streams, int M, int D, float eps, const float* y, long ldy, const float* mix,
+                                   const float* out, const float* in, const float* gain, void* h, long ldh, void* stream);
+
+/* State-space mixer (the Mamba-2 form) between its projections, B sequences x n new tokens at positions ctx[b]..:
+ *   x | B | C <- silu(causal convolution with conv taps + bias);  dt <- softplus(dt + dt_bias)
+ *   S_t = exp(A dt) S_{t-1} + dt B_t x_t^T,  y_t = S_t^T C_t + D x_t   per head (head h: group h / (heads / groups))
+ *   out = (y * silu(z)) / rms, in norm_groups equal parts, * gain
+ * proj [B*n][flexllm_ssm_row]: z [heads][P8] | x [heads][P8] | B [groups][N8] | C [groups][N8] | dt [heads], with P8, N8 = vdim and
+ * state rounded up to 8 (padding: zeros) and dt padded to 8. conv_w [conv][channels], conv_b [channels] over x | B | C (channels =
+ * flexllm_ssm_channels, last row of conv_w: the current token), A, D, dt_bias [heads], gain [heads][P8]: device fp32, zero in the
+ * padding. state [slots][flexllm_ssm_state_floats] fp32 and conv_state [slots][conv][channels] of type dtype belong to the
+ * sequences and are advanced; sequence b uses slot b and starts from zero where ctx[b] is 0. state <= 256. out [B*n][heads * P8]. */
+typedef struct { int heads, vdim, state, groups, conv, norm_groups; float eps; } flexllm_ssm_shape;
+FLEXLLM_API long flexllm_ssm_row(const flexllm_ssm_shape* s);
+FLEXLLM_API long flexllm_ssm_channels(const flexllm_ssm_shape* s);
+FLEXLLM_API size_t flexllm_ssm_state_floats(const flexllm_ssm_shape* s);
+FLEXLLM_API size_t flexllm_ssm_workspace(const flexllm_ssm_shape* s, int B, int n);
+FLEXLLM_API int flexllm_ssm(int dtype, const flexllm_ssm_shape* s, const void* proj, const float* conv_w, const float* conv_b, const float* dt_bias,
+                            const float* A, const float* D, const float* gain, float* state, void* conv_state, const int32_t* ctx, int B, int n,
+                            void* out, void* workspace, size_t workspace_bytes, void* stream);
+
 /* Windowed grouped-query attention on one layer of a floating-point cache, B sequences x n new tokens at positions ctx[b]..:
  *   q, k = rms norm of the whole q (k) projection * gain;  s = softcap * tanh(scale * (q . k) / softcap) + bias[head][i - j]
- *   for 0 <= i - j < window;  p = exp(s) / (sink + sum exp(s));  out = (sum p v) * logistic(gate)
+ *   for 0 <= i - j < window or 0 <= j < keep_first, j <= i;  p = exp(s) / (sink + sum exp(s));  out = (sum p v) * logistic(gate)
+ * q_gain and k_gain NULL: no norms; bias NULL: none (needed with keep_first); softcap 0: none; sink 0: none, 1: a score of 0,
+ * 2: exp(sinks[head]), sinks [heads] device fp32. shared_kv: proj has no k and v parts, the layer's keys and values up to the
+ * call's positions are in the cache already and nothing is appended.
  * The new keys and values are appended to the cache first. proj: rows of q | k | v | gate, each part padded to a multiple of 8
  * columns, row length flexllm_attn_window_row(shape) (gate 0: no gate part); cache element type = dtype, kdim = dim rounded up
  * to 8. bias: flexllm_attn_window_bias_floats(shape) floats in device memory made by flexllm_attn_window_bias from a table
  * [rows][heads] in host memory: distance d < rows/2 uses row d, larger ones min(rows-1, rows/2 + floor(ln(d/(rows/2)) /
  * ln(bias_max/(rows/2)) * (rows - rows/2))); bias_abs: its largest magnitude. max_ctx: largest position the page table covers.
  * out [B*n][ldo] of type dtype, ldo >= heads * vdim. n == 1 is the decode form. */
-typedef struct { int heads, kv_heads, dim, vdim, window, sink, gate; float scale, softcap, eps; } flexllm_attn_window_shape;
+typedef struct { int heads, kv_heads, dim, vdim, window, sink, gate; float scale, softcap, eps; int keep_first, shared_kv; } flexllm_attn_window_shape;
 FLEXLLM_API long flexllm_attn_window_row(const flexllm_attn_window_shape* s);
 FLEXLLM_API size_t flexllm_attn_window_bias_floats(const flexllm_attn_window_shape* s);
 FLEXLLM_API int flexllm_attn_window_bias(const flexllm_attn_window_shape* s, const float* table_host, int rows, int bias_max, float* bias,
                                          void* stream);
 FLEXLLM_API size_t flexllm_attn_window_workspace(const flexllm_attn_window_shape* s, int B, int n);
 FLEXLLM_API int flexllm_attn_window(int dtype, flexllm_kv_cache* c, int layer, const flexllm_attn_window_shape* s, const void* proj,
-                                    const float* q_gain, const float* k_gain, const float* bias, float bias_abs,
+                                    const float* q_gain, const float* k_gain, const float* bias, float bias_abs, const float* sinks,
                                     const int32_t* page_table, int max_pages, const int32_t* ctx, int max_ctx, int B, int n, void* out,
                                     long ldo, void* workspace, size_t workspace_bytes, void* stream);
 
