@@ -6,6 +6,9 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.environ.get("FLEXLLM_B200_LIB") or os.path.join(_HERE, "libflexllm_b200.so")   # the override is a development aid
 
 F32, BF16 = 0, 1
+MIXER_ATTENTION, MIXER_SSM = 0, 1
+ATTN_HEAD_SINKS, ATTN_PIBIDRA = 32, 31
+FF_GELU_GATE, FF_RELU2 = 1, 2
 OK, EINVAL, ECUDA, ETIMEDOUT, ENOTSUP, ENOMEM, ETOOBIG, EDEVDATA, EIO = 0, -1, -2, -3, -4, -5, -6, -7, -8
 
 # name -> argument types, in the order of include/flexllm_b200.h (return type is int unless noted)
@@ -117,12 +120,14 @@ class ModelConfig(C.Structure):
 
 class DecoderLayer(C.Structure):
     _fields_ = [("heads", _I), ("kv_heads", _I), ("dim", _I), ("vdim", _I), ("window", _I), ("bias_max", _I), ("scale", _F), ("softcap", _F),
-                ("ff", _I)]
+                ("ff", _I), ("mixer", _I), ("features", _I), ("act", _I), ("keep_first", _I), ("kv_from", _I), ("state", _I), ("groups", _I),
+                ("conv", _I), ("norm_groups", _I)]
 
 
 class DecoderConfig(C.Structure):
     _fields_ = [("layers", _I), ("width", _I), ("vocab", _I), ("eps", _F), ("embed_scale", _F), ("loop_start", _I), ("loop_stop", _I),
-                ("loop_times", _I), ("max_batch", _I), ("max_prefill", _I), ("max_ctx", _I), ("dtype", _I), ("layer", C.POINTER(DecoderLayer))]
+                ("loop_times", _I), ("max_batch", _I), ("max_prefill", _I), ("max_ctx", _I), ("dtype", _I), ("layer", C.POINTER(DecoderLayer)),
+                ("streams", _I), ("residual_mult", _F), ("logit_scale", _F)]
 
 
 class KvShape(C.Structure):

@@ -363,7 +363,7 @@ extern "C" int flexllm_kv_cache_create(flexllm_kv_cache** out, int layers, int n
 // Floating-point flavour: one pool pair per layer, each with its own shape (256-byte aligned inside two allocations).
 extern "C" int flexllm_kv_cache_create_float(flexllm_kv_cache** out, int layers, int n_pages, const flexllm_kv_shape* shapes, int page,
                                              int elem_bytes) {
-    FLEXLLM_REQUIRE(out && layers > 0 && n_pages > 0 && shapes && (elem_bytes == 2 || elem_bytes == 4));
+    FLEXLLM_REQUIRE(out && layers >= 0 && n_pages > 0 && (shapes || layers == 0) && (elem_bytes == 2 || elem_bytes == 4));
     if (page != PAGE) return FLEXLLM_ENOTSUP;
     for (int l = 0; l < layers; l++) FLEXLLM_REQUIRE(shapes[l].hkv > 0 && shapes[l].kdim > 0 && shapes[l].vdim > 0);
     flexllm_kv_cache* c = new (std::nothrow) flexllm_kv_cache();
@@ -379,8 +379,8 @@ extern "C" int flexllm_kv_cache_create_float(flexllm_kv_cache** out, int layers,
         nv += align_up((size_t)n_pages * shapes[l].hkv * PAGE * shapes[l].vdim * elem_bytes, 256);
     }
     c->k_bytes = nk; c->v_bytes = nv;
-    cudaError_t e = cudaMalloc(&c->k, nk);
-    if (e == cudaSuccess) e = cudaMalloc(&c->v, nv);
+    cudaError_t e = cudaMalloc(&c->k, nk ? nk : 256);
+    if (e == cudaSuccess) e = cudaMalloc(&c->v, nv ? nv : 256);
     if (e != cudaSuccess) {
         flexllm_kv_cache_destroy(c);
         g_last_cuda_error = (int)e;
@@ -390,9 +390,23 @@ extern "C" int flexllm_kv_cache_create_float(flexllm_kv_cache** out, int layers,
     return flexllm_kv_cache_reset(c, nullptr);
 }
 
+int flexllm::kv_cache_add_states(flexllm_kv_cache* c, int slots, const std::vector<size_t>& slot_bytes) {
+    FLEXLLM_REQUIRE(c && !c->states && c->elem_bytes != 1 && slots > 0);
+    size_t n = 0;
+    for (size_t b : slot_bytes) {
+        c->s_off.push_back(n); c->s_slot.push_back(b);
+        n += align_up(b * slots, 256);
+    }
+    c->states_bytes = n;
+    if (n == 0) return FLEXLLM_OK;
+    const cudaError_t e = cudaMalloc(&c->states, n);
+    if (e != cudaSuccess) { g_last_cuda_error = (int)e; return e == cudaErrorMemoryAllocation ? FLEXLLM_ENOMEM : FLEXLLM_ECUDA; }
+    return cuda_status(cudaMemset(c->states, 0, n));
+}
+
 extern "C" int flexllm_kv_cache_destroy(flexllm_kv_cache* c) {
     if (!c) return FLEXLLM_OK;
-    cudaFree(c->k); cudaFree(c->v); cudaFree(c->ks); cudaFree(c->vs);
+    cudaFree(c->k); cudaFree(c->v); cudaFree(c->ks); cudaFree(c->vs); cudaFree(c->states);
     delete c;
     return FLEXLLM_OK;
 }
@@ -403,6 +417,7 @@ extern "C" int flexllm_kv_cache_reset(flexllm_kv_cache* c, void* stream) {
     if (c->elem_bytes != 1) {
         FLEXLLM_CHECK_CUDA(cudaMemsetAsync(c->k, 0, c->k_bytes, st));
         FLEXLLM_CHECK_CUDA(cudaMemsetAsync(c->v, 0, c->v_bytes, st));
+        if (c->states) FLEXLLM_CHECK_CUDA(cudaMemsetAsync(c->states, 0, c->states_bytes, st));
         return FLEXLLM_OK;
     }
     FLEXLLM_CHECK_CUDA(cudaMemsetAsync(c->k, 0, c->page_bytes * c->layers, st));

@@ -118,8 +118,9 @@ using namespace flexllm;
 
 // What every family's runner holds: page table, context lengths, token tables, row list, logits. Sequence b owns pages
 // [b * seq_pages, (b + 1) * seq_pages) and logical page i lies in the (i % seq_pages)-th of them: with seq_pages == max_pages
-// every position has its own slot; fewer make the pages of a sliding-window model a ring.
-static int runner_alloc(flexllm_model* m, int seq_pages) {
+// every position has its own slot; fewer make the pages of a sliding-window model a ring. The first keep_pages logical pages
+// (windows that keep a sequence's first tokens) have their own places and the rest form the ring.
+static int runner_alloc(flexllm_model* m, int seq_pages, int keep_pages = 0) {
     const flexllm_model_config& c = m->cfg;
     TRY(dmalloc(m, &m->page_table, (size_t)c.max_batch * m->max_pages));
     TRY(dmalloc(m, &m->ctx, 64));
@@ -133,7 +134,8 @@ static int runner_alloc(flexllm_model* m, int seq_pages) {
     TRY(dmalloc(m, &m->logits, (size_t)m->logits_rows * c.vocab));
     std::vector<int32_t> pt((size_t)c.max_batch * m->max_pages);
     for (int b = 0; b < c.max_batch; b++)
-        for (int i = 0; i < m->max_pages; i++) pt[(size_t)b * m->max_pages + i] = b * seq_pages + i % seq_pages;
+        for (int i = 0; i < m->max_pages; i++)
+            pt[(size_t)b * m->max_pages + i] = b * seq_pages + (i < keep_pages ? i : keep_pages + (i - keep_pages) % (seq_pages - keep_pages));
     FLEXLLM_CHECK_CUDA(cudaMemcpy(m->page_table, pt.data(), pt.size() * 4, cudaMemcpyHostToDevice));
     return FLEXLLM_OK;
 }
@@ -219,12 +221,12 @@ extern "C" int flexllm_model_create_tp(flexllm_model** out, const flexllm_model_
 
 // A runner around another family: `seq_pages` pages per sequence of a cache the family has created.
 int flexllm::runner_create(flexllm_model** out, const flexllm_model_config& cfg, ModelFamily* fam, flexllm_kv_cache* cache, int seq_pages,
-                           size_t x_floats) {
+                           int keep_pages, size_t x_floats) {
     flexllm_model* m = new (std::nothrow) flexllm_model();
     if (!m) { delete fam; flexllm_kv_cache_destroy(cache); return FLEXLLM_ENOMEM; }
     m->cfg = cfg; m->fam = fam; m->cache = cache;
     m->max_pages = (cfg.max_ctx + 64) / 64;
-    int rc = runner_alloc(m, seq_pages);
+    int rc = runner_alloc(m, seq_pages, keep_pages);
     if (!rc) rc = dmalloc(m, &m->x, x_floats);
     if (!rc) rc = cuda_status(cudaMemset(m->x, 0, x_floats * 4));
     if (!rc) rc = flexllm_model_reset(m, nullptr);

@@ -25,8 +25,10 @@ struct ModelFamily {
     virtual int logits(flexllm_model* m, const int32_t* rows, int n, float* out, cudaStream_t st) = 0;
     virtual int set_trace(float*, size_t) { return FLEXLLM_ENOTSUP; }
 };
-// Takes over fam and cache (also on failure). x_floats: residual stream of the largest chunk.
-int runner_create(flexllm_model** out, const flexllm_model_config& cfg, ModelFamily* fam, flexllm_kv_cache* cache, int seq_pages, size_t x_floats);
+// Takes over fam and cache (also on failure). seq_pages: pages per sequence, of which the first keep_pages stay outside the ring;
+// x_floats: residual stream of the largest chunk.
+int runner_create(flexllm_model** out, const flexllm_model_config& cfg, ModelFamily* fam, flexllm_kv_cache* cache, int seq_pages, int keep_pages,
+                  size_t x_floats);
 }  // namespace flexllm
 
 struct LayerW {

@@ -75,6 +75,20 @@ class HostModel:
         call("flexllm_model_set_sampling_host", self._h, lanes, top_k, (C.c_float * max(1, len(rnd)))(*rnd), n_new, B)
 
 
+# --------------------------------------------------------------------------------------------- decoder family
+ALL = 2 ** 31 - 1       # window of a layer without one
+
+
+def create_decoder(cfg, c_config):
+    h = C.c_void_p()
+    call("flexllm_model_create_decoder", C.byref(h), C.byref(c_config))
+    return HostModel(h, cfg["vocab"])
+
+
+def load_safetensors(model, folder):
+    call("flexllm_model_load_safetensors", model._h, os.path.join(folder, "model.safetensors").encode(), None)
+
+
 # --------------------------------------------------------------------------------------------- Pibidra
 def pibidra_config(cfg, max_batch, max_prefill, max_ctx, dtype):
     """config.json -> (C configuration, the layer array it points to)."""
@@ -87,8 +101,9 @@ def pibidra_config(cfg, max_batch, max_prefill, max_ctx, dtype):
         if f is not None and f.get("kind", "dense") != "dense":
             raise ValueError("layer %d: unknown feed-forward %r" % (i, f["kind"]))
         mask = m.get("mask")
-        layers[i] = _lib.DecoderLayer(m["heads"], m["kv_heads"], m["dim"], m["vdim"], mask["size"] if mask else 2 ** 31 - 1, m["bias_max"],
-                                      m["scale"], m.get("softcap") or 0.0, f["ff"] if f else 0)
+        layers[i] = _lib.DecoderLayer(m["heads"], m["kv_heads"], m["dim"], m["vdim"], mask["size"] if mask else ALL, m["bias_max"],
+                                      m["scale"], m.get("softcap") or 0.0, f["ff"] if f else 0, _lib.MIXER_ATTENTION, _lib.ATTN_PIBIDRA,
+                                      _lib.FF_GELU_GATE, 0, -1)
     loop = cfg.get("loop") or dict(start=0, stop=0, times=0)
     c = _lib.DecoderConfig(n, cfg["width"], cfg["vocab"], cfg["norm"]["eps"], cfg["embedding"]["scale"], loop["start"], loop["stop"],
                            loop["times"], max_batch, max_prefill, max_ctx, dtype, layers)
@@ -103,13 +118,56 @@ class Pibidra:
     @staticmethod
     def create(cfg, max_batch, max_prefill, max_ctx, dtype):
         c, keep = pibidra_config(cfg, max_batch, max_prefill, max_ctx, DTYPES[dtype])
-        h = C.c_void_p()
-        call("flexllm_model_create_decoder", C.byref(h), C.byref(c))
-        return HostModel(h, cfg["vocab"])
+        return create_decoder(cfg, c)
 
     @staticmethod
     def load_weights(model, folder, cfg):
-        call("flexllm_model_load_safetensors", model._h, os.path.join(folder, "model.safetensors").encode(), None)
+        load_safetensors(model, folder)
+
+
+# --------------------------------------------------------------------------------------------- Sabisun
+def sabisun_config(cfg, max_batch, max_prefill, max_ctx, dtype):
+    """config.json -> (C configuration, the layer array it points to)."""
+    n = len(cfg["layers"])
+    layers = (_lib.DecoderLayer * n)()
+    for i, l in enumerate(cfg["layers"]):
+        m, f = l["mixer"], l.get("mlp")
+        if f is not None and f.get("kind", "dense") != "dense":
+            raise ValueError("layer %d: unknown feed-forward %r" % (i, f["kind"]))
+        d = layers[i]
+        d.heads, d.vdim, d.kv_from = m["heads"], m["vdim"], -1
+        d.ff, d.act = f["ff"] if f else 0, _lib.FF_RELU2
+        if l["type"] == "attention":
+            mask = m.get("mask")
+            d.mixer, d.features = _lib.MIXER_ATTENTION, _lib.ATTN_HEAD_SINKS
+            d.kv_heads, d.dim, d.scale = m["kv_heads"], m["dim"], m["scale"]
+            d.window, d.keep_first = (mask["size"], mask.get("keep_first", 0)) if mask else (ALL, 0)
+            if m.get("kv_from") is not None:
+                d.kv_from = m["kv_from"]
+        elif l["type"] == "mamba2":
+            d.mixer = _lib.MIXER_SSM
+            d.state, d.groups, d.conv, d.norm_groups = m["state"], m["groups"], m["conv"], m["norm_groups"]
+        else:
+            raise ValueError("layer %d: unknown mixer %r" % (i, l["type"]))
+    c = _lib.DecoderConfig(n, cfg["width"], cfg["vocab"], cfg["norm"]["eps"], 1.0, 0, 0, 0, max_batch, max_prefill, max_ctx, dtype, layers,
+                           cfg["streams"], cfg["residual_mult"], cfg["logit_scale"])
+    return c, layers
+
+
+class Sabisun:
+    """State-space and windowed-attention layers between mixed residual streams (hyper-connections), squared-ReLU feed-forward,
+    tied embeddings; one .safetensors file."""
+    name = "Sabisun"
+    dtypes = ("bfloat16", "float32")
+
+    @staticmethod
+    def create(cfg, max_batch, max_prefill, max_ctx, dtype):
+        c, keep = sabisun_config(cfg, max_batch, max_prefill, max_ctx, DTYPES[dtype])
+        return create_decoder(cfg, c)
+
+    @staticmethod
+    def load_weights(model, folder, cfg):
+        load_safetensors(model, folder)
 
 
 # --------------------------------------------------------------------------------------------- W8A8 Llama
@@ -153,7 +211,7 @@ class SpinQuantLlama:
         check("flexllm_device_status", lib().flexllm_device_status())
 
 
-REGISTRY = {e.name: e for e in (SpinQuantLlama, Pibidra)}
+REGISTRY = {e.name: e for e in (SpinQuantLlama, Pibidra, Sabisun)}
 
 
 def entry(cfg):

@@ -255,19 +255,26 @@ class WindowAttention:
     """One layer of windowed attention with its own floating-point paged cache (dtype bf16 or fp32).
 
     table [rows,heads] (CPU fp32): learned bias by bucketed distance. Call with proj [B*n, row] (q | k | v | gate, parts padded
-    to multiples of 8 columns), ctx [B] int32 (tokens already cached). Returns [B*n, heads*vdim]."""
+    to multiples of 8 columns), ctx [B] int32 (tokens already cached). Returns [B*n, heads*vdim]. table, q_gain and k_gain may be
+    None; sinks [heads]: learned sink scores; kv_of: the operator whose cache holds the keys and values (proj is q | gate)."""
 
     def __init__(self, heads, kv_heads, dim, vdim, window, scale, softcap, table, bias_max, q_gain, k_gain, page_table, n_pages, max_ctx,
-                 eps=1e-5, sink=True, gate=True, dtype=torch.bfloat16):
-        self.shape = _lib.AttnWindowShape(heads, kv_heads, dim, vdim, window, 1 if sink else 0, 1 if gate else 0, scale, softcap, eps)
+                 eps=1e-5, sink=True, gate=True, dtype=torch.bfloat16, keep_first=0, sinks=None, kv_of=None):
+        self.shape = _lib.AttnWindowShape(heads, kv_heads, dim, vdim, window, 2 if sinks is not None else 1 if sink else 0, 1 if gate else 0, scale,
+                                          softcap, eps, keep_first, 1 if kv_of else 0)
+        self.sinks, self.kv_of = sinks, kv_of
         self.dtype, self.q_gain, self.k_gain, self.page_table, self.max_ctx = dtype, q_gain, k_gain, page_table, max_ctx
         self.row = lib().flexllm_attn_window_row(C.byref(self.shape))
-        self.bias = torch.empty((lib().flexllm_attn_window_bias_floats(C.byref(self.shape)),), dtype=torch.float32, device=q_gain.device)
-        t = table.contiguous()
-        self.bias_abs = float(t.abs().max())
-        _check("flexllm_attn_window_bias", lib().flexllm_attn_window_bias(C.byref(self.shape), C.c_void_p(t.data_ptr()), t.shape[0], bias_max,
-                                                                          _ptr(self.bias), _stream()))
+        self.bias, self.bias_abs = None, 0.0
+        if table is not None:
+            self.bias = torch.empty((lib().flexllm_attn_window_bias_floats(C.byref(self.shape)),), dtype=torch.float32, device=page_table.device)
+            t = table.contiguous()
+            self.bias_abs = float(t.abs().max())
+            _check("flexllm_attn_window_bias", lib().flexllm_attn_window_bias(C.byref(self.shape), C.c_void_p(t.data_ptr()), t.shape[0], bias_max,
+                                                                              _ptr(self.bias), _stream()))
         self._h = C.c_void_p()
+        if kv_of:
+            return
         kv = _lib.KvShape(kv_heads, (dim + 7) // 8 * 8, vdim)
         _check("flexllm_kv_cache_create_float", lib().flexllm_kv_cache_create_float(C.byref(self._h), 1, n_pages, C.byref(kv), 64,
                                                                                     2 if dtype == torch.bfloat16 else 4))
@@ -284,8 +291,8 @@ class WindowAttention:
         out = torch.empty((B * n, self.shape.heads * self.shape.vdim), dtype=self.dtype, device=proj.device)
         nbytes = lib().flexllm_attn_window_workspace(C.byref(self.shape), B, n)
         ws = torch.empty((nbytes,), dtype=torch.uint8, device=proj.device)
-        _call("flexllm_attn_window", _lib.BF16 if self.dtype == torch.bfloat16 else _lib.F32, self._h, 0, C.byref(self.shape), _ptr(proj),
-              _ptr(self.q_gain), _ptr(self.k_gain), _ptr(self.bias), self.bias_abs, _ptr(self.page_table), self.page_table.shape[1],
+        _call("flexllm_attn_window", _lib.BF16 if self.dtype == torch.bfloat16 else _lib.F32, (self.kv_of or self)._h, 0, C.byref(self.shape), _ptr(proj),
+              _ptr(self.q_gain), _ptr(self.k_gain), _ptr(self.bias), self.bias_abs, _ptr(self.sinks), _ptr(self.page_table), self.page_table.shape[1],
               _ptr(ctx), self.max_ctx, B, n, _ptr(out), out.shape[1], _ptr(ws), nbytes)
         return out
 

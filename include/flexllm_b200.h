@@ -342,19 +342,39 @@ FLEXLLM_API int flexllm_model_extend_host(flexllm_model* m, const int32_t* token
 /* Ends the live sequences: their pages are free for the next ones. */
 FLEXLLM_API int flexllm_model_reset(flexllm_model* m, void* stream);
 
-/* Decoder family with floating-point weights (the Pibidra design; no counterpart in the reference). Per layer
+/* Decoder family with floating-point weights (the Pibidra and Sabisun designs; no counterpart in the reference). Pibidra, per layer
  *     x += norm1b(attention(norm1(x)));   x += norm2b(down(gelu_tanh(gate h) * up h)), h = norm2(x)     (ff 0: no second part)
  * with norm(x) = x / sqrt(mean x^2 + eps) * (1 + w); attention: see flexllm_attn_window. Layers loop_start .. loop_stop-1
  * run loop_times times with the same weights (0: no loop); before pass t the vector loop.step[t], and from the second pass
  * on also the embedding output, is added to x. Every layer run has its own cache. The pages of a sequence are a ring that
  * holds the widest window and one chunk of max_prefill tokens, so memory does not grow with max_ctx.
- * dtype FLEXLLM_BF16: bf16 products and activations, fp32 residual stream, norms, scores and softmax; FLEXLLM_F32: all fp32.
+ * Sabisun (streams > 0): the residual is a set of `streams` copies of the embedding output. Around a sublayer f with coefficients
+ * in, out and mix: y = f(norm(sum_s in[s] x_s)), x_t <- sum_s mix[s][t] x_s + residual_mult * out[t] * y, norm(x) = x / rms(x) * w; the
+ * head reads the sum of the streams and uses the embedding table, times logit_scale. Mixers: attention (features 0 with
+ * FLEXLLM_ATTN_HEAD_SINKS; kv_from names the layer whose keys and values it uses), or the state-space mixer of flexllm_ssm, whose
+ * state and convolution history live beside the pages, one slot per sequence. Feed-forward: down(max(up h, 0)^2).
+ * dtype FLEXLLM_BF16: bf16 products and activations, fp32 residual stream, norms, scores, softmax and states; FLEXLLM_F32: all fp32.
  * The model is an ordinary flexllm_model: prefill (any length), begin, decode, generate_host, set_sampling, extend. */
+#define FLEXLLM_MIXER_ATTENTION 0
+#define FLEXLLM_MIXER_SSM 1
+#define FLEXLLM_ATTN_QK_NORM 1            /* norms over the whole q and k projections (mix.q.norm, mix.k.norm) */
+#define FLEXLLM_ATTN_PROJ_BIAS 2          /* biases of q, k and v */
+#define FLEXLLM_ATTN_DISTANCE_BIAS 4      /* mix.rel */
+#define FLEXLLM_ATTN_GATE 8               /* mix.g */
+#define FLEXLLM_ATTN_UNIT_SINK 16         /* a score of 0 in the softmax ... */
+#define FLEXLLM_ATTN_HEAD_SINKS 32        /* ... or one learned score per head (mix.sink) */
+#define FLEXLLM_ATTN_PIBIDRA 31
+#define FLEXLLM_FF_GELU_GATE 1            /* down(gelu_tanh(gate h) * up h) */
+#define FLEXLLM_FF_RELU2 2                /* down(max(up h, 0)^2) */
 typedef struct {
-    int heads, kv_heads, dim, vdim;       /* attention: query heads, key/value heads, query/key size, value size */
+    int heads, kv_heads, dim, vdim;       /* attention: query heads, key/value heads, query/key size, value size; state-space: heads, -, -, value size */
     int window, bias_max;                 /* i sees j with 0 <= i - j < window; distance at which the bias table saturates */
     float scale, softcap;                 /* softcap 0: none */
     int ff;                               /* feed-forward size, 0: none */
+    int mixer, features, act;             /* FLEXLLM_MIXER_*, FLEXLLM_ATTN_* bits, FLEXLLM_FF_* */
+    int keep_first;                       /* i also sees every j < keep_first */
+    int kv_from;                          /* layer whose keys and values this one uses, -1: its own */
+    int state, groups, conv, norm_groups; /* state-space: state size, groups of B and C, convolution taps, parts of the norm */
 } flexllm_decoder_layer;
 typedef struct {
     int layers, width, vocab;
@@ -363,10 +383,13 @@ typedef struct {
     int max_batch, max_prefill, max_ctx;
     int dtype;
     const flexllm_decoder_layer* layer;   /* [layers] */
+    int streams;                          /* 0: one stream with norms before and after every sublayer; else hyper-connections */
+    float residual_mult, logit_scale;     /* with streams > 0 */
 } flexllm_decoder_config;
 FLEXLLM_API int flexllm_model_create_decoder(flexllm_model** out, const flexllm_decoder_config* cfg);
 /* One bf16 weight tensor by name (host or device memory, dense; linear weights [out][in]): embed, head, final.norm, loop.step,
- * l<i>.norm1 / norm1b / norm2 / norm2b, l<i>.mix.{q,k,v}[.b], .q.norm, .k.norm, .rel, .g, .o, l<i>.mlp.{gate,up,down}.
+ * l<i>.norm1 / norm1b / norm2 / norm2b, l<i>.mix.{q,k,v}[.b], .q.norm, .k.norm, .rel, .g, .sink, .o, l<i>.mlp.{gate,up,down};
+ * l<i>.mix.{in,conv,conv.b,dt_bias,A_log,D,norm,o}; l<i>.hc{1,2}.{in,out,mix}.
  * Steps are refused (FLEXLLM_EINVAL) until every tensor is there. */
 FLEXLLM_API int flexllm_model_load_tensor(flexllm_model* m, const char* name, int dtype, int ndim, const int64_t* shape, const void* data,
                                           void* stream);
