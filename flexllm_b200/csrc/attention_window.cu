@@ -397,17 +397,20 @@ __global__ void __launch_bounds__(256) attn_row_kernel(const AttnCall c, int L, 
 //   values: dimensions on the 16-row side (V^T page rows), heads on the 8-column side, the tile's keys as the inner index,
 //           cut into KS slices when there are fewer than 8 blocks of 16 dimensions (MPW blocks per warp)
 // Every operand row is read with 16-byte loads: lane % 4 holds elements 8 c .. 8 c + 7 of each 32, i.e. the inner index is
-// permuted, the same way in both operands. K of the next tile and V of this one are in flight during the arithmetic. The
-// scores are bounded (see the prompt kernel), so exp(s) needs no running maximum and splits just add up.
+// permuted, the same way in both operands. K of the next tile and V of this one are in flight during the arithmetic. Bounded
+// scores (see the prompt kernel) need no running maximum and splits just add up; ONLINE (no softcap, no bias): the warps agree on
+// a tile's maxima through shared memory, and a running maximum that grows by more than kSlack rescales sums and outputs.
 struct DecodeArgs { AttnCall c; float a2, b2, shift2; int tiles_max; int* error_flag; };
+constexpr float kSlack = 8.0f;             // log2 units by which a score may exceed the softmax shift of its row
+constexpr float kNoScore = -1e30f;         // initial running maximum without a sink: below every score
 constexpr int DT_KEYS = 128, DT_PS = DT_KEYS + 8;      // keys per tile, row pitch of the weights in shared memory
 
 __host__ __device__ inline size_t decode_smem(int dkp, int dv, int KS, int tiles_max) {
-    // page ids, q [8][dkp + 8], weights [2][8][DT_PS], sums [8][8], outputs [KS][8][dv]
-    return (size_t)((2 * tiles_max + 3) & ~3) * 4 + 8 * (size_t)(dkp + 8) * 2 + 2 * 8 * DT_PS * 2 + 64 * 4 + (size_t)KS * 8 * dv * 4;
+    // page ids, q [8][dkp + 8], weights [2][8][DT_PS], sums [8][8], outputs [KS][8][dv]; ONLINE: maxima [2][8][8] before the outputs
+    return (size_t)((2 * tiles_max + 3) & ~3) * 4 + 8 * (size_t)(dkp + 8) * 2 + 2 * 8 * DT_PS * 2 + (64 + 128) * 4 + (size_t)KS * 8 * dv * 4;
 }
 
-template <int DKC, int KS, int MPW>
+template <bool ONLINE, int DKC, int KS, int MPW>
 __global__ void __launch_bounds__(256, DKC == 8 || MPW == 2 ? 1 : 2) attn_decode_mma_kernel(const __grid_constant__ DecodeArgs a) {
     constexpr int MTP = MPW == 2 ? 8 : 8 / KS;             // warps along the dimensions
     constexpr int NCH = 4 / KS;                            // 32-key chunks of a warp's slice
@@ -421,29 +424,30 @@ __global__ void __launch_bounds__(256, DKC == 8 || MPW == 2 ? 1 : 2) attn_decode
     bf16* q_sm = reinterpret_cast<bf16*>(raw + (size_t)((2 * a.tiles_max + 3) & ~3) * 4);
     bf16* p_sm = q_sm + 8 * (s.dkp + 8);
     float* l_sm = reinterpret_cast<float*>(p_sm + 2 * 8 * DT_PS);
-    float* o_sm = l_sm + 64;
+    float* mx_sm = l_sm + 64;
+    float* o_sm = mx_sm + 128;
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, lr = lane >> 2, lc = lane & 3;
     const int split = blockIdx.x, n_split = gridDim.x, g = blockIdx.y, b = blockIdx.z;
     pdl_sync();
     const int pos = start_pos(c, b, a.error_flag);
-    const int lo = max(0, pos - s.window + 1);
-    const int p_lo = lo / PG, n_pg = pos / PG - p_lo + 1, n_tiles = (n_pg + 1) / 2;
+    const KeyPages pages(s, pos, pos);
+    const int n_pg = pages.n, n_tiles = (n_pg + 1) / 2;
     const int t_beg = (int)((long)split * n_tiles / n_split), t_end = (int)((long)(split + 1) * n_tiles / n_split);
-    const int32_t* pt = c.page_table + (long)b * c.max_pages + p_lo;
+    const int32_t* pt = c.page_table + (long)b * c.max_pages;
     const bf16* prow = (const bf16*)c.proj + (long)b * s.ld;
     const long kh = (long)PG * s.dkp, vh = (long)PG * s.dv;
-    for (int i = tid; i < 2 * (t_end - t_beg); i += 256) pt_sm[i] = 2 * t_beg + i < n_pg ? pt[2 * t_beg + i] : -1;
-    const int nq = s.H * s.dk, nk = s.G * s.dk, nv = s.dkp >> 3;
-    const float2 ss = block_sum2<256>(share_sumsq<256>(prow + s.q_off, nq, tid), share_sumsq<256>(prow + s.k_off, nk, tid), red);
-    const float rq = 1.0f / sqrtf(ss.x / (float)nq + c.eps), rk = 1.0f / sqrtf(ss.y / (float)nk + c.eps);
+    for (int i = tid; i < 2 * (t_end - t_beg); i += 256) pt_sm[i] = 2 * t_beg + i < n_pg ? pt[pages.at(2 * t_beg + i)] : -1;
+    const int nv = s.dkp >> 3;
+    const float2 rms = qk_rms(c, prow, tid, red);
+    const float rq = rms.x, rk = rms.y;
     for (int i = tid; i < 8 * nv; i += 256) {
         const int r = i / nv, e0 = (i - r * nv) * 8;
         float f[8] = {0, 0, 0, 0, 0, 0, 0, 0};
         if (r < R) normed8(prow + s.q_off, c.q_gain, (g * R + r) * s.dk, e0, s.dk, rq, f);
         store8(q_sm + r * (s.dkp + 8) + e0, f);
     }
-    if (split == n_split - 1) {
-        const long page = pt[n_pg - 1];
+    if (s.k_off >= 0 && split == n_split - 1) {
+        const long page = pt[pages.at(n_pg - 1)];
         const int slot = pos & (PG - 1);
         bf16* kp = (bf16*)c.k_pool + (page * s.G + g) * kh + (long)slot * s.dkp;
         for (int i = tid; i < nv; i += 256) {
@@ -477,8 +481,8 @@ __global__ void __launch_bounds__(256, DKC == 8 || MPW == 2 ? 1 : 2) attn_decode
     const int mt = warp % MTP, slice = warp / MTP;
     const bool pv_on = slice < KS;
     float acc[MPW][4] = {};
-    float lsum[2] = {0.0f, 0.0f};
-    const float* bias_g = c.bias + (long)g * (2 * kBiasPad + s.window) * R;
+    float lsum[2] = {0.0f, 0.0f}, m_run[2] = {kNoScore, kNoScore};
+    const float* bias_g = ONLINE ? nullptr : c.bias + (long)g * (2 * kBiasPad + s.window) * R;
     const float badd = s.softcap * kLog2e - a.shift2;
     if (t_beg < t_end) load_k(t_beg);
     for (int t = t_beg; t < t_end; t++) {
@@ -499,8 +503,9 @@ __global__ void __launch_bounds__(256, DKC == 8 || MPW == 2 ? 1 : 2) attn_decode
             }
         }
         // biases of this thread's two keys and two heads (-inf: masked, or no such head)
-        const int d0 = pos - ((p_lo + 2 * t) * PG + warp * 16 + lr);
+        const int d0 = pos - (pages.at(2 * t + (warp >> 2)) * PG + (warp & 3) * 16 + lr);        // distance of this thread's first key
         float bi[2][2];
+        if (!ONLINE)
 #pragma unroll
         for (int h = 0; h < 2; h++)
 #pragma unroll
@@ -514,11 +519,43 @@ __global__ void __launch_bounds__(256, DKC == 8 || MPW == 2 ? 1 : 2) attn_decode
         }
         if (t + 1 < t_end) load_k(t + 1);
         bf16* pb = p_sm + (t & 1) * 8 * DT_PS + warp * 16 + lr;
+        if (ONLINE) {
+            float* mx = mx_sm + (t & 1) * 64;
+            const bool in0 = 2 * t + (warp >> 2) < n_pg && sees(s, pos, pos - d0), in1 = 2 * t + (warp >> 2) < n_pg && sees(s, pos, pos - d0 + 8);
+            float tm[2];
+#pragma unroll
+            for (int u = 0; u < 2; u++) {
+                const bool head = lc * 2 + u < R;
+                sc[u] = in0 && head ? sc[u] * a.a2 : -INFINITY;
+                sc[2 + u] = in1 && head ? sc[2 + u] * a.a2 : -INFINITY;
+                tm[u] = fmaxf(sc[u], sc[2 + u]);
+#pragma unroll
+                for (int o = 4; o < 32; o <<= 1) tm[u] = fmaxf(tm[u], __shfl_xor_sync(0xffffffffu, tm[u], o));
+            }
+            if (lr == 0) *reinterpret_cast<float2*>(mx + warp * 8 + lc * 2) = make_float2(tm[0], tm[1]);
+            __syncthreads();
+            float al[2];
+#pragma unroll
+            for (int u = 0; u < 2; u++) {
+                float v = mx[lc * 2 + u];
+#pragma unroll
+                for (int w = 1; w < 8; w++) v = fmaxf(v, mx[w * 8 + lc * 2 + u]);
+                const float m_new = v > m_run[u] + kSlack ? v : m_run[u];
+                al[u] = ex2_fast(m_run[u] - m_new);
+                m_run[u] = m_new;
+                lsum[u] *= al[u];
+            }
+#pragma unroll
+            for (int m = 0; m < MPW; m++)
+#pragma unroll
+                for (int i = 0; i < 4; i++) acc[m][i] *= al[i & 1];
+        }
 #pragma unroll
         for (int h = 0; h < 2; h++)
 #pragma unroll
             for (int u = 0; u < 2; u++) {
-                const float s2 = __fmaf_rn(a.b2, rcp_fast(1.0f + ex2_fast(sc[2 * h + u] * a.a2)), __fmaf_rn(bi[h][u], kLog2e, badd));
+                const float s2 = ONLINE ? sc[2 * h + u] - m_run[u]
+                                        : __fmaf_rn(a.b2, rcp_fast(1.0f + ex2_fast(sc[2 * h + u] * a.a2)), __fmaf_rn(bi[h][u], kLog2e, badd));
                 const float p = ex2_fast(s2);
                 lsum[u] += p;
                 pb[(lc * 2 + u) * DT_PS + 8 * h] = __float2bfloat16_rn(p);
@@ -554,13 +591,16 @@ __global__ void __launch_bounds__(256, DKC == 8 || MPW == 2 ? 1 : 2) attn_decode
     __syncthreads();
     auto head_l = [&](int r) { float v = 0.0f; for (int w = 0; w < 8; w++) v += l_sm[w * 8 + r]; return v; };
     auto head_o = [&](int r, int d) { float v = 0.0f; for (int k = 0; k < KS; k++) v += o_sm[((long)k * 8 + r) * s.dv + d]; return v; };
+    // ONLINE: the heads' running maxima, the same in all warps
+    if (ONLINE && tid < 4) { mx_sm[lc * 2] = m_run[0]; mx_sm[lc * 2 + 1] = m_run[1]; }
+    if (ONLINE) __syncthreads();
     const float sink = s.sink ? ex2_fast(-a.shift2) : 0.0f;
-    const long stride = (long)R * (s.dv + 1);
+    const long stride = (long)R * (s.dv + (ONLINE ? 2 : 1)), o_at = ONLINE ? 2 * R : R;
     float* part = c.ws + ((long)b * s.G + g) * n_split * stride;
     if (n_split > 1) {
         float* mine = part + split * stride;
-        for (int i = tid; i < R; i += 256) mine[i] = head_l(i);
-        for (int i = tid; i < R * s.dv; i += 256) mine[R + i] = head_o(i / s.dv, i % s.dv);
+        for (int i = tid; i < R; i += 256) { mine[i] = head_l(i); if (ONLINE) mine[R + i] = mx_sm[i]; }
+        for (int i = tid; i < R * s.dv; i += 256) mine[o_at + i] = head_o(i / s.dv, i % s.dv);
         __threadfence();
         __syncthreads();
         int* cnt = c.counters + (long)b * s.G + g;
@@ -574,7 +614,25 @@ __global__ void __launch_bounds__(256, DKC == 8 || MPW == 2 ? 1 : 2) attn_decode
     for (int i = tid; i < R * s.dv; i += 256) {
         const int r = i / s.dv;
         float l = sink, v = 0.0f;
-        if (n_split > 1) {
+        if (ONLINE) {
+            const float snk = sink_score(c, g * R + r) * kLog2e;             // -inf without a sink
+            float m = fmaxf(snk, kNoScore);
+            if (n_split > 1) {
+                for (int k = 0; k < n_split; k++) m = fmaxf(m, __ldcg(part + k * stride + R + r));
+                l = ex2_fast(snk - m);
+#pragma unroll 4
+                for (int k = 0; k < n_split; k++) {
+                    const float w = ex2_fast(__ldcg(part + k * stride + R + r) - m);
+                    l = __fmaf_rn(__ldcg(part + k * stride + r), w, l);
+                    v = __fmaf_rn(__ldcg(part + k * stride + o_at + i), w, v);
+                }
+            } else {
+                m = fmaxf(m, mx_sm[r]);
+                const float w = ex2_fast(mx_sm[r] - m);
+                l = __fmaf_rn(head_l(r), w, ex2_fast(snk - m));
+                v = head_o(r, i - r * s.dv) * w;
+            }
+        } else if (n_split > 1) {
 #pragma unroll 4
             for (int k = 0; k < n_split; k++) { l += __ldcg(part + k * stride + r); v += __ldcg(part + k * stride + R + i); }
         } else {
@@ -589,8 +647,10 @@ __global__ void __launch_bounds__(256, DKC == 8 || MPW == 2 ? 1 : 2) attn_decode
 // ---------------------------------------------------------------------------------------------------------------
 // Prompt attention on the tensor cores. A CTA takes TQ = 128 / R consecutive positions x the R query heads of one key/value
 // head (row = position * R + head: the heads of a group share the K and V tiles, and a small window wastes few keys), and
-// walks the key pages its window reaches. The scores are bounded by softcap + max|bias|, so the softmax shift is a constant
-// (`shift2`) and the values accumulate in TMEM over all pages without rescaling.
+// walks the key pages its window reaches (and those of the kept first positions). Scores bounded by softcap + max|bias| have a
+// constant softmax shift (`shift2`) and the values accumulate in TMEM over all pages without rescaling. ONLINE (no softcap, no
+// bias): a row's shift is its running maximum, lazily: only when a score exceeds it by more than kSlack does the row's warp wait
+// for the products so far and rescale the accumulator in TMEM.
 //   warps 0..3  softmax: one row per thread        warp 4  TMA: Q, then K and V pages        warp 5  MMA issue, TMEM
 struct PrefillArgs {
     AttnCall c;
@@ -598,23 +658,25 @@ struct PrefillArgs {
     int kc, vrows;                    // 128-byte blocks of a Q/K row; rows of a V^T tile (dv rounded up to 16)
     float a2, b2, shift2;             // tanh argument factor and -2 softcap in log2 units; softmax shift
     int tmem_cols, o_col, p_bufs;
+    bool online;
     int* error_flag;
 };
 constexpr int PF_S_COLS = 64;
 
 struct PrefillSmem { uint32_t k, v, p, bias, bars, total; };
-__host__ __device__ inline PrefillSmem prefill_smem(int kc, int vrows, int R, int TQ, int p_bufs) {
+__host__ __device__ inline PrefillSmem prefill_smem(int kc, int vrows, int R, int TQ, int p_bufs, bool online) {
     PrefillSmem o;
     o.k = (uint32_t)kc * 16384u;                                   // Q first
     o.v = o.k + 2u * (uint32_t)kc * 8192u;
     o.p = o.v + 2u * (((uint32_t)vrows * 128u + 1023u) & ~1023u);
     o.bias = o.p + (uint32_t)p_bufs * 16384u;
-    const uint32_t bias_floats = (uint32_t)((TQ + 63) * R + 128);
+    const uint32_t bias_floats = online ? 0u : (uint32_t)((TQ + 63) * R + 128);
     o.bars = o.bias + 2u * ((bias_floats * 4u + 15u) & ~15u);
     o.total = o.bars + 256u + 1024u;
     return o;
 }
 
+template <bool ONLINE>
 __global__ void __launch_bounds__(192, 2) attn_window_prefill_kernel(const __grid_constant__ CUtensorMap tmapQ,
                                                                   const __grid_constant__ CUtensorMap tmapK,
                                                                   const __grid_constant__ CUtensorMap tmapV,
@@ -625,7 +687,7 @@ __global__ void __launch_bounds__(192, 2) attn_window_prefill_kernel(const __gri
     uint8_t* base_ptr = smem_raw + (base - raw);
     const AttnShape& s = a.c.s;
     const int R = a.R, TQ = a.TQ;
-    const PrefillSmem o = prefill_smem(a.kc, a.vrows, R, TQ, a.p_bufs);
+    const PrefillSmem o = prefill_smem(a.kc, a.vrows, R, TQ, a.p_bufs, ONLINE);
     const uint32_t k_bytes = (uint32_t)a.kc * 8192u, v_bytes = (uint32_t)a.vrows * 128u, v_stride = (v_bytes + 1023u) & ~1023u;
     uint64_t* bars = reinterpret_cast<uint64_t*>(base_ptr + o.bars);
     const uint32_t bar_q = smem_u32(bars);
@@ -656,9 +718,9 @@ __global__ void __launch_bounds__(192, 2) attn_window_prefill_kernel(const __gri
     const int p0 = start_pos(a.c, b, a.error_flag);
     const int q0 = p0 + qt * TQ;                                         // first position of the tile
     const int q1 = min(p0 + a.c.Sc, q0 + TQ) - 1;                        // last one
-    const int pg_lo = max(0, q0 - s.window + 1) / PG, pg_hi = q1 / PG;
-    const int n_kt = pg_hi - pg_lo + 1;
-    const int32_t* pt = a.c.page_table + (long)b * a.c.max_pages + pg_lo;
+    const KeyPages pages(s, q0, q1);
+    const int n_kt = pages.n;
+    const int32_t* pt = a.c.page_table + (long)b * a.c.max_pages;
 
     if (warp == 4) {
         if (lane == 0) {
@@ -669,7 +731,7 @@ __global__ void __launch_bounds__(192, 2) attn_window_prefill_kernel(const __gri
             for (int j = 0; ok && j < n_kt; j++) {
                 const int sb = j & 1;
                 const uint32_t ph = (uint32_t)((j >> 1) & 1) ^ 1u;
-                const int page = __ldg(pt + j);
+                const int page = __ldg(pt + pages.at(j));
                 if (!mbar_wait(bar_ke + 8 * sb, ph, abort_flag)) break;
                 mbar_expect_tx(bar_kf + 8 * sb, k_bytes);
                 for (int i = 0; i < a.kc; i++)
@@ -717,10 +779,10 @@ __global__ void __launch_bounds__(192, 2) attn_window_prefill_kernel(const __gri
     } else {
         const int rr = warp * 32 + lane;                       // row: position rr / R of the tile, head rr % R of the group
         const uint32_t lane_addr = (uint32_t)(warp * 32) << 16;
-        const int n_bias = (TQ + 63) * R;
+        const int n_bias = ONLINE ? 0 : (TQ + 63) * R;
         float* bias_sm = reinterpret_cast<float*>(base_ptr + o.bias);
         const int bias_stride = (n_bias + 128 + 3) & ~3;
-        const float* bias_g = a.c.bias + (long)g * (2 * kBiasPad + s.window) * R;
+        const float* bias_g = ONLINE ? nullptr : a.c.bias + (long)g * (2 * kBiasPad + s.window) * R;
         auto wait_bar = [&](uint32_t bar, uint32_t parity) {
             int got = (lane == 0) ? (mbar_wait(bar, parity, abort_flag) ? 1 : 0) : 1;
             return __shfl_sync(0xffffffffu, got, 0) != 0;
@@ -732,7 +794,7 @@ __global__ void __launch_bounds__(192, 2) attn_window_prefill_kernel(const __gri
         constexpr int NB = 9;                                            // (TQ + 63) * R <= 1136 for R <= 16
         float nb[NB];
         auto fetch_bias = [&](int j) {
-            const int dmin = q0 - (pg_lo + j) * PG - 63;                 // distance of the first entry
+            const int dmin = q0 - pages.at(j) * PG - 63;                 // distance of the first entry
             const float* src = bias_g + (long)(dmin + kBiasPad) * R;
 #pragma unroll
             for (int i = 0; i < NB; i++) nb[i] = rr + 128 * i < n_bias ? src[rr + 128 * i] : 0.0f;
@@ -743,10 +805,87 @@ __global__ void __launch_bounds__(192, 2) attn_window_prefill_kernel(const __gri
             for (int i = 0; i < NB; i++)
                 if (rr + 128 * i < n_bias) dst[rr + 128 * i] = __fmaf_rn(nb[i], kLog2e, badd);
         };
-        fetch_bias(0);
-        stage_bias(0);
         float l = 0.0f;
         bool ok = true;
+        // ---- ONLINE: this row's position, its softmax shift and, per tile, the keys it sees
+        const int my_pos = q0 + rr / R;
+        const float snk = ONLINE ? sink_score(a.c, g * R + rr % R) * kLog2e : 0.0f;
+        float m = ONLINE ? fmaxf(snk, kNoScore) : 0.0f;
+        if (ONLINE)
+        for (int j = 0; j < n_kt; j++) {
+            const int sb = j & 1, pb = a.p_bufs == 2 ? sb : 0;
+            if (!wait_bar(bar_sf + 8 * sb, (uint32_t)((j >> 1) & 1))) { ok = false; break; }
+            tc_fence_after();
+            const uint32_t tS = tmem_base + sb * PF_S_COLS + lane_addr;
+            uint32_t v[4][16];
+#pragma unroll
+            for (int cc = 0; cc < 4; cc++) tmem_ld_32x16(tS + 16 * cc, v[cc]);
+            tmem_ld_wait();
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(bar_se + 8 * sb);                 // the scores are in registers: the next product may start
+            const int key0 = pages.at(j) * PG;
+            const int hi = my_pos - key0, lo = hi - s.window + 1, kept = s.keep - key0;      // sees key c: c <= hi, c >= lo or c < kept
+            const bool all = hi >= PG - 1 && (lo <= 0 || kept >= PG);
+            float mx = -INFINITY;
+#pragma unroll
+            for (int cc = 0; cc < 4; cc++)
+#pragma unroll
+                for (int i = 0; i < 16; i++) v[cc][i] = __float_as_uint(__uint_as_float(v[cc][i]) * a.a2);
+            if (!__all_sync(0xffffffffu, all))
+#pragma unroll
+                for (int cc = 0; cc < 4; cc++)
+#pragma unroll
+                    for (int i = 0; i < 16; i++) {
+                        const int c = cc * 16 + i;
+                        if (c > hi || (c < lo && c >= kept)) v[cc][i] = 0xff800000u;
+                    }
+#pragma unroll
+            for (int cc = 0; cc < 4; cc++)
+#pragma unroll
+                for (int i = 0; i < 16; i++) mx = fmaxf(mx, __uint_as_float(v[cc][i]));
+            const bool grow = mx > m + kSlack;
+            if (__any_sync(0xffffffffu, grow)) {
+                const float m_new = grow ? mx : m, al = ex2_fast(m - m_new);
+                m = m_new;
+                l *= al;
+                if (j > 0) {
+                    // the products up to tile j - 1 are in the accumulator; tile j's waits for this warp's weights
+                    const int ob = a.p_bufs == 2 ? (j - 1) & 1 : 0;
+                    if (!wait_bar(bar_pe + 8 * ob, (uint32_t)((a.p_bufs == 2 ? (j - 1) >> 1 : j - 1) & 1))) { ok = false; break; }
+                    tc_fence_after();
+                    for (int d0 = 0; d0 < a.vrows; d0 += 16) {
+                        uint32_t w[16];
+                        tmem_ld_32x16(tmem_base + a.o_col + d0 + lane_addr, w);
+                        tmem_ld_wait();
+#pragma unroll
+                        for (int i = 0; i < 16; i++) w[i] = __float_as_uint(__uint_as_float(w[i]) * al);
+                        tmem_st_32x16(tmem_base + a.o_col + d0 + lane_addr, w);
+                    }
+                    tmem_st_wait();
+                    tc_fence_before();
+                }
+            }
+            if (!wait_bar(bar_pe + 8 * pb, (uint32_t)((a.p_bufs == 2 ? j >> 1 : j) & 1) ^ 1u)) { ok = false; break; }
+            uint8_t* prow = base_ptr + o.p + pb * 16384 + rr * 128;
+#pragma unroll
+            for (int cc = 0; cc < 4; cc++) {
+                uint32_t pk[8];
+#pragma unroll
+                for (int i = 0; i < 16; i += 2) {
+                    const float p0 = ex2_fast(__uint_as_float(v[cc][i]) - m), p1 = ex2_fast(__uint_as_float(v[cc][i + 1]) - m);
+                    l += p0 + p1;
+                    pk[i >> 1] = bf_pack(p0, p1);
+                }
+                *reinterpret_cast<uint4*>(prow + (((2 * cc) ^ (rr & 7)) << 4)) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+                *reinterpret_cast<uint4*>(prow + (((2 * cc + 1) ^ (rr & 7)) << 4)) = make_uint4(pk[4], pk[5], pk[6], pk[7]);
+            }
+            fence_proxy_async_smem();
+            __syncwarp();
+            if (lane == 0) mbar_arrive(bar_pf + 8 * pb);
+        }
+        if (!ONLINE) { fetch_bias(0); stage_bias(0); }
+        if (!ONLINE)
         for (int j = 0; j < n_kt; j++) {
             const int sb = j & 1, pb = a.p_bufs == 2 ? sb : 0;
             named_sync<1, 128>();                                        // tile j's biases are in place; j - 1's reads are over
@@ -801,7 +940,7 @@ __global__ void __launch_bounds__(192, 2) attn_window_prefill_kernel(const __gri
             tc_fence_after();
             const int t = rr / R, r = rr - t * R;
             const bool row_ok = rr < TQ * R && q0 + t <= q1;
-            const float rl = 1.0f / (l + (s.sink ? ex2_fast(-a.shift2) : 0.0f));
+            const float rl = 1.0f / (l + (ONLINE ? ex2_fast(snk - m) : s.sink ? ex2_fast(-a.shift2) : 0.0f));
             const long m = (long)b * a.c.Sc + qt * TQ + t;
             const long hcol = (long)(g * R + r) * s.dv;
             bf16* out = (bf16*)a.c.out + m * a.c.ldo + hcol;
@@ -896,40 +1035,49 @@ bool bounded_scores(const AttnCall& c, float* a2, float* b2, float* shift2) {
     return *shift2 <= (s.sink ? 80.0f : 20.0f);
 }
 
-template <int DKC, int KS, int MPW> int launch_decode(DecodeArgs& a, int splits, cudaStream_t st) {
+template <bool ONLINE, int DKC, int KS, int MPW> int launch_decode(DecodeArgs& a, int splits, cudaStream_t st) {
     const AttnCall& c = a.c;
     const size_t smem = decode_smem(c.s.dkp, c.s.dv, KS, a.tiles_max);
-    auto kern = attn_decode_mma_kernel<DKC, KS, MPW>;
+    auto kern = attn_decode_mma_kernel<ONLINE, DKC, KS, MPW>;
     if (smem > 200 * 1024) return FLEXLLM_ENOTSUP;
     TRY_RC(set_smem((const void*)kern, smem));
     launch_k(kern, dim3(splits, c.s.G, c.B), dim3(256), smem, st, a);
     return launch_status();
 }
-template <int DKC> int pick_decode(DecodeArgs& a, int splits, cudaStream_t st) {
+template <bool ONLINE, int DKC> int pick_decode(DecodeArgs& a, int splits, cudaStream_t st) {
     const int dv = a.c.s.dv;
-    if (dv <= 32) return launch_decode<DKC, 4, 1>(a, splits, st);
-    if (dv <= 64) return launch_decode<DKC, 2, 1>(a, splits, st);
-    if (dv <= 128) return launch_decode<DKC, 1, 1>(a, splits, st);
-    return launch_decode<DKC, 1, 2>(a, splits, st);
+    if (dv <= 32) return launch_decode<ONLINE, DKC, 4, 1>(a, splits, st);
+    if (dv <= 64) return launch_decode<ONLINE, DKC, 2, 1>(a, splits, st);
+    if (dv <= 128) return launch_decode<ONLINE, DKC, 1, 1>(a, splits, st);
+    return launch_decode<ONLINE, DKC, 1, 2>(a, splits, st);
+}
+template <bool ONLINE> int pick_decode_dk(DecodeArgs& a, int splits, cudaStream_t st) {
+    if (a.c.s.dkp <= 64) return pick_decode<ONLINE, 2>(a, splits, st);
+    if (a.c.s.dkp <= 128) return pick_decode<ONLINE, 4>(a, splits, st);
+    return pick_decode<ONLINE, 8>(a, splits, st);
+}
+// Whether the ONLINE forms cover the scores; their factor to log2 units.
+bool plain_scores(const AttnCall& c, float* a2) {
+    *a2 = c.s.scale * kLog2e;
+    return c.s.softcap <= 0.0f && !c.bias;
 }
 // FLEXLLM_ENOTSUP: the row kernel takes the call.
 int run_decode(const AttnCall& c, cudaStream_t st) {
     const AttnShape& s = c.s;
     DecodeArgs a;
     a.c = c; a.error_flag = device_error_flag();
-    if (s.H / s.G > 8 || s.dkp > 256 || s.dv > 256 || c.B > 65535 || !bounded_scores(c, &a.a2, &a.b2, &a.shift2)) return FLEXLLM_ENOTSUP;
+    const bool bounded = bounded_scores(c, &a.a2, &a.b2, &a.shift2);
+    if (s.H / s.G > 8 || s.dkp > 256 || s.dv > 256 || c.B > 65535 || (!bounded && !plain_scores(c, &a.a2))) return FLEXLLM_ENOTSUP;
     const int reach = s.window < c.max_pos + 1 ? s.window : c.max_pos + 1;
-    const int tiles = (reach + 2 * PG - 2) / PG / 2 + 1;
+    const int tiles = ((reach + 2 * PG - 2) / PG + attn_keep_pages(s.keep)) / 2 + 1;
     const long ctas = (long)c.B * s.G;
     long splits = (kDecodeCtas + ctas - 1) / ctas;
     if (splits > tiles / 2) splits = tiles / 2;
-    const long per = ctas * (s.H / s.G) * (s.dv + 1);
+    const long per = ctas * (s.H / s.G) * (s.dv + 2);
     if (splits * per > (long)c.ws_floats) splits = (long)c.ws_floats / per;
     if (splits < 1 || ctas > c.n_counters || !c.ws) splits = 1;
     a.tiles_max = (int)((tiles + splits - 1) / splits + 1);
-    if (s.dkp <= 64) return pick_decode<2>(a, (int)splits, st);
-    if (s.dkp <= 128) return pick_decode<4>(a, (int)splits, st);
-    return pick_decode<8>(a, (int)splits, st);
+    return bounded ? pick_decode_dk<false>(a, (int)splits, st) : pick_decode_dk<true>(a, (int)splits, st);
 }
 
 // Whether the tensor-core kernel covers the call (bf16 only).
@@ -938,7 +1086,8 @@ bool prefill_covers(const AttnCall& c, PrefillArgs* a) {
     a->c = c;
     a->R = s.H / s.G; a->TQ = a->R <= 16 ? 128 / a->R : 0;
     if (a->R > 16 || s.dkp > 256 || s.dv > 256) return false;
-    if (!bounded_scores(c, &a->a2, &a->b2, &a->shift2)) return false;
+    a->online = !bounded_scores(c, &a->a2, &a->b2, &a->shift2);
+    if (a->online && !plain_scores(c, &a->a2)) return false;
     a->kc = (s.dkp + 63) / 64; a->vrows = (s.dv + 15) / 16 * 16;
     a->n_qt = (c.Sc + a->TQ - 1) / a->TQ;
     a->o_col = 2 * PF_S_COLS;
@@ -946,11 +1095,11 @@ bool prefill_covers(const AttnCall& c, PrefillArgs* a) {
     while (cols < a->o_col + a->vrows) cols *= 2;
     a->tmem_cols = cols;
     // two CTAs per SM where one P buffer makes that possible
-    a->p_bufs = prefill_smem(a->kc, a->vrows, a->R, a->TQ, 2).total <= 113 * 1024 ? 2
-              : prefill_smem(a->kc, a->vrows, a->R, a->TQ, 1).total <= 113 * 1024 ? 1 : 2;
-    if (prefill_smem(a->kc, a->vrows, a->R, a->TQ, a->p_bufs).total > 227 * 1024) a->p_bufs = 1;
+    a->p_bufs = prefill_smem(a->kc, a->vrows, a->R, a->TQ, 2, a->online).total <= 113 * 1024 ? 2
+              : prefill_smem(a->kc, a->vrows, a->R, a->TQ, 1, a->online).total <= 113 * 1024 ? 1 : 2;
+    if (prefill_smem(a->kc, a->vrows, a->R, a->TQ, a->p_bufs, a->online).total > 227 * 1024) a->p_bufs = 1;
     a->error_flag = device_error_flag();
-    return prefill_smem(a->kc, a->vrows, a->R, a->TQ, a->p_bufs).total <= 227 * 1024;
+    return prefill_smem(a->kc, a->vrows, a->R, a->TQ, a->p_bufs, a->online).total <= 227 * 1024;
 }
 
 int run_prefill(const PrefillArgs& a, cudaStream_t st) {
@@ -960,8 +1109,8 @@ int run_prefill(const PrefillArgs& a, cudaStream_t st) {
     TRY_RC(make_tmap_rows3_u8(&tq, c.q, (uint64_t)c.B * c.Sc, (uint64_t)s.H, (uint64_t)s.dkp * 2, (uint32_t)a.TQ, (uint32_t)a.R));
     TRY_RC(cached_tmap_u8(&tk, c.k_pool, (uint64_t)c.n_pages * s.G * PG, (uint64_t)s.dkp * 2, PG, 0));
     TRY_RC(cached_tmap_u8(&tv, c.v_pool, (uint64_t)c.n_pages * s.G * s.dv, PG * 2, (uint32_t)a.vrows, 0));
-    const size_t smem = prefill_smem(a.kc, a.vrows, a.R, a.TQ, a.p_bufs).total;
-    auto kern = attn_window_prefill_kernel;
+    const size_t smem = prefill_smem(a.kc, a.vrows, a.R, a.TQ, a.p_bufs, a.online).total;
+    auto kern = a.online ? attn_window_prefill_kernel<true> : attn_window_prefill_kernel<false>;
     TRY_RC(set_smem((const void*)kern, smem));
     launch_k(kern, dim3(a.n_qt, s.G, c.B), dim3(192), smem, st, tq, tk, tv, a);
     return launch_status();
