@@ -251,6 +251,43 @@ def sandwich_norm(x, D, eps, y=None, gain_post=None, add_vec=None, gain_pre=None
     return h
 
 
+def hyper_norm(x, D, eps, y=None, mix=None, out=None, read=None, gain=None, dtype=torch.float32):
+    """Residual streams x [M,streams,ld] fp32 (in place): x_t <- sum_s mix[s,t] x_s + out[t] y; then, with gain, returns
+    rms norm(sum_s read[s] x_s) * gain as [M,ld] of dtype (columns up to D)."""
+    M, n, ld = x.shape
+    h = torch.zeros((M, ld), dtype=dtype, device=x.device) if gain is not None else None
+    _call("flexllm_hyper_norm", _lib.BF16 if dtype == torch.bfloat16 else _lib.F32, _ptr(x), ld, n, M, D, eps, _ptr(y),
+          y.shape[1] if y is not None else 0, _ptr(mix), _ptr(out), _ptr(read), _ptr(gain), _ptr(h), ld)
+    return h
+
+
+class StateSpaceMixer:
+    """A Mamba-2 form mixer between its projections, with `slots` sequences' states (dtype bf16 or fp32).
+
+    conv_w [conv,channels], conv_b [channels], gain [heads*P8], dt_bias, A (negative), D [heads]: fp32 CUDA tensors in the padded
+    column order of flexllm_ssm. Call with proj [B*n,row] and ctx [B] (tokens already seen). Returns [B*n,heads*P8]."""
+
+    def __init__(self, heads, vdim, state, groups, conv, norm_groups, conv_w, conv_b, dt_bias, A, D, gain, slots, eps=1e-5, dtype=torch.bfloat16):
+        self.shape = _lib.SsmShape(heads, vdim, state, groups, conv, norm_groups, eps)
+        self.w, self.dtype = (conv_w, conv_b, dt_bias, A, D, gain), dtype
+        self.row = lib().flexllm_ssm_row(C.byref(self.shape))
+        self.channels = lib().flexllm_ssm_channels(C.byref(self.shape))
+        dev = conv_w.device
+        self.state = torch.zeros((slots, lib().flexllm_ssm_state_floats(C.byref(self.shape))), dtype=torch.float32, device=dev)
+        self.history = torch.zeros((slots, conv, self.channels), dtype=dtype, device=dev)
+
+    def __call__(self, proj, ctx):
+        B = ctx.numel()
+        n = proj.shape[0] // B
+        assert proj.shape[1] == self.row and proj.dtype == self.dtype and B <= self.state.shape[0]
+        out = torch.empty((B * n, self.shape.heads * ((self.shape.vdim + 7) // 8 * 8)), dtype=self.dtype, device=proj.device)
+        nbytes = lib().flexllm_ssm_workspace(C.byref(self.shape), B, n)
+        ws = torch.empty((nbytes,), dtype=torch.uint8, device=proj.device)
+        _call("flexllm_ssm", _lib.BF16 if self.dtype == torch.bfloat16 else _lib.F32, C.byref(self.shape), _ptr(proj), *map(_ptr, self.w),
+              _ptr(self.state), _ptr(self.history), _ptr(ctx), B, n, _ptr(out), _ptr(ws), nbytes)
+        return out
+
+
 class WindowAttention:
     """One layer of windowed attention with its own floating-point paged cache (dtype bf16 or fp32).
 
