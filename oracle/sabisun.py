@@ -2,13 +2,18 @@
 
 Test infrastructure: nothing here is shared with the product, and nothing here is fast. `forward` takes a parsed config and a
 dict of tensors (numpy, any float type) and returns the logits of every position, optionally with the sum of the residual
-streams after every layer.
+streams after every layer. `act` is applied to every activation that may be kept in 16 bits (sublayer inputs, projections, keys and
+values, convolution outputs, gated outputs): with a rounding function it tells how much rounding alone moves the results.
 """
 import math
 
 import numpy as np
 
 F = np.float64
+
+
+def exact(v):
+    return v
 
 
 def rms_norm(x, eps, w=1.0):
@@ -68,17 +73,17 @@ def head_outputs(q, k, v, mask, scale, sinks):
     return o
 
 
-def keys_values(h, t, pre, mx):
+def keys_values(h, t, pre, mx, act=exact):
     S, G = h.shape[0], mx["kv_heads"]
-    return linear(t[pre + "k"], h).reshape(S, G, mx["dim"]), linear(t[pre + "v"], h).reshape(S, G, mx["vdim"])
+    return act(linear(t[pre + "k"], h)).reshape(S, G, mx["dim"]), act(linear(t[pre + "v"], h)).reshape(S, G, mx["vdim"])
 
 
-def attention(h, t, pre, mx, kv):
+def attention(h, t, pre, mx, kv, act=exact):
     """The mixer on h [S, width] with the keys and values kv (its own or another layer's)."""
     S, H = h.shape[0], mx["heads"]
-    q = linear(t[pre + "q"], h).reshape(S, H, mx["dim"])
+    q = act(linear(t[pre + "q"], h)).reshape(S, H, mx["dim"])
     o = head_outputs(q, kv[0], kv[1], mx.get("mask"), mx["scale"], t[pre + "sink"])
-    return linear(t[pre + "o"], o.reshape(S, H * mx["vdim"]))
+    return linear(t[pre + "o"], act(o.reshape(S, H * mx["vdim"])))
 
 
 # ------------------------------------------------------------------------------------------ state-space mixer
@@ -110,47 +115,53 @@ def ssm(x, B, C, dt, A_log, D, state=None):
     return y, st
 
 
-def gated_group_norm(y, z, w, groups, eps):
-    """rms norm of y * silu(z) in `groups` equal parts, times w."""
+def group_norm(y, w, groups, eps):
+    """rms norm of y in `groups` equal parts, times w."""
     S, n = y.shape
-    return rms_norm((y * silu(z)).reshape(S, groups, n // groups), eps).reshape(S, n) * w
+    return rms_norm(y.reshape(S, groups, n // groups), eps).reshape(S, n) * w
 
 
-def mamba2(h, t, pre, mx, eps):
-    S = h.shape[0]
+def mamba2(h, t, pre, mx, eps, act=exact):
+    p = act(linear(t[pre + "in"], h))
+    w = [t[pre + n] for n in ("conv", "conv.b", "dt_bias", "A_log", "D", "norm")]
+    return linear(t[pre + "o"], mamba2_inner(p, *w, mx, eps, act))
+
+
+def mamba2_inner(p, conv, conv_b, dt_bias, A_log, D, gain, mx, eps, act=exact):
+    """The mixer between its projections: p [S, z | x | B | C | dt] -> [S, inner]."""
+    S = p.shape[0]
     H, P, N, G = mx["heads"], mx["vdim"], mx["state"], mx["groups"]
     inner = H * P
-    p = linear(t[pre + "in"], h)
     z, xbc, dt = p[:, :inner], p[:, inner:2 * inner + 2 * G * N], p[:, 2 * inner + 2 * G * N:]
-    xbc = silu(causal_conv(xbc, t[pre + "conv"], t[pre + "conv.b"]))
+    xbc = act(silu(causal_conv(xbc, conv, conv_b)))
     x, B, C = xbc[:, :inner], xbc[:, inner:inner + G * N], xbc[:, inner + G * N:]
-    y, _ = ssm(x.reshape(S, H, P), B.reshape(S, G, N), C.reshape(S, G, N), softplus(dt + t[pre + "dt_bias"]), t[pre + "A_log"], t[pre + "D"])
-    return linear(t[pre + "o"], gated_group_norm(y.reshape(S, inner), z, t[pre + "norm"], mx["norm_groups"], eps))
+    y, _ = ssm(x.reshape(S, H, P), B.reshape(S, G, N), C.reshape(S, G, N), softplus(dt + dt_bias), A_log, D)
+    return act(group_norm(act(y.reshape(S, inner) * silu(z)), gain, mx["norm_groups"], eps))
 
 
 # ------------------------------------------------------------------------------------------ the model
-def feed_forward(h, t, pre):
-    return linear(t[pre + "down"], np.maximum(linear(t[pre + "up"], h), 0.0) ** 2)
+def feed_forward(h, t, pre, act=exact):
+    return linear(t[pre + "down"], act(np.maximum(linear(t[pre + "up"], h), 0.0) ** 2))
 
 
-def forward(cfg, tensors, tokens, want_layers=False):
+def forward(cfg, tensors, tokens, want_layers=False, act=exact):
     t = {k: np.asarray(v, F) for k, v in tensors.items()}
     eps, mult = cfg["norm"]["eps"], cfg["residual_mult"]
     xs = np.stack([t["embed"][np.asarray(tokens)]] * cfg["streams"])
     kv, trace = {}, []
     for i, spec in enumerate(cfg["layers"]):
         p, mx = "l%d." % i, spec["mixer"]
-        h = rms_norm(hyper_read(xs, t[p + "hc1.in"]), eps, t[p + "norm1"])
+        h = act(rms_norm(hyper_read(xs, t[p + "hc1.in"]), eps, t[p + "norm1"]))
         if spec["type"] == "mamba2":
-            y = mamba2(h, t, p + "mix.", mx, eps)
+            y = mamba2(h, t, p + "mix.", mx, eps, act)
         else:
             src = mx.get("kv_from")
-            kv[i] = kv[src] if src is not None else keys_values(h, t, p + "mix.", mx)
-            y = attention(h, t, p + "mix.", mx, kv[i])
+            kv[i] = kv[src] if src is not None else keys_values(h, t, p + "mix.", mx, act)
+            y = attention(h, t, p + "mix.", mx, kv[i], act)
         xs = hyper_write(xs, t[p + "hc1.mix"], t[p + "hc1.out"], mult, y)
         if spec["mlp"] is not None:
-            h = rms_norm(hyper_read(xs, t[p + "hc2.in"]), eps, t[p + "norm2"])
-            xs = hyper_write(xs, t[p + "hc2.mix"], t[p + "hc2.out"], mult, feed_forward(h, t, p + "mlp."))
+            h = act(rms_norm(hyper_read(xs, t[p + "hc2.in"]), eps, t[p + "norm2"]))
+            xs = hyper_write(xs, t[p + "hc2.mix"], t[p + "hc2.out"], mult, feed_forward(h, t, p + "mlp.", act))
         trace.append(xs.sum(0))
-    logits = linear(t["embed"], rms_norm(xs.sum(0), eps, t["final.norm"])) * cfg["logit_scale"]
+    logits = linear(t["embed"], act(rms_norm(xs.sum(0), eps, t["final.norm"]))) * cfg["logit_scale"]
     return (logits, np.stack(trace)) if want_layers else logits

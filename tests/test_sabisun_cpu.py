@@ -51,8 +51,7 @@ def test_restatement_convolution_and_recurrence():
 
 
 def test_restatement_norm_parts():
-    y, z = np.array([[3.0, 4.0, 1.0, 1.0]]), np.full((1, 4), 2.0)
-    got = P.gated_group_norm(y, z, np.ones(4), 2, 0.0)
+    got = P.group_norm(np.array([[3.0, 4.0, 1.0, 1.0]]), np.ones(4), 2, 0.0)
     assert np.allclose(got, [[3 / np.sqrt(12.5), 4 / np.sqrt(12.5), 1.0, 1.0]])
 
 

@@ -17,8 +17,7 @@ from test_pibidra_gpu import cuts_of, make, padded, run_cuts, up
 pytestmark = pytest.mark.gpu
 
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
-# bounds of the root mean square error over the logits' spread
-TOL = {"float32": 5e-5, "bfloat16": 0.06}
+TOL = 5e-5              # bound of the root mean square error over the logits' spread in 32 bits
 DT = {"float32": torch.float32, "bfloat16": torch.bfloat16}
 
 
@@ -27,6 +26,27 @@ def F():
     import flexllm_b200
     flexllm_b200.lib()
     return flexllm_b200
+
+
+def round16(v):
+    return bf16_round(np.asarray(v, np.float32)).astype(np.float64)
+
+
+class Reference:
+    """Exact logits of a model, and how much rounding alone moves each position's."""
+
+    def __init__(self, cfg, t, tok):
+        self.want = P.forward(cfg, t, tok)
+        self.rounding = rel_err(P.forward(cfg, t, tok, act=round16), self.want)
+
+    def check(self, dtype, got, what="", rows=slice(None)):
+        d = got - self.want[rows]
+        e = np.sqrt(((d - d.mean(-1, keepdims=True)) ** 2).mean(-1)) / self.want.std()
+        r = self.rounding[rows]
+        limit = TOL if dtype == "float32" else np.maximum(0.04, 4 * r)
+        assert (e < limit).all(), (dtype, what, int(e.argmax()), e.max(), r[e.argmax()])
+        if dtype == "bfloat16" and len(e) > 20:
+            assert np.median(e) < 1.5 * np.median(r), (what, np.median(e), np.median(r))
 
 
 def cuda(a):
@@ -102,16 +122,21 @@ class SsmCase:
         assert r.shape[2] == self.op.row
         return r
 
-    def want(self):
+    def want(self, act=P.exact):
         H, Pd, N, G, taps, parts = self.dims
-        out = []
-        for b in range(self.B):
-            u = np.concatenate([a[b].reshape(self.S, -1) for a in (self.x, self.Bm, self.C)], 1).astype(np.float64)
-            u = P.silu(P.causal_conv(u, self.cw.astype(np.float64), self.cb))
-            x, Bm, C = u[:, :H * Pd], u[:, H * Pd:H * Pd + G * N], u[:, H * Pd + G * N:]
-            y, _ = P.ssm(x.reshape(self.S, H, Pd), Bm.reshape(self.S, G, N), C.reshape(self.S, G, N), P.softplus(self.dt[b] + self.dtb), self.A_log, self.D)
-            out.append(P.gated_group_norm(y.reshape(self.S, -1), self.z[b].reshape(self.S, -1).astype(np.float64), self.gain, parts, self.eps))
-        return np.stack(out)
+        mx = dict(heads=H, vdim=Pd, state=N, groups=G, norm_groups=parts)
+        flat = lambda a, b: a[b].reshape(self.S, -1).astype(np.float64)
+        return np.stack([P.mamba2_inner(np.concatenate([flat(a, b) for a in (self.z, self.x, self.Bm, self.C, self.dt)], 1), self.cw.astype(np.float64),
+                                        self.cb, self.dtb, self.A_log, self.D, self.gain, mx, self.eps, act) for b in range(self.B)])
+
+    def check(self, got, what):
+        """fp32: close to the exact result; bf16: as close as rounding alone allows (rows in which terms cancel stand out)."""
+        want = self.want()
+        if self.dtype == torch.float32:
+            assert rms_rel(got, want).max() < 1e-5, what
+        else:
+            e, r = rms_rel(got, want), rms_rel(self.want(round16), want)
+            assert (e < np.maximum(1.5e-2, 4 * r)).all() and np.median(e) < 1.5 * np.median(r), (what, e.max(), r.max(), np.median(e), np.median(r))
 
     def run(self, cuts):
         H, Pd = self.dims[:2]
@@ -132,7 +157,8 @@ SSM_SHAPES = [  # heads, value size, state, groups, taps, parts of the norm
 
 
 def rms_rel(got, want):
-    return np.sqrt(((got - want) ** 2).mean(-1)).max() / np.sqrt((want ** 2).mean())
+    """Per row."""
+    return np.sqrt(((got - want) ** 2).mean(-1)) / np.sqrt((want ** 2).mean())
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -141,8 +167,7 @@ def test_state_space_shapes_and_portions(F, shape, dtype):
     S = 210
     for kind in ("whole", "portions", "tokens"):
         c = SsmCase(F, *shape, S, dtype=DT[dtype])
-        e = rms_rel(c.run(cuts_of(S, kind)), c.want())
-        assert e < (1e-5 if dtype == "float32" else 1.5e-2), (kind, e)
+        c.check(c.run(cuts_of(S, kind)), kind)
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -159,27 +184,25 @@ def test_state_space_memory(F, dtype):
         near = SsmCase(F, 2, 32, 32, 1, 3, 1, S, dtype=DT[dtype], A_log=(-6.0, -5.5), dt_bias=(-3.0, -2.5), seed=4)
         near.x[0, 20:] *= 0.05
         near.D[:] = 0.0
-        assert rms_rel(near.want()[:, 300:], want[:, 300:]) > 0.5
-        assert rms_rel(c.run(cuts_of(S, kind))[:, 300:], want[:, 300:]) < (1e-5 if dtype == "float32" else 2e-2), kind
+        assert np.median(rms_rel(near.want()[:, 300:], want[:, 300:])) > 0.5
+        c.check(c.run(cuts_of(S, kind)), kind)
 
 
 def test_state_space_extremes(F):
     """Decays that vanish within a token and steps that softplus leaves as they are or drives to zero."""
-    for dtype, tol in (("float32", 1e-5), ("bfloat16", 1.5e-2)):
+    for dtype in ("float32", "bfloat16"):
         for opts in (dict(A_log=(3.0, 4.0), dt_bias=(2.0, 5.0)), dict(A_log=(-9.0, -8.0), dt_bias=(-12.0, -9.0)), dict(dt_bias=(25.0, 40.0), A_log=(-8.0, -7.0))):
             for kind in ("whole", "portions"):
                 c = SsmCase(F, 4, 16, 24, 2, 4, 2, 150, dtype=DT[dtype], **opts)
-                e = rms_rel(c.run(cuts_of(150, kind)), c.want())
-                assert e < tol, (dtype, opts, kind, e)
+                c.check(c.run(cuts_of(150, kind)), (dtype, opts, kind))
 
 
 def test_state_space_batches_and_slots(F):
-    for dtype, tol in (("float32", 1e-5), ("bfloat16", 1.5e-2)):
+    for dtype in ("float32", "bfloat16"):
         c = SsmCase(F, 4, 24, 40, 2, 4, 3, 100, B=3, dtype=DT[dtype], seed=2)
-        want = c.want()
         other = c.op.state[3].clone()
         for cuts in ([100], cuts_of(100, "portions"), [60] + [1] * 40):            # the same slots again, old content in them
-            assert rms_rel(c.run(cuts), want) < tol
+            c.check(c.run(cuts), (dtype, cuts[:3]))
         assert torch.equal(c.op.state[3], other)                                  # a slot of nobody in the batch
 
 
@@ -350,7 +373,7 @@ def test_layers_and_logits(F, name, dtype):
     for i in range(len(layers)):
         e = np.sqrt(((got[i] - layers[i]) ** 2).mean()) / layers[i].std()
         assert e < (1e-5 if dtype == "float32" else 3e-2), (i, e)
-    assert rel_err(lg.cpu().numpy(), want).max() < TOL[dtype]
+    Reference(cfg, t, tok).check(dtype, lg.cpu().numpy())
     assert int(nx[0]) == int(lg[-1].argmax())
     m.close()
 
@@ -362,11 +385,10 @@ def test_portions_decoding_and_reuse(F, name, dtype):
     cfg = CONFIGS[name]
     t = weights(cfg, seed=3)
     tok = tokens(330, cfg["vocab"], seed=4)
-    want = P.forward(cfg, t, tok)
+    ref = Reference(cfg, t, tok)
     m = make(F, cfg, t, dtype, max_prefill=64, max_ctx=1200)
     for cuts in ([330], [200] + [1] * 130, cuts_of(330, "portions"), [2] * 165, [1] * 330, [330]):
-        e = rel_err(run_cuts(m, tok, cuts), want)
-        assert e.max() < TOL[dtype], (cuts[:4], int(e.argmax()), e.max())
+        ref.check(dtype, run_cuts(m, tok, cuts), cuts[:4])
         m.reset()
         m.step([tokens(97, cfg["vocab"], seed=len(cuts))])           # another request leaves its keys and states behind
     m.close()
@@ -376,11 +398,10 @@ def test_long_decoding(F):
     cfg = CONFIGS["plain"]
     t = weights(cfg, seed=5)
     tok = tokens(900, cfg["vocab"], seed=6)
-    want = P.forward(cfg, t, tok)
+    ref = Reference(cfg, t, tok)
     for dtype in ("float32", "bfloat16"):
         m = make(F, cfg, t, dtype, max_prefill=32, max_ctx=1000)
-        e = rel_err(run_cuts(m, tok, [300] + [1] * 600), want)
-        assert e.max() < TOL[dtype], (int(e.argmax()), e.max())
+        ref.check(dtype, run_cuts(m, tok, [300] + [1] * 600))
         m.close()
 
 
@@ -391,12 +412,11 @@ def test_many_state_heads_and_no_window(F):
     cfg = config([ssm(16, 32, 64, 4, 4, 8, 256), full, ssm(16, 32, 64, 4, 4, 1, 256)], 256, 1000, 2)
     t = weights(cfg, seed=15)
     tok = tokens(300, cfg["vocab"], seed=16)
-    want = P.forward(cfg, t, tok)
+    ref = Reference(cfg, t, tok)
     for dtype in ("float32", "bfloat16"):
         m = make(F, cfg, t, dtype, max_prefill=256, max_ctx=300)
         for cuts in ([300], [170] + [1] * 30 + [100]):
-            e = rel_err(run_cuts(m, tok, cuts), want)
-            assert e.max() < TOL[dtype], (dtype, int(e.argmax()), e.max())
+            ref.check(dtype, run_cuts(m, tok, cuts), cuts[:2])
         m.close()
 
 
@@ -465,7 +485,7 @@ def test_batch_steps(F, B):
             at += n
         got = np.concatenate(got, 1)
         for b in {0, B // 2, B - 1}:
-            assert rel_err(got[b], P.forward(cfg, t, toks[b])).max() < TOL[dtype]
+            Reference(cfg, t, toks[b]).check(dtype, got[b], b)
         m.close()
 
 
@@ -478,8 +498,7 @@ def test_extend_after_generation(F):
     out = m.generate([p], 8)[0]
     seq = p + out + tokens(20, cfg["vocab"], seed=2)                    # the last generated token has not been fed yet
     lg, _ = m.step([seq[57:]], range(len(seq) - 57))
-    e = rel_err(np.frombuffer(lg, np.float32).reshape(-1, m.vocab), P.forward(cfg, t, seq)[57:])
-    assert e.max() < TOL["float32"], e.max()
+    Reference(cfg, t, seq).check("float32", np.frombuffer(lg, np.float32).reshape(-1, m.vocab), rows=slice(57, None))
     m.close()
 
 
@@ -528,8 +547,6 @@ def test_folder_command_line_and_replay(F, tmp_path):
                            input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True)
         assert r.returncode == 0, r.stderr
         got = {i: np.fromfile(os.path.join(out, "%d.f32" % i), np.float32).reshape(-1, cfg["vocab"]) for i in (0, 2, 3, 4, 5)}
-        wa, wb = P.forward(cfg, t, a), P.forward(cfg, t, b)
-        for i, w in ((0, wa[:80]), (2, wa[82:83]), (3, wa[83:84]), (4, wa[84:]), (5, wb)):
-            d = got[i] - w
-            e = np.sqrt(((d - d.mean(1, keepdims=True)) ** 2).mean(1)) / wa.std()
-            assert e.max() < TOL[dtype], (dtype, i, e.max())
+        ra, rb = Reference(cfg, t, a), Reference(cfg, t, b)
+        for i, ref, rows in ((0, ra, slice(0, 80)), (2, ra, slice(82, 83)), (3, ra, slice(83, 84)), (4, ra, slice(84, None)), (5, rb, slice(None))):
+            ref.check(dtype, got[i], i, rows)
