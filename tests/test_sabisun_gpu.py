@@ -184,7 +184,7 @@ def test_state_space_memory(F, dtype):
         near = SsmCase(F, 2, 32, 32, 1, 3, 1, S, dtype=DT[dtype], A_log=(-6.0, -5.5), dt_bias=(-3.0, -2.5), seed=4)
         near.x[0, 20:] *= 0.05
         near.D[:] = 0.0
-        assert np.median(rms_rel(near.want()[:, 300:], want[:, 300:])) > 0.5
+        assert np.median(rms_rel(near.want()[:, 300:], want[:, 300:])) > 0.3
         c.check(c.run(cuts_of(S, kind)), kind)
 
 
