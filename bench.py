@@ -577,12 +577,14 @@ def micro(args):
         synthetic.load_random_weights(m, max_ctx=1040, seed=0, **cfg2)
         tok = torch.randint(0, CFG["vocab"], (8, 1024), dtype=torch.int32).cuda()
         fn = lambda: m.prefill(tok)
-    elif name in ("pibidra_prefill", "pibidra_decode"):      # two layers of the Llama's sizes: every kernel of the family at its model shapes
-        S, B = 1024, 8 if name == "pibidra_prefill" else 4
-        m = pibidra_model(F, torch, PIBIDRA_SIZES["llama1b"], B, S, S + 64, layers=2)
+    elif name in ("pibidra_prefill", "pibidra_decode", "sabisun_prefill", "sabisun_decode"):   # a few layers of the Llama's sizes: every kernel of the family
+        family, what = name.split("_")
+        S, B = 1024, 8 if what == "prefill" else 4
+        m = pibidra_model(F, torch, PIBIDRA_SIZES["llama1b"], B, S, S + 64, layers=2) if family == "pibidra" else \
+            sabisun_model(F, torch, SABISUN_SIZES["llama1b"], B, S, S + 64, layers=4)
         tok = torch.randint(0, CFG["vocab"], (B, S), dtype=torch.int32).cuda()
         m.prefill(tok); m.begin(32)
-        fn = (lambda: m.prefill(tok)) if name == "pibidra_prefill" else (lambda: m.decode(4, False))
+        fn = (lambda: m.prefill(tok)) if what == "prefill" else (lambda: m.decode(4, False))
     elif name == "decode_step":         # whole-model decode steps (one persistent kernel each) at a short context: small enough for ncu
         S, n = 128, 6
         m = F.Model(max_batch=BATCH, max_prefill=S, max_ctx=S + 16, **CFG)
@@ -684,6 +686,17 @@ def graph_ms(torch, fn, n=40):
     return e0.elapsed_time(e1) / n
 
 
+def prefill_decode_ms(torch, m, vocab, B, S, n_dec, args):
+    """Device times of a prefill of B prompts of S and of a decode step after it."""
+    tok = torch.randint(0, vocab, (B, S), dtype=torch.int32).cuda()
+    pre = event_ms(torch, lambda i: m.prefill(tok), max(2, args.steps), warm=args.warmup)
+    m.prefill(tok); m.begin(2 * n_dec + 8)
+    m.decode(8, True); torch.cuda.synchronize()
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    e0.record(); m.decode(n_dec, True); e1.record(); torch.cuda.synchronize()
+    return pre, e0.elapsed_time(e1) / n_dec
+
+
 def pibidra_kernels(F, torch, peaks):
     """The family's kernels beside the like kernels of the W8A8 Llama at the Llama's layer sizes: time and fraction of the
     roofline (bf16 products against the measured bf16 peak, int8 ones against twice that; bytes against the copy rate)."""
@@ -765,15 +778,7 @@ def pibidra_arm(args):
     line = {"metric": "pibidra_prefill_decode", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic, random weights", "n_gpus": 1, "sizes": {},
             "config": {"prefill_len": S, "decode_steps": n_dec, "window": "as listed", "l2": "weights exceed the 126 MB L2 (small: 0.4 GB); no flush"}}
 
-    def measure(m, vocab, B):
-        tok = torch.randint(0, vocab, (B, S), dtype=torch.int32).cuda()
-        pre = event_ms(torch, lambda i: m.prefill(tok), max(2, args.steps), warm=args.warmup)
-        m.prefill(tok); m.begin(2 * n_dec + 8)
-        m.decode(8, True); torch.cuda.synchronize()
-        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        e0.record(); m.decode(n_dec, True); e1.record(); torch.cuda.synchronize()
-        return pre, e0.elapsed_time(e1) / n_dec
-
+    measure = lambda m, vocab, B: prefill_decode_ms(torch, m, vocab, B, S, n_dec, args)
     for name, z in PIBIDRA_SIZES.items():
         rows = {}
         for B in (1, 4, 32):
@@ -797,6 +802,183 @@ def pibidra_arm(args):
     line["value"] = line["sizes"]["llama1b"]["batch32"]["decode_tokens_per_s"]
     if not args.no_extras:
         line["kernels"] = pibidra_kernels(F, torch, peaks)
+    line["clocks"] = sampler.stop()
+    print(json.dumps(line))
+
+
+# ------------------------------------------------------------------------------------ the Sabisun family
+# the Pibidra sizes with state-space mixers in three of four layers (inner size twice the width) and windowed attention in the
+# rest, every second one with the keys and values of the one before; two residual streams
+SABISUN_SIZES = {n: dict(z, ssm_heads=2 * z["width"] // 64, ssm_vdim=64, state=128, groups=8, conv=4, streams=2, keep=4) for n, z in PIBIDRA_SIZES.items()}
+
+
+def sabisun_config(z, layers=None):
+    out, last = [], None
+    for i in range(layers or z["layers"]):
+        mlp = {"kind": "dense", "ff": z["ff"]}
+        if i % 4 != 3:
+            out.append({"type": "mamba2", "mlp": mlp, "mixer": dict(heads=z["ssm_heads"], vdim=z["ssm_vdim"], state=z["state"], groups=z["groups"],
+                                                                    conv=z["conv"], norm_groups=z["groups"])})
+            continue
+        m = dict(heads=z["heads"], kv_heads=z["kv_heads"], dim=z["dim"], vdim=z["vdim"], mask={"size": z["window"], "keep_first": z["keep"]}, scale=z["dim"] ** -0.5)
+        if last is not None:
+            m["kv_from"], last = last, None
+        else:
+            last = i
+        out.append({"type": "attention", "mixer": m, "mlp": mlp})
+    return {"architecture": "Sabisun", "layers": out, "logit_scale": 1.0, "norm": {"eps": 1e-5}, "residual_mult": 1.0, "streams": z["streams"],
+            "vocab": z["vocab"], "width": z["width"]}
+
+
+def sabisun_model(F, torch, z, max_batch, max_prefill, max_ctx, layers=None, seed=0):
+    """A model of size z with random bf16 weights, made on the device."""
+    from flexllm_b200 import models
+    cfg = sabisun_config(z, layers)
+    m = F.Model.adopt(models.create(cfg, max_batch, max_prefill, max_ctx, "bfloat16"))
+    g = torch.Generator(device="cuda").manual_seed(seed)
+    D, V, n = z["width"], z["vocab"], z["streams"]
+    rn = lambda *sh, s=1.0: (torch.randn(sh, device="cuda", generator=g) * s).to(torch.bfloat16)
+    m.load_tensor("embed", rn(V, D, s=D ** -0.5)); m.load_tensor("final.norm", 1 + rn(D, s=0.1))
+    for i, l in enumerate(cfg["layers"]):
+        p, x = "l%d." % i, l["mixer"]
+        for q in "12":
+            m.load_tensor(p + "norm" + q, 1 + rn(D, s=0.1))
+            m.load_tensor(p + "hc" + q + ".in", 0.5 + rn(n, s=0.1)); m.load_tensor(p + "hc" + q + ".out", 1 + rn(n, s=0.1))
+            m.load_tensor(p + "hc" + q + ".mix", (torch.eye(n, device="cuda") * 0.9).to(torch.bfloat16) + rn(n, n, s=0.05))
+        if l["type"] == "mamba2":
+            inner, ch = x["heads"] * x["vdim"], x["heads"] * x["vdim"] + 2 * x["groups"] * x["state"]
+            t = {"in": rn(inner + ch + x["heads"], D, s=D ** -0.5), "conv": rn(ch, x["conv"], s=0.5), "conv.b": rn(ch, s=0.1), "dt_bias": rn(x["heads"]) - 3,
+                 "A_log": rn(x["heads"]), "D": 1 + rn(x["heads"], s=0.1), "norm": 1 + rn(inner, s=0.1), "o": rn(D, inner, s=inner ** -0.5)}
+        else:
+            H, G, dk, dv = x["heads"], x["kv_heads"], x["dim"], x["vdim"]
+            t = {"q": rn(H * dk, D, s=D ** -0.5), "sink": rn(H), "o": rn(D, H * dv, s=(H * dv) ** -0.5)}
+            if "kv_from" not in x:
+                t.update(k=rn(G * dk, D, s=D ** -0.5), v=rn(G * dv, D, s=D ** -0.5))
+        for k, v in t.items():
+            m.load_tensor(p + "mix." + k, v)
+        m.load_tensor(p + "mlp.up", rn(z["ff"], D, s=D ** -0.5)); m.load_tensor(p + "mlp.down", rn(D, z["ff"], s=z["ff"] ** -0.5))
+    return m
+
+
+def sabisun_work(z, B, S, ctx):
+    """(prefill FLOPs of B prompts of S, bytes one decode step of B sequences at context ctx has to read or write)."""
+    D, ff, V, W = (z[k] for k in ("width", "ff", "vocab", "window"))
+    pairs = sum(min(i + 1, W) for i in range(S))
+    flops, w, moved = 2.0 * B * V * D, V * D, 0.0
+    for l in sabisun_config(z)["layers"]:
+        x = l["mixer"]
+        lw = 2 * D * ff
+        if l["type"] == "mamba2":
+            inner, gn = x["heads"] * x["vdim"], x["groups"] * x["state"]
+            lw += D * (3 * inner + 2 * gn + x["heads"])
+            flops += 4.0 * B * S * inner * x["state"]
+            moved += B * inner * x["state"] * 8.0                          # the state, read and written
+        else:
+            H, G, dk, dv = x["heads"], x["kv_heads"], x["dim"], x["vdim"]
+            lw += D * H * (dk + dv) + (0 if "kv_from" in x else D * G * (dk + dv))
+            flops += 2.0 * B * H * (dk + dv) * pairs
+            moved += 2.0 * B * min(ctx, W) * G * (dk + dv)
+        flops += 2.0 * B * S * lw
+        w += lw
+    return flops, 2.0 * w + moved
+
+
+def sabisun_kernels(F, torch, peaks):
+    """The family's kernels beside the like kernels of Pibidra at the 1B layer sizes: time and fraction of the roofline."""
+    hbm, tf = peaks.get("hbm_gbs") or 6650.0, peaks.get("bf16_tflops") or 1590.0
+    out = {}
+
+    def note(name, ms, flops=0.0, nbytes=0.0):
+        floor = max(flops / tf / 1e9, nbytes / hbm / 1e6)
+        out[name] = {"us": round(ms * 1e3, 2), "roofline": round(floor / ms, 4)}
+
+    bf = lambda *sh: torch.randn(sh, device="cuda").to(torch.bfloat16)
+    # products: the state-space input projection, the squared-ReLU up projection and its like
+    for N, K, kw in ((10304, 2048, {}), (2048, 4096, {}), (8192, 2048, dict(relu2=True)), (16384, 2048, dict(gelu_gate=True))):
+        label = " squared relu" if "relu2" in kw else " gated gelu (Pibidra)" if kw else ""
+        M, n_out = 8192, N // 2 if "gelu_gate" in kw else N
+        a, w = bf(M, K), bf(N, K)
+        note(f"prompt product {M}x{N}x{K}{label}", event_ms(torch, lambda i: F.linear_float(a, w, **kw), 20), 2.0 * M * N * K, 2.0 * (M * K + N * K + M * n_out))
+        ws = [bf(N, K) for _ in range(max(2, int(300e6 // (2 * N * K)) + 1))]
+        for B in (1, 4, 32):
+            a = bf(B, K)
+            note(f"decode product {B}x{N}x{K}{label}", graph_ms(torch, lambda i: F.linear_float(a, ws[i % len(ws)], **kw)), 2.0 * B * N * K, 2.0 * N * K)
+        del ws
+    # norms of 32768 rows
+    M, D, g = 32768, 2048, torch.ones(2048, device="cuda")
+    y = torch.randn((M, D), device="cuda")
+    for n in (2, 4):
+        x, c = torch.randn((M, n, D), device="cuda"), torch.ones(n, device="cuda")
+        mix = torch.eye(n, device="cuda")
+        note(f"streams {M}x{n}x{D} (mix, add, norm)", event_ms(torch, lambda i: F.hyper_norm(x, D, 1e-5, y, mix, c, c, g, torch.bfloat16), 20), 0, M * D * (8.0 * n + 6))
+        del x
+    x = torch.randn((M, D), device="cuda")
+    note(f"norms {M}x{D} (Pibidra: norm, add, norm)", event_ms(torch, lambda i: F.sandwich_norm(x, D, 1e-5, y, g, None, g, torch.bfloat16), 20), 0, M * D * 14.0)
+    del x, y
+    # attention: prompts of 4 x 1024 (window 1024 and 256), decoding of 64 sequences at context 4096
+    H, G, dk = 32, 8, 64
+    pages = lambda B, S: torch.arange(B * (S // 64 + 1), dtype=torch.int32, device="cuda").reshape(B, -1)
+    kept = lambda B, S, W: F.WindowAttention(H, G, dk, dk, W, dk ** -0.5, 0.0, None, 0, None, None, pages(B, S), B * (S // 64 + 1), S, sink=False, gate=False,
+                                             keep_first=4, sinks=torch.ones(H, device="cuda"))
+    full = lambda B, S, W: F.WindowAttention(H, G, dk, dk, W, dk ** -0.5, 30.0, torch.randn((32, H)), W, torch.ones(H * dk, device="cuda"),
+                                             torch.ones(G * dk, device="cuda"), pages(B, S), B * (S // 64 + 1), S)
+    for who, mk in (("", kept), (" (Pibidra)", full)):
+        for W in (1024, 256):
+            B, S = 4, 1024
+            op = mk(B, S, W)
+            proj, ctx = bf(B * S, op.row), torch.zeros(B, dtype=torch.int32, device="cuda")
+            note(f"prompt attention {B}x{S}, window {W}{who}", event_ms(torch, lambda i: op(proj, ctx), 20), 4.0 * B * H * dk * sum(min(i + 1, W) for i in range(S)))
+            op.close()
+        B, S = 64, 4096
+        op = mk(B, S, S)
+        proj, ctx = bf(B, op.row), torch.full((B,), S - 1, dtype=torch.int32, device="cuda")
+        note(f"decode attention {B} sequences, {S} keys{who}", event_ms(torch, lambda i: op(proj, ctx), 20), 0, 2.0 * B * S * G * 2 * dk)
+        op.close()
+    # state-space mixer between its projections: 64 heads of 64, state 128, 8 groups
+    H, P, N, G, taps = 64, 64, 128, 8, 4
+    ch = H * P + 2 * G * N
+    for B, S in ((8, 1024), (1, 8192), (64, 1), (1, 1)):
+        f32 = lambda *sh: torch.rand(sh, device="cuda")
+        op = F.StateSpaceMixer(H, P, N, G, taps, G, f32(taps, ch) - 0.5, f32(ch), f32(H) - 3, -f32(H) - 0.1, f32(H), f32(H * P), B)
+        ctx = torch.full((B,), 64, dtype=torch.int32, device="cuda")
+        projs = [bf(B * S, op.row) for _ in range(3 if S > 1 else 1)]
+        name = f"state-space mixer {B}x{S}" + (" tokens" if S > 1 else " token")
+        note(name, event_ms(torch, lambda i: op(projs[i % len(projs)], ctx), 20) if S > 1 else graph_ms(torch, lambda i: op(projs[0], ctx)),
+             4.0 * B * S * H * P * N, 2.0 * B * S * (op.row + H * P) + 8.0 * B * H * P * N)
+    return out
+
+
+def sabisun_arm(args):
+    """python bench.py --design sabisun: prefill and decode throughput of the Sabisun family at a few sizes, Pibidra at the same
+    sizes, and the kernels of both. One JSON line."""
+    import torch
+    import flexllm_b200 as F
+    torch.cuda.set_device(0)
+    F.lib()
+    try:
+        peaks = json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))
+    except Exception:
+        peaks = {}
+    hbm, tf = peaks.get("hbm_gbs") or 6650.0, peaks.get("bf16_tflops_sustained") or 1400.0
+    sampler = ClockSampler(0); sampler.start(); sampler.mark()
+    S, n_dec = 1024, 64
+    line = {"metric": "sabisun_prefill_decode", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic, random weights", "n_gpus": 1, "sizes": {},
+            "config": {"prefill_len": S, "decode_steps": n_dec, "window": "as listed", "l2": "weights exceed the 126 MB L2 (small: 0.4 GB); no flush"}}
+    for name, z in SABISUN_SIZES.items():
+        rows = {}
+        for who, make, work in (("", sabisun_model, sabisun_work), ("pibidra_", pibidra_model, pibidra_work)):
+            for B in (1, 4, 32):
+                m = make(F, torch, z, B, S, S + 2 * n_dec + 16)
+                pre, dec = prefill_decode_ms(torch, m, z["vocab"], B, S, n_dec, args)
+                m.close()
+                fl, by = work(z, B, S, S + n_dec // 2)
+                rows["%sbatch%d" % (who, B)] = {
+                    "prefill_ms": round(pre, 3), "prefill_tokens_per_s": round(B * S / pre * 1e3), "prefill_tflops_frac": round(fl / pre / 1e9 / tf, 3),
+                    "decode_ms": round(dec, 4), "decode_tokens_per_s": round(B / dec * 1e3), "decode_hbm_frac": round(by / dec / 1e6 / hbm, 3)}
+        line["sizes"][name] = dict(shape=z, **rows)
+    line["value"] = line["sizes"]["llama1b"]["batch32"]["decode_tokens_per_s"]
+    if not args.no_extras:
+        line["kernels"] = sabisun_kernels(F, torch, peaks)
     line["clocks"] = sampler.stop()
     print(json.dumps(line))
 
@@ -1020,12 +1202,13 @@ def main():
                     help="N > 1: headline partition - tensor parallel over the N GPUs with a fixed total batch of 32 (default: the "
                          "partition the workload names), or independent batch-parallel replicas; the other one is reported under "
                          "other_partition")
-    ap.add_argument("--design", default="llama", choices=["llama", "pibidra"],
-                    help="pibidra: throughput of that model family at a few sizes beside the W8A8 Llama (one GPU) instead of the headline workload")
+    ap.add_argument("--design", default="llama", choices=["llama", "pibidra", "sabisun"],
+                    help="pibidra, sabisun: throughput of that model family at a few sizes beside the W8A8 Llama or Pibidra (one GPU) instead "
+                         "of the headline workload")
     ap.add_argument("--decode-len", type=int, default=NEW)
     ap.add_argument("--no-extras", action="store_true", help="skip roofline kernel timing and the CPU baseline")
     ap.add_argument("--micro", default=None, help="run one kernel on a small case and exit (attn_prefill, attn_prefill_online, gemm_prefill, "
-                                                  "gemm_prefill_k8192, decode_linear, gemv_b1, decode_attention, swiglu_fht, rmsnorm_prefill, prefill_small, decode_step, pibidra_prefill, pibidra_decode)")
+                                                  "gemm_prefill_k8192, decode_linear, gemv_b1, decode_attention, swiglu_fht, rmsnorm_prefill, prefill_small, decode_step, pibidra_prefill, pibidra_decode, sabisun_prefill, sabisun_decode)")
     args = ap.parse_args()
     globals()["NEW"] = args.decode_len
     args.warmup = max(args.warmup, 0)
@@ -1034,6 +1217,9 @@ def main():
         return
     if args.design == "pibidra":
         pibidra_arm(args)
+        return
+    if args.design == "sabisun":
+        sabisun_arm(args)
         return
     if args.impl == "reference":
         if env_int("RANK", 0) == 0:
