@@ -56,6 +56,20 @@ template <class T> __device__ __forceinline__ void keep_history(const SsmCall& k
 // ---------------------------------------------------------------------------------------------------------------
 // Convolution and silu: one thread has 8 channels of TT consecutive tokens. TAPS 0: any number of taps.
 constexpr int kConvTokens = 8;
+// 8 elements as they lie in memory
+template <class T> struct Vec8;
+template <> struct Vec8<bf16> {
+    uint4 v;
+    __device__ __forceinline__ void load(const bf16* p) { v = *reinterpret_cast<const uint4*>(p); }
+    __device__ __forceinline__ void zero() { v = make_uint4(0, 0, 0, 0); }
+    __device__ __forceinline__ void get(float (&f)[8]) const { unpack8(v, f); }
+};
+template <> struct Vec8<float> {
+    float4 a, b;
+    __device__ __forceinline__ void load(const float* p) { a = load4(p); b = load4(p + 4); }
+    __device__ __forceinline__ void zero() { a = b = make_float4(0.f, 0.f, 0.f, 0.f); }
+    __device__ __forceinline__ void get(float (&f)[8]) const { f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w; }
+};
 template <class T, int TAPS>
 __global__ void __launch_bounds__(128) ssm_conv_kernel(const SsmCall k) {
     constexpr bool FAST = sizeof(T) == 2;
@@ -78,25 +92,29 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const SsmCall k) {
     float bias[8];
     load8(k.conv_b + c, bias);
     if constexpr (TAPS > 0) {
-        float w[TAPS][8], h[TAPS][8];                       // h: inputs of the last TAPS positions, oldest first
+        float w[TAPS][8];
+        Vec8<T> in[TAPS - 1 + kConvTokens];                 // all inputs are asked for before the first is used
+#pragma unroll
+        for (int j = 0; j < TAPS - 1 + kConvTokens; j++) {
+            const int at = p0 + t0 - (TAPS - 1) + j;
+            if (at >= 0 && at < p0 + t1) in[j].load(conv_row<T>(k, b, p0, at) + c); else in[j].zero();
+        }
 #pragma unroll
         for (int j = 0; j < TAPS; j++) load8(k.conv_w + (long)j * s.ch + c, w[j]);
 #pragma unroll
-        for (int j = 1; j < TAPS; j++) load(p0 + t0 - TAPS + j, h[j]);
-        for (int t = t0; t < t1; t++) {
-#pragma unroll
-            for (int j = 0; j + 1 < TAPS; j++)
-#pragma unroll
-                for (int e = 0; e < 8; e++) h[j][e] = h[j + 1][e];
-            load(p0 + t, h[TAPS - 1]);
+        for (int t = 0; t < kConvTokens; t++) {
+            if (t0 + t >= t1) break;
             float v[8];
 #pragma unroll
-            for (int e = 0; e < 8; e++) {
-                v[e] = bias[e];
+            for (int e = 0; e < 8; e++) v[e] = bias[e];
 #pragma unroll
-                for (int j = 0; j < TAPS; j++) v[e] = __fmaf_rn(w[j][e], h[j][e], v[e]);
+            for (int j = 0; j < TAPS; j++) {
+                float x[8];
+                in[t + j].get(x);
+#pragma unroll
+                for (int e = 0; e < 8; e++) v[e] = __fmaf_rn(w[j][e], x[e], v[e]);
             }
-            put(t, v);
+            put(t0 + t, v);
         }
     } else {
         for (int t = t0; t < t1; t++) {
@@ -116,34 +134,33 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const SsmCall k) {
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// Recurrence token by token: a CTA has 32 value dimensions of one head, 8 lanes share a state row (NV float4 each). FUSED: one
+// Recurrence token by token: a CTA has 32 PR value dimensions of one head, 8 lanes share a state row (NV float4 each). FUSED: one
 // token per sequence, with its convolution.
-template <class T, int NV, bool FUSED>
+template <class T, int NV, int PR, bool FUSED>
 __global__ void __launch_bounds__(256) ssm_scan_kernel(const SsmCall k) {
     constexpr bool FAST = sizeof(T) == 2;
-    constexpr int TT = FUSED ? 1 : kScanTile, NW = 32 * NV;
+    constexpr int TT = FUSED ? 1 : kScanTile, NW = 32 * NV, NP = 32 * PR;
     __shared__ __align__(16) float b_sm[TT][NW], c_sm[TT][NW];
-    __shared__ float x_sm[TT][32], dt_sm[TT], dec_sm[TT];
+    __shared__ float x_sm[TT][NP], dt_sm[TT], dec_sm[TT];
     const SsmShape& s = k.s;
     const int tid = threadIdx.x, h = blockIdx.y, b = blockIdx.z, g = h / (s.H / s.G);
-    const int pb = blockIdx.x * 32, p = pb + (tid >> 3), ns = tid & 7;
-    const bool on = p < s.P;
+    const int pb = blockIdx.x * NP, pr = tid >> 3, ns = tid & 7;            // rows pr, pr + 32, ..
     pdl_sync();
     const int p0 = first_pos(k, b);
-    float* st = k.state + (((long)b * s.H + h) * s.P + (on ? p : 0)) * s.Np;
-    float4 S[NV];
+    float* st = k.state + (((long)b * s.H + h) * s.P + pb + pr) * s.Np + 4 * ns;
+    float4 S[PR][NV];
 #pragma unroll
-    for (int i = 0; i < NV; i++) {
-        const int n = 32 * i + 4 * ns;
-        S[i] = on && p0 > 0 && n < s.Np ? load4(st + n) : make_float4(0.f, 0.f, 0.f, 0.f);
-    }
+    for (int r = 0; r < PR; r++)
+#pragma unroll
+        for (int i = 0; i < NV; i++)
+            S[r][i] = pb + pr + 32 * r < s.P && p0 > 0 && 32 * i + 4 * ns < s.Np ? load4(st + (long)32 * r * s.Np + 32 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
     const float A = k.A[h], Dh = k.D[h], dtb = k.dt_bias[h];
     const int xc = h * s.P8 + pb, bc = s.inner + g * s.N8, cc = bc + s.G * s.N8;       // first channels of x, B and C
     for (int t0 = 0; t0 < k.Sc; t0 += TT) {
         const int nt = min(TT, k.Sc - t0);
         if (t0) __syncthreads();
-        for (int i = tid; i < nt * (2 * NW + 32); i += 256) {
-            const int t = i / (2 * NW + 32), j = i - t * (2 * NW + 32);
+        for (int i = tid; i < nt * (2 * NW + NP); i += 256) {
+            const int t = i / (2 * NW + NP), j = i - t * (2 * NW + NP);
             const int e = j < NW ? j : j < 2 * NW ? j - NW : j - 2 * NW;
             const bool in = j < 2 * NW ? e < s.N8 : pb + e < s.P8;
             const int c = (j < NW ? bc : j < 2 * NW ? cc : xc) + e;
@@ -159,29 +176,41 @@ __global__ void __launch_bounds__(256) ssm_scan_kernel(const SsmCall k) {
         }
         __syncthreads();
         for (int t = 0; t < nt; t++) {
-            const float x = x_sm[t][tid >> 3], dec = dec_sm[t], dx = dt_sm[t] * x;
-            float y = 0.0f;
+            const float dec = dec_sm[t];
+            float y[PR];
 #pragma unroll
-            for (int i = 0; i < NV; i++) {
-                const float4 bv = load4(&b_sm[t][32 * i + 4 * ns]), cv = load4(&c_sm[t][32 * i + 4 * ns]);
-                S[i].x = __fmaf_rn(S[i].x, dec, bv.x * dx); S[i].y = __fmaf_rn(S[i].y, dec, bv.y * dx);
-                S[i].z = __fmaf_rn(S[i].z, dec, bv.z * dx); S[i].w = __fmaf_rn(S[i].w, dec, bv.w * dx);
-                y = __fmaf_rn(S[i].x, cv.x, y); y = __fmaf_rn(S[i].y, cv.y, y); y = __fmaf_rn(S[i].z, cv.z, y); y = __fmaf_rn(S[i].w, cv.w, y);
+            for (int r = 0; r < PR; r++) {
+                const float dx = dt_sm[t] * x_sm[t][pr + 32 * r];
+                y[r] = 0.0f;
+#pragma unroll
+                for (int i = 0; i < NV; i++) {
+                    const float4 bv = load4(&b_sm[t][32 * i + 4 * ns]), cv = load4(&c_sm[t][32 * i + 4 * ns]);
+                    float4& q = S[r][i];
+                    q.x = __fmaf_rn(q.x, dec, bv.x * dx); q.y = __fmaf_rn(q.y, dec, bv.y * dx);
+                    q.z = __fmaf_rn(q.z, dec, bv.z * dx); q.w = __fmaf_rn(q.w, dec, bv.w * dx);
+                    y[r] = __fmaf_rn(q.x, cv.x, y[r]); y[r] = __fmaf_rn(q.y, cv.y, y[r]); y[r] = __fmaf_rn(q.z, cv.z, y[r]); y[r] = __fmaf_rn(q.w, cv.w, y[r]);
+                }
             }
 #pragma unroll
-            for (int o = 4; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-            if (ns == 0 && p < s.P8) {
-                const long r = (long)b * k.Sc + t0 + t;
+            for (int o = 4; o > 0; o >>= 1)
+#pragma unroll
+                for (int r = 0; r < PR; r++) y[r] += __shfl_xor_sync(0xffffffffu, y[r], o);
+#pragma unroll
+            for (int r = 0; r < PR; r++) {
+                const int p = pb + pr + 32 * r;
+                if (ns != 0 || p >= s.P8) continue;
+                const long row = (long)b * k.Sc + t0 + t;
                 const int col = h * s.P8 + p;
-                const float z = to_f(((const T*)k.proj)[r * s.ld + col]);
-                ((T*)k.y)[r * s.inner + col] = from_f<T>(on ? __fmaf_rn(Dh, x, y) * silu_t<FAST>(z) : 0.0f);
+                const float z = to_f(((const T*)k.proj)[row * s.ld + col]);
+                ((T*)k.y)[row * s.inner + col] = from_f<T>(p < s.P ? __fmaf_rn(Dh, x_sm[t][pr + 32 * r], y[r]) * silu_t<FAST>(z) : 0.0f);
             }
         }
     }
-    if (on)
+#pragma unroll
+    for (int r = 0; r < PR; r++)
 #pragma unroll
         for (int i = 0; i < NV; i++)
-            if (32 * i + 4 * ns < s.Np) store4(st + 32 * i + 4 * ns, S[i]);
+            if (pb + pr + 32 * r < s.P && 32 * i + 4 * ns < s.Np) store4(st + (long)32 * r * s.Np + 32 * i, S[r][i]);
     keep_history<T>(k, b, p0, blockIdx.x + gridDim.x * blockIdx.y, gridDim.x * gridDim.y);
 }
 
@@ -283,23 +312,23 @@ __device__ __forceinline__ void split2(float x, float y, uint32_t* hi, uint32_t*
     *lo = bf_pack(x - bf_lo(h), y - bf_hi(h));
 }
 
-struct ChunkSmem { uint32_t c, b, x, s, f, total; };        // byte offsets; C, B and x twice (the next chunk is in flight)
-__host__ __device__ constexpr ChunkSmem chunk_smem(int NK, int PT) {
+struct ChunkSmem { uint32_t c, b, x, s, f, total; };        // byte offsets; NB buffers of C, B and x
+__host__ __device__ constexpr ChunkSmem chunk_smem(int NK, int PT, int NB) {
     ChunkSmem o{};
     const uint32_t rn = (uint32_t)(NK * 16 + 8) * 2, rp = (uint32_t)(PT * 8 + 8) * 2;       // row pitches
     o.c = 0;
-    o.b = o.c + 2 * kChunk * rn;
-    o.x = o.b + 2 * kChunk * rn;
-    o.s = o.x + 2 * kChunk * rp;                             // state, hi then lo: [NK * 16][PT * 8]
+    o.b = o.c + NB * kChunk * rn;
+    o.x = o.b + NB * kChunk * rn;
+    o.s = o.x + NB * kChunk * rp;                            // state, hi then lo: [NK * 16][PT * 8]
     o.f = o.s + 2 * NK * 16 * rp;                            // cum [64], dt [64], weight [64]
     o.total = o.f + 3 * kChunk * 4;
     return o;
 }
 
-template <int NK, int PT>
-__global__ void __launch_bounds__(128) ssm_chunk_kernel(const SsmCall k) {
+template <int NK, int PT, int NB, int CTAS>
+__global__ void __launch_bounds__(128, CTAS) ssm_chunk_kernel(const SsmCall k) {
     constexpr int MT = NK / 4;                               // 16-row blocks of the state per warp
-    constexpr ChunkSmem o = chunk_smem(NK, PT);
+    constexpr ChunkSmem o = chunk_smem(NK, PT, NB);
     constexpr uint32_t RN = (NK * 16 + 8) * 2, RP = (PT * 8 + 8) * 2;
     extern __shared__ __align__(16) uint8_t sm[];
     const SsmShape& s = k.s;
@@ -308,7 +337,6 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(const SsmCall k) {
     const uint32_t base = (uint32_t)__cvta_generic_to_shared(sm);
     float *cum = reinterpret_cast<float*>(sm + o.f), *dts = cum + kChunk, *wts = dts + kChunk;
     const int np = min(PT * 8, s.P8 - pb);                   // value dimensions of this CTA (multiple of 8)
-    const int nk = (s.N8 + 15) >> 4;
     pdl_sync();
     const int p0 = first_pos(k, b);
     const float A2 = k.A[h] * kLog2e, Dh = k.D[h], dtb = k.dt_bias[h];
@@ -371,11 +399,11 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(const SsmCall k) {
 
     const int n_chunks = (k.Sc + kChunk - 1) / kChunk;
     for (int ch = 0; ch < n_chunks; ch++) {
-        const int t0 = ch * kChunk, buf = ch & 1;
+        const int t0 = ch * kChunk, buf = NB == 2 ? ch & 1 : 0;
         if (tid < kChunk) dts[tid] = t0 + tid < k.Sc ? softplus_f(dt_next + dtb) : 0.0f;
         cp_wait<0>();
         __syncthreads();                                     // tiles, state and dt are in place; the other buffers are free
-        if (ch + 1 < n_chunks) { fetch(t0 + kChunk, buf ^ 1); dt_next = raw_dt(t0 + kChunk); }
+        if (ch + 1 < n_chunks) { if (NB == 2) fetch(t0 + kChunk, buf ^ 1); dt_next = raw_dt(t0 + kChunk); }
         float end;                                           // every warp: running sums in fp32
         {
             const float d0 = A2 * dts[2 * lane], d1 = A2 * dts[2 * lane + 1];
@@ -390,26 +418,35 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(const SsmCall k) {
         __syncthreads();
         const uint32_t cB = base + o.c + buf * kChunk * RN, bB = base + o.b + buf * kChunk * RN, xB = base + o.x + buf * kChunk * RP;
         const uint32_t sB = base + o.s;
-        // ---- output of this warp's 16 tokens
+        // ---- output of this warp's 16 tokens (their gates are asked for here and used at the end)
+        uint32_t z[PT][2];
+#pragma unroll
+        for (int j = 0; j < PT; j++)
+#pragma unroll
+            for (int u = 0; u < 2; u++) {
+                const int t = t0 + 16 * warp + lr + 8 * u;
+                z[j][u] = t < k.Sc && j * 8 < np ? *reinterpret_cast<const uint32_t*>(proj + (long)t * s.ld + xc + 8 * j + lc) : 0u;
+            }
         float y[PT][4] = {};
         uint32_t cf[NK][4];
 #pragma unroll
-        for (int q = 0; q < NK; q++)
-            if (q < nk) {
-                ldsm4(cB + (uint32_t)(16 * warp + (lane & 15)) * RN + (q * 16 + (lane >> 4) * 8) * 2, cf[q]);
+        for (int q = 0; q < NK; q++) {
+            ldsm4(cB + (uint32_t)(16 * warp + (lane & 15)) * RN + (q * 16 + (lane >> 4) * 8) * 2, cf[q]);
+            // (here and below) products into one accumulator lie PT apart, and nothing depends on the true sizes: straight-line
+            // code in which loads and products of independent accumulators overlap; the padding of the tiles is zero
+#pragma unroll
+            for (int part = 0; part < 2; part++) {
+                uint32_t f[PT / 2][4];
 #pragma unroll
                 for (int j = 0; j < PT; j += 2)
-                    if (j * 8 < np) {
-                        const uint32_t ad = sB + (uint32_t)(q * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * RP + (j * 8 + (lane >> 4) * 8) * 2;
-                        uint32_t f[4];
-                        ldsm4t(ad, f);
-                        mma_bf16(y[j], cf[q][0], cf[q][1], cf[q][2], cf[q][3], f[0], f[1]);
-                        mma_bf16(y[j + 1], cf[q][0], cf[q][1], cf[q][2], cf[q][3], f[2], f[3]);
-                        ldsm4t(ad + NK * 16 * RP, f);
-                        mma_bf16(y[j], cf[q][0], cf[q][1], cf[q][2], cf[q][3], f[0], f[1]);
-                        mma_bf16(y[j + 1], cf[q][0], cf[q][1], cf[q][2], cf[q][3], f[2], f[3]);
-                    }
+                    ldsm4t(sB + (uint32_t)(part * NK * 16 + q * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * RP + (j * 8 + (lane >> 4) * 8) * 2, f[j / 2]);
+#pragma unroll
+                for (int j = 0; j < PT; j += 2) {
+                    mma_bf16(y[j], cf[q][0], cf[q][1], cf[q][2], cf[q][3], f[j / 2][0], f[j / 2][1]);
+                    mma_bf16(y[j + 1], cf[q][0], cf[q][1], cf[q][2], cf[q][3], f[j / 2][2], f[j / 2][3]);
+                }
             }
+        }
         const int tr = 16 * warp + lr;                       // rows tr and tr + 8 of the chunk
         const float ct0 = cum[tr], ct1 = cum[tr + 8];
         {
@@ -418,38 +455,38 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(const SsmCall k) {
             for (int j = 0; j < PT; j++) { y[j][0] *= e0; y[j][1] *= e0; y[j][2] *= e1; y[j][3] *= e1; }
         }
         for (int q = 0; q <= warp; q++) {                    // 16 source tokens at a time
-            float gm[2][4] = {};
+            float gm[2][4] = {}, g2[2][4] = {};
 #pragma unroll
-            for (int n = 0; n < NK; n++)
-                if (n < nk) {
-                    uint32_t f[4];
-                    ldsm4(bB + (uint32_t)(16 * q + (lane & 7) + (lane >> 4) * 8) * RN + (n * 16 + ((lane >> 3) & 1) * 8) * 2, f);
-                    mma_bf16(gm[0], cf[n][0], cf[n][1], cf[n][2], cf[n][3], f[0], f[1]);
-                    mma_bf16(gm[1], cf[n][0], cf[n][1], cf[n][2], cf[n][3], f[2], f[3]);
-                }
-            uint32_t hi[4], lo[4];
+            for (int n = 0; n < NK; n++) {
+                uint32_t f[4];
+                ldsm4(bB + (uint32_t)(16 * q + (lane & 7) + (lane >> 4) * 8) * RN + (n * 16 + ((lane >> 3) & 1) * 8) * 2, f);
+                mma_bf16(n & 1 ? g2[0] : gm[0], cf[n][0], cf[n][1], cf[n][2], cf[n][3], f[0], f[1]);
+                mma_bf16(n & 1 ? g2[1] : gm[1], cf[n][0], cf[n][1], cf[n][2], cf[n][3], f[2], f[3]);
+            }
+            uint32_t xf[PT / 2][4];
+#pragma unroll
+            for (int j = 0; j < PT; j += 2)
+                ldsm4t(xB + (uint32_t)(16 * q + (lane & 7) + ((lane >> 3) & 1) * 8) * RP + (j * 8 + (lane >> 4) * 8) * 2, xf[j / 2]);
+            uint32_t wf[2][4];                               // hi, lo
 #pragma unroll
             for (int u = 0; u < 2; u++) {
                 float w[4];
 #pragma unroll
                 for (int i = 0; i < 4; i++) {
                     const int sr = 16 * q + 8 * u + lc + (i & 1), t = tr + 8 * (i >> 1);
-                    float v = sr <= t ? gm[u][i] * (ex2_fast((i >> 1 ? ct1 : ct0) - cum[sr]) * dts[sr]) : 0.0f;
+                    float v = sr <= t ? (gm[u][i] + g2[u][i]) * (ex2_fast((i >> 1 ? ct1 : ct0) - cum[sr]) * dts[sr]) : 0.0f;
                     if (sr == t) v += Dh;
                     w[i] = v;
                 }
-                split2(w[0], w[1], &hi[2 * u], &lo[2 * u]);
-                split2(w[2], w[3], &hi[2 * u + 1], &lo[2 * u + 1]);
+                split2(w[0], w[1], &wf[0][2 * u], &wf[1][2 * u]);
+                split2(w[2], w[3], &wf[0][2 * u + 1], &wf[1][2 * u + 1]);
             }
 #pragma unroll
-            for (int j = 0; j < PT; j += 2)
-                if (j * 8 < np) {
-                    uint32_t f[4];
-                    ldsm4t(xB + (uint32_t)(16 * q + (lane & 7) + ((lane >> 3) & 1) * 8) * RP + (j * 8 + (lane >> 4) * 8) * 2, f);
-                    mma_bf16(y[j], hi[0], hi[1], hi[2], hi[3], f[0], f[1]);
-                    mma_bf16(y[j + 1], hi[0], hi[1], hi[2], hi[3], f[2], f[3]);
-                    mma_bf16(y[j], lo[0], lo[1], lo[2], lo[3], f[0], f[1]);
-                    mma_bf16(y[j + 1], lo[0], lo[1], lo[2], lo[3], f[2], f[3]);
+            for (int part = 0; part < 2; part++)
+#pragma unroll
+                for (int j = 0; j < PT; j += 2) {
+                    mma_bf16(y[j], wf[part][0], wf[part][1], wf[part][2], wf[part][3], xf[j / 2][0], xf[j / 2][1]);
+                    mma_bf16(y[j + 1], wf[part][0], wf[part][1], wf[part][2], wf[part][3], xf[j / 2][2], xf[j / 2][3]);
                 }
         }
         // ---- gate and store
@@ -459,10 +496,9 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(const SsmCall k) {
 #pragma unroll
                 for (int u = 0; u < 2; u++) {
                     const int t = t0 + tr + 8 * u;
-                    if (t >= k.Sc) continue;
-                    const uint32_t z = *reinterpret_cast<const uint32_t*>(proj + (long)t * s.ld + xc + 8 * j + lc);
-                    *reinterpret_cast<uint32_t*>((bf16*)k.y + ((long)b * k.Sc + t) * s.inner + xc + 8 * j + lc) =
-                        bf_pack(y[j][2 * u] * silu_t<true>(bf_lo(z)), y[j][2 * u + 1] * silu_t<true>(bf_hi(z)));
+                    if (t < k.Sc)
+                        *reinterpret_cast<uint32_t*>((bf16*)k.y + ((long)b * k.Sc + t) * s.inner + xc + 8 * j + lc) =
+                            bf_pack(y[j][2 * u] * silu_t<true>(bf_lo(z[j][u])), y[j][2 * u + 1] * silu_t<true>(bf_hi(z[j][u])));
                 }
         // ---- state after the chunk
         {
@@ -479,30 +515,28 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(const SsmCall k) {
             uint32_t xf[PT / 2][4];
 #pragma unroll
             for (int j = 0; j < PT; j += 2)
-                if (j * 8 < np)
-                    ldsm4t(xB + (uint32_t)(16 * q + (lane & 7) + ((lane >> 3) & 1) * 8) * RP + (j * 8 + (lane >> 4) * 8) * 2, xf[j / 2]);
+                ldsm4t(xB + (uint32_t)(16 * q + (lane & 7) + ((lane >> 3) & 1) * 8) * RP + (j * 8 + (lane >> 4) * 8) * 2, xf[j / 2]);
             const float2 w0 = *reinterpret_cast<const float2*>(wts + 16 * q + lc), w1 = *reinterpret_cast<const float2*>(wts + 16 * q + lc + 8);
 #pragma unroll
             for (int m = 0; m < MT; m++) {
-                if (16 * (MT * warp + m) >= s.N8) continue;
-                uint32_t f[4], hi[4], lo[4];
+                uint32_t f[4], wb[2][4];
                 ldsm4t(bB + (uint32_t)(16 * q + (lane & 7) + (lane >> 4) * 8) * RN + (16 * (MT * warp + m) + ((lane >> 3) & 1) * 8) * 2, f);
 #pragma unroll
                 for (int i = 0; i < 4; i++) {
                     const float2 w = i < 2 ? w0 : w1;
-                    split2(bf_lo(f[i]) * w.x, bf_hi(f[i]) * w.y, &hi[i], &lo[i]);
+                    split2(bf_lo(f[i]) * w.x, bf_hi(f[i]) * w.y, &wb[0][i], &wb[1][i]);
                 }
 #pragma unroll
-                for (int j = 0; j < PT; j += 2)
-                    if (j * 8 < np) {
-                        mma_bf16(S[m][j], hi[0], hi[1], hi[2], hi[3], xf[j / 2][0], xf[j / 2][1]);
-                        mma_bf16(S[m][j + 1], hi[0], hi[1], hi[2], hi[3], xf[j / 2][2], xf[j / 2][3]);
-                        mma_bf16(S[m][j], lo[0], lo[1], lo[2], lo[3], xf[j / 2][0], xf[j / 2][1]);
-                        mma_bf16(S[m][j + 1], lo[0], lo[1], lo[2], lo[3], xf[j / 2][2], xf[j / 2][3]);
+                for (int part = 0; part < 2; part++)
+#pragma unroll
+                    for (int j = 0; j < PT; j += 2) {
+                        mma_bf16(S[m][j], wb[part][0], wb[part][1], wb[part][2], wb[part][3], xf[j / 2][0], xf[j / 2][1]);
+                        mma_bf16(S[m][j + 1], wb[part][0], wb[part][1], wb[part][2], wb[part][3], xf[j / 2][2], xf[j / 2][3]);
                     }
             }
         }
         __syncthreads();                                     // everyone has read the state (and this chunk's tiles)
+        if (NB == 1 && ch + 1 < n_chunks) fetch(t0 + kChunk, 0);
         stage_state();
     }
 #pragma unroll
@@ -517,20 +551,22 @@ __global__ void __launch_bounds__(128) ssm_chunk_kernel(const SsmCall k) {
     keep_history<bf16>(k, b, p0, blockIdx.x + gridDim.x * blockIdx.y, gridDim.x * gridDim.y);
 }
 
-template <class T, int NV, bool FUSED> int launch_scan(const SsmCall& c, cudaStream_t st) {
-    launch_k(ssm_scan_kernel<T, NV, FUSED>, dim3((c.s.P8 + 31) / 32, c.s.H, c.B), dim3(256), 0, st, c);
+template <class T, int NV, int PR, bool FUSED> int launch_scan(const SsmCall& c, cudaStream_t st) {
+    launch_k(ssm_scan_kernel<T, NV, PR, FUSED>, dim3((c.s.P8 + 32 * PR - 1) / (32 * PR), c.s.H, c.B), dim3(256), 0, st, c);
     return launch_status();
 }
 template <class T, bool FUSED> int run_scan(const SsmCall& c, cudaStream_t st) {
-    if (c.s.N8 <= 32) return launch_scan<T, 1, FUSED>(c, st);
-    if (c.s.N8 <= 64) return launch_scan<T, 2, FUSED>(c, st);
-    if (c.s.N8 <= 128) return launch_scan<T, 4, FUSED>(c, st);
-    return launch_scan<T, 8, FUSED>(c, st);
+    // one token: wide CTAs, whose convolution of B and C serves more rows, once there are enough of them
+    const bool wide = FUSED && (long)c.B * c.s.H * ((c.s.P8 + 63) / 64) > 2 * gemm_sm_count();
+    if (c.s.N8 <= 32) return wide ? launch_scan<T, 1, 2, FUSED>(c, st) : launch_scan<T, 1, 1, FUSED>(c, st);
+    if (c.s.N8 <= 64) return wide ? launch_scan<T, 2, 2, FUSED>(c, st) : launch_scan<T, 2, 1, FUSED>(c, st);
+    if (c.s.N8 <= 128) return wide ? launch_scan<T, 4, 2, FUSED>(c, st) : launch_scan<T, 4, 1, FUSED>(c, st);
+    return launch_scan<T, 8, 1, FUSED>(c, st);
 }
 
-template <int NK, int PT> int launch_chunk(const SsmCall& c, cudaStream_t st) {
-    constexpr size_t smem = chunk_smem(NK, PT).total;
-    auto kern = ssm_chunk_kernel<NK, PT>;
+template <int NK, int PT, int NB, int CTAS> int launch_chunk(const SsmCall& c, cudaStream_t st) {
+    constexpr size_t smem = chunk_smem(NK, PT, NB).total;
+    auto kern = ssm_chunk_kernel<NK, PT, NB, CTAS>;
     FLEXLLM_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     launch_k(kern, dim3((c.s.P8 + PT * 8 - 1) / (PT * 8), c.s.H, c.B), dim3(128), smem, st, c);
     return launch_status();
@@ -538,9 +574,11 @@ template <int NK, int PT> int launch_chunk(const SsmCall& c, cudaStream_t st) {
 template <class T> int run_chunks(const SsmCall&, cudaStream_t) { return FLEXLLM_ENOTSUP; }
 template <> int run_chunks<bf16>(const SsmCall& c, cudaStream_t st) {
     if (c.Sc < kScanTile) return FLEXLLM_ENOTSUP;
-    if (c.s.N8 <= 64) return launch_chunk<4, 8>(c, st);
-    if (c.s.N8 <= 128) return launch_chunk<8, 8>(c, st);
-    return launch_chunk<16, 4>(c, st);
+    // 64 value dimensions per CTA do the least work; 32 when those would not fill the SMs
+    const bool many = (long)c.B * c.s.H * ((c.s.P8 + 63) / 64) > gemm_sm_count();
+    if (c.s.N8 <= 64) return many ? launch_chunk<4, 8, 1, 2>(c, st) : launch_chunk<4, 4, 2, 2>(c, st);
+    if (c.s.N8 <= 128) return many ? launch_chunk<8, 8, 1, 2>(c, st) : launch_chunk<8, 4, 2, 2>(c, st);
+    return launch_chunk<16, 4, 1, 2>(c, st);
 }
 
 template <class T> int run_conv(const SsmCall& c, cudaStream_t st) {
