@@ -156,12 +156,12 @@ struct SsmCall {
     void* conv_state;                       // T [slot][taps][ch]: inputs of the convolution, position p in row p % taps
     const int32_t* ctx;                     // position of the first of the call's Sc tokens per sequence (0: the state starts at zero)
     int B, Sc;
-    void* xbc;                              // scratch T [rows][ch] (unused by the decode form)
+    void* xbc;                              // scratch T [rows][ch]
     void* y;                                // scratch T [rows][inner]: gated outputs before the norm
     void* out;                              // T [rows][inner]
 };
-// Sc == 1: convolution, state update and gate in one kernel; else convolution, then the recurrence (bf16: in chunks on the tensor
-// cores, fp32: token by token). Then the norm. States and histories of the call's sequences are advanced.
+// Convolution, then the recurrence and the gate (bf16 prompts: in chunks on the tensor cores; otherwise token by token), then the
+// norm. States and histories of the call's sequences are advanced.
 template <class T> int ssm_mixer(const SsmCall& c, cudaStream_t st);
 void ssm_layout(SsmShape* s);               // fills in the derived members
 bool ssm_supported(const SsmShape& s);

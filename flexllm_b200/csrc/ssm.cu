@@ -3,9 +3,10 @@
 //   S_t = exp(A dt) S_{t-1} + dt B_t x_t^T       y_t = S_t^T C_t + D x_t         (per head; A = -exp(A_log))
 //   out = rms norm in parts of (y * silu(z)) * gain
 // Decays, steps and states are fp32. x, B and C are rounded to the activation type after the convolution.
-//   one token per sequence : ssm_scan_kernel<FUSED>: convolution, state update, gate in one launch, then the norm
-//   prompts, bf16          : ssm_conv_kernel, then ssm_chunk_kernel on warp MMAs (chunks of 64 tokens, state in registers)
-//   prompts, otherwise     : ssm_conv_kernel, then ssm_scan_kernel token by token
+// ssm_conv_kernel, then
+//   prompts, bf16   : ssm_chunk_kernel on warp MMAs (chunks of 64 tokens, state in registers)
+//   otherwise       : ssm_scan_kernel token by token (decoding: one state read and write)
+// both with the gate in their epilogue, then ssm_norm_kernel.
 // A state row holds one value dimension: [head][value dimension][state]. The inputs of the convolution are kept in a ring of
 // `taps` rows per sequence, position p in row p % taps. A sequence at position 0 starts from zero whatever its slot holds.
 #include "float_common.cuh"
@@ -26,19 +27,10 @@ template <class T> __device__ __forceinline__ const T* conv_row(const SsmCall& k
     if (at >= p0) return (const T*)k.proj + ((long)b * k.Sc + (at - p0)) * k.s.ld + k.s.x_off;
     return (const T*)k.conv_state + ((long)b * k.s.taps + at % k.s.taps) * k.s.ch;
 }
-template <class T> __device__ __forceinline__ float conv_one(const SsmCall& k, int b, int p0, int pos, int c) {
-    float v = k.conv_b[c];
-    const int taps = k.s.taps;
-    for (int j = 0; j < taps; j++) {
-        const int at = pos - (taps - 1) + j;
-        if (at >= 0) v = __fmaf_rn(k.conv_w[(long)j * k.s.ch + c], to_f(conv_row<T>(k, b, p0, at)[c]), v);
-    }
-    return to_f(from_f<T>(silu_t<sizeof(T) == 2>(v)));
-}
 __device__ __forceinline__ int first_pos(const SsmCall& k, int b) { return max(0, k.ctx[b]); }
 
-// The last inputs of the call go to the history. Every CTA of sequence b takes a share (id of n). Callers run after all reads
-// of older history (a later launch), except in the decode form, whose one row is not among those it reads.
+// The last inputs of the call go to the history. Every CTA of sequence b takes a share (id of n); the convolution, which reads the
+// older history, was an earlier launch.
 template <class T> __device__ __forceinline__ void keep_history(const SsmCall& k, int b, int p0, int id, int n) {
     const SsmShape& s = k.s;
     const int rows = min(k.Sc, s.taps), vecs = s.ch >> 3;
@@ -134,38 +126,39 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const SsmCall k) {
 }
 
 // ---------------------------------------------------------------------------------------------------------------
-// Recurrence token by token: a CTA has 32 PR value dimensions of one head, 8 lanes share a state row (NV float4 each). FUSED: one
-// token per sequence, with its convolution.
-template <class T, int NV, int PR, bool FUSED>
+// Recurrence token by token, TT tokens staged at a time: a CTA has 32 value dimensions of one head, 8 lanes share a state row (NV
+// float4 each).
+template <class T, int NV, int TT>
 __global__ void __launch_bounds__(256) ssm_scan_kernel(const SsmCall k) {
     constexpr bool FAST = sizeof(T) == 2;
-    constexpr int TT = FUSED ? 1 : kScanTile, NW = 32 * NV, NP = 32 * PR;
+    constexpr int NW = 32 * NV;
     __shared__ __align__(16) float b_sm[TT][NW], c_sm[TT][NW];
-    __shared__ float x_sm[TT][NP], dt_sm[TT], dec_sm[TT];
+    __shared__ float x_sm[TT][32], dt_sm[TT], dec_sm[TT];
     const SsmShape& s = k.s;
     const int tid = threadIdx.x, h = blockIdx.y, b = blockIdx.z, g = h / (s.H / s.G);
-    const int pb = blockIdx.x * NP, pr = tid >> 3, ns = tid & 7;            // rows pr, pr + 32, ..
+    const int pb = blockIdx.x * 32, pr = tid >> 3, p = pb + pr, ns = tid & 7;
+    const bool on = p < s.P;
     pdl_sync();
     const int p0 = first_pos(k, b);
-    float* st = k.state + (((long)b * s.H + h) * s.P + pb + pr) * s.Np + 4 * ns;
-    float4 S[PR][NV];
+    float* st = k.state + (((long)b * s.H + h) * s.P + (on ? p : 0)) * s.Np;
+    float4 S[NV];
 #pragma unroll
-    for (int r = 0; r < PR; r++)
-#pragma unroll
-        for (int i = 0; i < NV; i++)
-            S[r][i] = pb + pr + 32 * r < s.P && p0 > 0 && 32 * i + 4 * ns < s.Np ? load4(st + (long)32 * r * s.Np + 32 * i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 0; i < NV; i++) {
+        const int n = 32 * i + 4 * ns;
+        S[i] = on && p0 > 0 && n < s.Np ? load4(st + n) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
     const float A = k.A[h], Dh = k.D[h], dtb = k.dt_bias[h];
     const int xc = h * s.P8 + pb, bc = s.inner + g * s.N8, cc = bc + s.G * s.N8;       // first channels of x, B and C
     for (int t0 = 0; t0 < k.Sc; t0 += TT) {
         const int nt = min(TT, k.Sc - t0);
         if (t0) __syncthreads();
-        for (int i = tid; i < nt * (2 * NW + NP); i += 256) {
-            const int t = i / (2 * NW + NP), j = i - t * (2 * NW + NP);
+        for (int i = tid; i < nt * (2 * NW + 32); i += 256) {
+            const int t = i / (2 * NW + 32), j = i - t * (2 * NW + 32);
             const int e = j < NW ? j : j < 2 * NW ? j - NW : j - 2 * NW;
             const bool in = j < 2 * NW ? e < s.N8 : pb + e < s.P8;
             const int c = (j < NW ? bc : j < 2 * NW ? cc : xc) + e;
             float v = 0.0f;
-            if (in) v = FUSED ? conv_one<T>(k, b, p0, p0, c) : to_f(((const T*)k.xbc)[((long)b * k.Sc + t0 + t) * s.ch + c]);
+            if (in) v = to_f(((const T*)k.xbc)[((long)b * k.Sc + t0 + t) * s.ch + c]);
             if (j < NW) b_sm[t][e] = v; else if (j < 2 * NW) c_sm[t][e] = v; else x_sm[t][e] = v;
         }
         if (tid < nt) {
@@ -176,41 +169,29 @@ __global__ void __launch_bounds__(256) ssm_scan_kernel(const SsmCall k) {
         }
         __syncthreads();
         for (int t = 0; t < nt; t++) {
-            const float dec = dec_sm[t];
-            float y[PR];
+            const float x = x_sm[t][pr], dec = dec_sm[t], dx = dt_sm[t] * x;
+            float y = 0.0f;
 #pragma unroll
-            for (int r = 0; r < PR; r++) {
-                const float dx = dt_sm[t] * x_sm[t][pr + 32 * r];
-                y[r] = 0.0f;
-#pragma unroll
-                for (int i = 0; i < NV; i++) {
-                    const float4 bv = load4(&b_sm[t][32 * i + 4 * ns]), cv = load4(&c_sm[t][32 * i + 4 * ns]);
-                    float4& q = S[r][i];
-                    q.x = __fmaf_rn(q.x, dec, bv.x * dx); q.y = __fmaf_rn(q.y, dec, bv.y * dx);
-                    q.z = __fmaf_rn(q.z, dec, bv.z * dx); q.w = __fmaf_rn(q.w, dec, bv.w * dx);
-                    y[r] = __fmaf_rn(q.x, cv.x, y[r]); y[r] = __fmaf_rn(q.y, cv.y, y[r]); y[r] = __fmaf_rn(q.z, cv.z, y[r]); y[r] = __fmaf_rn(q.w, cv.w, y[r]);
-                }
+            for (int i = 0; i < NV; i++) {
+                const float4 bv = load4(&b_sm[t][32 * i + 4 * ns]), cv = load4(&c_sm[t][32 * i + 4 * ns]);
+                S[i].x = __fmaf_rn(S[i].x, dec, bv.x * dx); S[i].y = __fmaf_rn(S[i].y, dec, bv.y * dx);
+                S[i].z = __fmaf_rn(S[i].z, dec, bv.z * dx); S[i].w = __fmaf_rn(S[i].w, dec, bv.w * dx);
+                y = __fmaf_rn(S[i].x, cv.x, y); y = __fmaf_rn(S[i].y, cv.y, y); y = __fmaf_rn(S[i].z, cv.z, y); y = __fmaf_rn(S[i].w, cv.w, y);
             }
 #pragma unroll
-            for (int o = 4; o > 0; o >>= 1)
-#pragma unroll
-                for (int r = 0; r < PR; r++) y[r] += __shfl_xor_sync(0xffffffffu, y[r], o);
-#pragma unroll
-            for (int r = 0; r < PR; r++) {
-                const int p = pb + pr + 32 * r;
-                if (ns != 0 || p >= s.P8) continue;
+            for (int o = 4; o > 0; o >>= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+            if (ns == 0 && p < s.P8) {
                 const long row = (long)b * k.Sc + t0 + t;
                 const int col = h * s.P8 + p;
                 const float z = to_f(((const T*)k.proj)[row * s.ld + col]);
-                ((T*)k.y)[row * s.inner + col] = from_f<T>(p < s.P ? __fmaf_rn(Dh, x_sm[t][pr + 32 * r], y[r]) * silu_t<FAST>(z) : 0.0f);
+                ((T*)k.y)[row * s.inner + col] = from_f<T>(on ? __fmaf_rn(Dh, x, y) * silu_t<FAST>(z) : 0.0f);
             }
         }
     }
-#pragma unroll
-    for (int r = 0; r < PR; r++)
+    if (on)
 #pragma unroll
         for (int i = 0; i < NV; i++)
-            if (pb + pr + 32 * r < s.P && 32 * i + 4 * ns < s.Np) store4(st + (long)32 * r * s.Np + 32 * i, S[r][i]);
+            if (32 * i + 4 * ns < s.Np) store4(st + 32 * i + 4 * ns, S[i]);
     keep_history<T>(k, b, p0, blockIdx.x + gridDim.x * blockIdx.y, gridDim.x * gridDim.y);
 }
 
@@ -551,17 +532,15 @@ __global__ void __launch_bounds__(128, CTAS) ssm_chunk_kernel(const SsmCall k) {
     keep_history<bf16>(k, b, p0, blockIdx.x + gridDim.x * blockIdx.y, gridDim.x * gridDim.y);
 }
 
-template <class T, int NV, int PR, bool FUSED> int launch_scan(const SsmCall& c, cudaStream_t st) {
-    launch_k(ssm_scan_kernel<T, NV, PR, FUSED>, dim3((c.s.P8 + 32 * PR - 1) / (32 * PR), c.s.H, c.B), dim3(256), 0, st, c);
+template <class T, int NV, int TT> int launch_scan(const SsmCall& c, cudaStream_t st) {
+    launch_k(ssm_scan_kernel<T, NV, TT>, dim3((c.s.P8 + 31) / 32, c.s.H, c.B), dim3(256), 0, st, c);
     return launch_status();
 }
-template <class T, bool FUSED> int run_scan(const SsmCall& c, cudaStream_t st) {
-    // one token: wide CTAs, whose convolution of B and C serves more rows, once there are enough of them
-    const bool wide = FUSED && (long)c.B * c.s.H * ((c.s.P8 + 63) / 64) > 2 * gemm_sm_count();
-    if (c.s.N8 <= 32) return wide ? launch_scan<T, 1, 2, FUSED>(c, st) : launch_scan<T, 1, 1, FUSED>(c, st);
-    if (c.s.N8 <= 64) return wide ? launch_scan<T, 2, 2, FUSED>(c, st) : launch_scan<T, 2, 1, FUSED>(c, st);
-    if (c.s.N8 <= 128) return wide ? launch_scan<T, 4, 2, FUSED>(c, st) : launch_scan<T, 4, 1, FUSED>(c, st);
-    return launch_scan<T, 8, 1, FUSED>(c, st);
+template <class T, int TT> int run_scan(const SsmCall& c, cudaStream_t st) {
+    if (c.s.N8 <= 32) return launch_scan<T, 1, TT>(c, st);
+    if (c.s.N8 <= 64) return launch_scan<T, 2, TT>(c, st);
+    if (c.s.N8 <= 128) return launch_scan<T, 4, TT>(c, st);
+    return launch_scan<T, 8, TT>(c, st);
 }
 
 template <int NK, int PT, int NB, int CTAS> int launch_chunk(const SsmCall& c, cudaStream_t st) {
@@ -608,16 +587,12 @@ template <class T> int ssm_mixer(const SsmCall& c, cudaStream_t st) {
     const SsmShape& s = c.s;
     FLEXLLM_REQUIRE(s.H > 0 && s.P > 0 && s.N > 0 && s.G > 0 && s.H % s.G == 0 && s.taps > 0 && s.parts > 0 && (s.H * s.P) % s.parts == 0);
     FLEXLLM_REQUIRE(c.proj && c.conv_w && c.conv_b && c.dt_bias && c.A && c.D && c.gain && c.state && c.conv_state && c.ctx && c.y && c.out);
-    FLEXLLM_REQUIRE(c.B > 0 && c.Sc > 0 && (c.Sc == 1 || c.xbc));
+    FLEXLLM_REQUIRE(c.B > 0 && c.Sc > 0 && c.xbc);
     if (!ssm_supported(s) || c.B > 65535 || c.Sc > 65535 * kConvTokens) return FLEXLLM_ENOTSUP;
-    if (c.Sc == 1) {
-        TRY_RC((run_scan<T, true>(c, st)));
-    } else {
-        TRY_RC(run_conv<T>(c, st));
-        int rc = run_chunks<T>(c, st);
-        if (rc == FLEXLLM_ENOTSUP) rc = run_scan<T, false>(c, st);
-        TRY_RC(rc);
-    }
+    TRY_RC(run_conv<T>(c, st));
+    int rc = c.Sc == 1 ? run_scan<T, 1>(c, st) : run_chunks<T>(c, st);
+    if (rc == FLEXLLM_ENOTSUP) rc = run_scan<T, kScanTile>(c, st);
+    TRY_RC(rc);
     launch_k(ssm_norm_kernel<T>, dim3(c.B * c.Sc), dim3(256), (size_t)(s.parts + 8) * 4, st, c);
     return launch_status();
 }
