@@ -1,4 +1,4 @@
-// Decoder family with floating-point weights (the Pibidra design) on the common model runner: create, load, then the same
+// Decoder family with floating-point weights (the Pibidra and Sabisun designs) on the common model runner: create, load, then the same
 // prefill / decode / generate calls as every model, plus steps of any length with logits at chosen places.
 #pragma once
 #include "common.hpp"
